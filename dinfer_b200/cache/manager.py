@@ -31,10 +31,13 @@ from .block_pool import BlockPool, PoolError, StateSlots
 class GroupSpec:
     """``window`` None: every token's keys are kept; else the last ``window`` (the token itself counts).
     ``block_size`` None: the manager's page size; else this group's own.  ``keep_first``: with a window, the first
-    so many tokens of a request stay visible behind it, so the pages that hold them are never given back early."""
+    so many tokens of a request stay visible behind it, so the pages that hold them are never given back early.
+    ``chunked``: the window is a chunk of positions counted from the sequence's first; the pages before the chunk of the
+    next token to come are given back."""
     window: Optional[int] = None
     block_size: Optional[int] = None
     keep_first: int = 0
+    chunked: bool = False
 
 
 @dataclass
@@ -102,7 +105,8 @@ class CacheManager:
         w = self.groups[group].window
         if w is None:
             return 0
-        first_pos = max(0, num_computed - w + 1)      # oldest key a query at num_computed still sees
+        # oldest key a query at num_computed still sees
+        first_pos = num_computed // w * w if self.groups[group].chunked else max(0, num_computed - w + 1)
         return first_pos // self.block_sizes[group]
 
     def _need(self, held: Optional[_Held], total_tokens: int) -> List[int]:

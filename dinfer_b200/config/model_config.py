@@ -896,3 +896,179 @@ class PorovikConfig:
         if self.eos_token_ids:
             d["eos_token_id"] = list(self.eos_token_ids)
         return d
+
+
+# ---------------------------------------------------------------- Datozen
+
+@dataclass(frozen=True)
+class ChunkAttentionSizes:
+    """An ``attention`` mixer of Datozen: grouped heads with a norm of q and k, a rotation of the first ``rot_dims``
+    elements in halves (stretched by a ramp with ``scaling``), chunks of ``chunk`` positions, values of ``vdim`` elements
+    that turn with their position, a learned sink and one gate per head."""
+    heads: int
+    kv_heads: int
+    dim: int
+    vdim: int
+    scale: float
+    chunk: int
+    rot_base: float
+    rot_dims: int
+    scaling: Optional[RampScaling] = None
+
+    @classmethod
+    def from_dict(cls, m: Dict[str, Any], where: str) -> "ChunkAttentionSizes":
+        heads, dim = _take(m, "heads", int), _take(m, "dim", int)
+        rot = _section(m, "rot", where)
+        sc = _section(rot, "scaling", where, optional=True)
+        s = cls(heads=heads, kv_heads=_take(m, "kv_heads", int, heads), dim=dim, vdim=_take(m, "vdim", int, dim),
+                scale=_take(m, "scale", float), chunk=_take(_section(m, "mask", where), "size", int),
+                rot_base=_take(rot, "base", float), rot_dims=_take(rot, "dims", int),
+                scaling=RampScaling.from_dict(sc, where) if sc else None)
+        _positive(s, ("heads", "kv_heads", "dim", "vdim", "chunk", "rot_base"), where)
+        if s.heads % s.kv_heads:
+            raise ConfigError(f"config.json: {where}heads {s.heads} must be a multiple of kv_heads {s.kv_heads}")
+        if s.rot_dims <= 0 or s.rot_dims % 2 or s.rot_dims > s.dim:
+            raise ConfigError(f"config.json: {where}rot.dims {s.rot_dims} must be even and at most dim {s.dim}")
+        if s.vdim % 2:
+            raise ConfigError(f"config.json: {where}vdim {s.vdim} must be even (the values turn in pairs)")
+        return s
+
+    def to_dict(self) -> Dict[str, Any]:
+        rot = {"base": self.rot_base, "dims": self.rot_dims}
+        if self.scaling:
+            rot["scaling"] = self.scaling.to_dict()
+        return {"heads": self.heads, "kv_heads": self.kv_heads, "dim": self.dim, "vdim": self.vdim, "scale": self.scale,
+                "rot": rot, "mask": {"size": self.chunk}}
+
+
+@dataclass(frozen=True)
+class GroupedExpertSizes:
+    """A ``moe`` feed-forward of Datozen: ``experts`` gated experts ``ff`` wide and ``identity`` experts without tensors, of
+    which a token uses ``top`` out of the ``keep`` best of ``groups`` groups; ``shared_ff`` > 0: a shared expert."""
+    ff: int
+    experts: int
+    top: int
+    identity: int = 0
+    groups: int = 1
+    keep: int = 1
+    shared_ff: int = 0
+    kind: str = "moe"
+
+    @classmethod
+    def from_dict(cls, m: Dict[str, Any], where: str) -> "GroupedExpertSizes":
+        router = _section(m, "router", where)
+        groups = _section(router, "groups", where, optional=True)
+        shared = _section(m, "shared", where, optional=True)
+        s = cls(ff=_take(_section(m, "expert", where), "ff", int), experts=_take(router, "experts", int),
+                top=_take(router, "top", int), identity=_take(router, "identity", int, 0),
+                groups=_take(groups, "count", int) if groups else 1, keep=_take(groups, "keep", int) if groups else 1,
+                shared_ff=_take(shared, "ff", int) if shared else 0)
+        _positive(s, ("ff", "experts", "top", "groups", "keep"), where)
+        if s.identity < 0 or s.shared_ff < 0:
+            raise ConfigError(f"config.json: {where}router.identity and shared.ff must not be negative")
+        every = s.experts + s.identity
+        if every % s.groups or s.keep > s.groups:
+            raise ConfigError(f"config.json: {where}router.groups: {s.groups} must divide the {every} experts (identity experts "
+                              f"included) and keep {s.keep} be at most as many")
+        if s.top > s.keep * (every // s.groups):
+            raise ConfigError(f"config.json: {where}router.top {s.top} is more than the kept groups hold")
+        return s
+
+    def to_dict(self) -> Dict[str, Any]:
+        d = {"kind": "moe", "expert": {"ff": self.ff},
+             "router": {"experts": self.experts, "top": self.top, "identity": self.identity,
+                        "groups": {"count": self.groups, "keep": self.keep}}}
+        if self.shared_ff:
+            d["shared"] = {"ff": self.shared_ff}
+        return d
+
+
+@dataclass(frozen=True)
+class LayerLoop:
+    """Layers ``start`` to ``stop - 1`` run ``times`` times in a row."""
+    start: int
+    stop: int
+    times: int
+
+
+@dataclass(frozen=True)
+class DatozenLayer:
+    type: str
+    mixer: ChunkAttentionSizes
+    mlp: Any                        # FeedForwardSizes ("dense"), GroupedExpertSizes ("moe") or None
+
+
+@dataclass(frozen=True)
+class DatozenConfig:
+    """``config.json`` of a Datozen model: ``vocab``, ``width``, ``max_positions`` (rows of the learned position table),
+    ``norm.eps``, ``token_side.dim``, ``loop`` (layers that run several times) and the list ``layers``, each entry with its
+    ``type`` (``attention``), the mixer's sizes and its feed-forward (``mlp``: dense, a mixture of experts, or null)."""
+    vocab: int
+    width: int
+    norm_eps: float
+    max_positions: int
+    side_dim: int
+    layers: Tuple[DatozenLayer, ...]
+    loop: Optional[LayerLoop] = None
+    eos_token_ids: Tuple[int, ...] = ()
+    architecture: str = "Datozen"
+
+    MIXER_TYPES = {"attention": ChunkAttentionSizes}
+
+    @classmethod
+    def from_dict(cls, d: Dict[str, Any]) -> "DatozenConfig":
+        raw = d.get("layers")
+        if not isinstance(raw, list) or not raw:
+            raise ConfigError("config.json: 'layers' must be a non-empty list")
+        layers = []
+        for i, l in enumerate(raw):
+            where = f"layers[{i}]: "
+            if not isinstance(l, dict):
+                raise ConfigError(f"config.json: {where}must be an object")
+            kind = _take(l, "type", str)
+            if kind not in cls.MIXER_TYPES:
+                raise ConfigError(f"config.json: {where}unknown type {kind!r} ({', '.join(cls.MIXER_TYPES)})")
+            mixer = cls.MIXER_TYPES[kind].from_dict(_section(l, "mixer", where), where)
+            mlp = _section(l, "mlp", where, optional=True)
+            ff = None
+            if mlp is not None:
+                ff = GroupedExpertSizes.from_dict(mlp, where) if mlp.get("kind") == "moe" else FeedForwardSizes.from_dict(mlp, where)
+            layers.append(DatozenLayer(kind, mixer, ff))
+        lp = _section(d, "loop", "", optional=True)
+        loop = LayerLoop(*(_take(lp, k, int) for k in ("start", "stop", "times"))) if lp else None
+        if loop is not None and not (0 <= loop.start < loop.stop <= len(layers) and loop.times >= 1):
+            raise ConfigError(f"config.json: loop: layers {loop.start} to {loop.stop} of {len(layers)}, {loop.times} times")
+        eos = d.get("eos_token_id")
+        eos_ids = (eos,) if isinstance(eos, int) and not isinstance(eos, bool) else \
+            tuple(int(x) for x in eos) if isinstance(eos, (list, tuple)) else ()
+        cfg = cls(vocab=_take(d, "vocab", int), width=_take(d, "width", int),
+                  norm_eps=_take(_section(d, "norm", ""), "eps", float), max_positions=_take(d, "max_positions", int),
+                  side_dim=_take(_section(d, "token_side", ""), "dim", int), layers=tuple(layers), loop=loop,
+                  eos_token_ids=eos_ids, architecture=str(d.get("architecture") or (d.get("architectures") or ["Datozen"])[0]))
+        if cfg.vocab <= 0 or cfg.width <= 0 or cfg.max_positions <= 1 or cfg.side_dim <= 0:
+            raise ConfigError("config.json: vocab, width and token_side.dim must be positive, max_positions at least 2")
+        if not cfg.norm_eps > 0:
+            raise ConfigError(f"config.json: norm.eps must be positive, got {cfg.norm_eps}")
+        return cfg
+
+    def schedule(self) -> Tuple[int, ...]:
+        """The layers in the order in which they run."""
+        n = len(self.layers)
+        if self.loop is None:
+            return tuple(range(n))
+        lp = self.loop
+        return tuple(range(lp.start)) + tuple(range(lp.start, lp.stop)) * lp.times + tuple(range(lp.stop, n))
+
+    def to_dict(self) -> Dict[str, Any]:
+        def mlp(f):
+            if f is None:
+                return None
+            return {"kind": "dense", "ff": f.ff} if f.kind == "dense" else f.to_dict()
+        d = {"architecture": self.architecture, "vocab": self.vocab, "width": self.width, "norm": {"eps": self.norm_eps},
+             "max_positions": self.max_positions, "token_side": {"dim": self.side_dim},
+             "layers": [{"type": l.type, "mixer": l.mixer.to_dict(), "mlp": mlp(l.mlp)} for l in self.layers]}
+        if self.loop is not None:
+            d["loop"] = {"start": self.loop.start, "stop": self.loop.stop, "times": self.loop.times}
+        if self.eos_token_ids:
+            d["eos_token_id"] = list(self.eos_token_ids)
+        return d

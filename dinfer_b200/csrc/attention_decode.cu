@@ -37,8 +37,9 @@ struct Params {
   const __nv_bfloat16* cache;
   const int* block_table; int max_blocks;
   const int* cu_seqlens; const int* seq_lens;
-  int H, Hkv, group, block_size, bs_log2, window;
-  int sink;          // one more softmax term of score 0 without a value (the TMA variant)
+  int H, Hkv, group, block_size, bs_log2, window, chunked;
+  int sink;          // one more softmax term without a value, of score sinks[head] (null: 0) (the TMA variant)
+  const float* sinks;
   float scale_log2;
   const float* slopes;   // [H] or null: a distance bias, score - slopes[h] * (i - j) (the TMA variant)
   int splits;
@@ -139,7 +140,7 @@ __global__ void __launch_bounds__(NT, 2) attention_decode_kernel(const Params p)
   if (p.cu_seqlens[b + 1] - t0 != 1) return;               // not a decoded token: another kernel's request
   const int seq_len = p.seq_lens[b];
   const int pos = seq_len - 1;
-  const int lo = p.window > 0 ? max(0, pos - p.window + 1) : 0, hi = seq_len;
+  const int lo = first_key(pos, p.window, p.chunked), hi = seq_len;
   const int* table = p.block_table + (int64_t)b * p.max_blocks;
   int tile_begin = lo / BN, tile_end = (hi + BN - 1) / BN;
   {
@@ -455,7 +456,7 @@ attention_decode_tma_kernel(const __grid_constant__ CUtensorMap map_kv, const Pa
   if (p.splits > 1) cluster_arrive_relaxed();
   const int seq_len = p.seq_lens[b];
   const int pos = seq_len - 1;
-  const int lo = p.window > 0 ? max(0, pos - p.window + 1) : 0, hi = seq_len;
+  const int lo = first_key(pos, p.window, p.chunked), hi = seq_len;
   const int* table = p.block_table + (int64_t)b * p.max_blocks;
   int tile_begin = lo / BN, tile_end = (hi + BN - 1) / BN;
   {
@@ -687,7 +688,7 @@ attention_decode_tma_kernel(const __grid_constant__ CUtensorMap map_kv, const Pa
         acc += sm_o[(w * NHEADS + head) * D + d] * f;
       }
       if (!clustered) {
-        if (p.sink) L += exp2f(-M);                           // the sink: exp(0 - m), in the denominator only
+        if (p.sink) L += exp2f(sink_log2(p.sinks, hk * p.group + head) - M);   // the sink, in the denominator only
         p.out[(int64_t)t0 * p.ldo + (int64_t)(hk * p.group + head) * D + d] = __float2bfloat16_rn(L > 0.f ? acc / L : 0.f);
       } else {
         const int owner = idx / share;
@@ -726,7 +727,7 @@ attention_decode_tma_kernel(const __grid_constant__ CUtensorMap map_kv, const Pa
         L += recv_ml[(sp * p.group + head) * 2 + 1] * f;
         acc += recv[sp * share + i] * f;
       }
-      if (p.sink) L += exp2f(-M);
+      if (p.sink) L += exp2f(sink_log2(p.sinks, hk * p.group + head) - M);
       p.out[(int64_t)t0 * p.ldo + (int64_t)(hk * p.group + head) * D + d] = __float2bfloat16_rn(L > 0.f ? acc / L : 0.f);
     }
   }
@@ -847,7 +848,7 @@ DINFER_API int dinfer_attention_decode(const void* q, int64_t ldq, void* out, in
   p.cu_seqlens = cu_seqlens; p.seq_lens = seq_lens; p.H = H; p.Hkv = Hkv; p.group = H / Hkv;
   p.block_size = block_size; p.bs_log2 = 0;
   while ((1 << p.bs_log2) < block_size) ++p.bs_log2;
-  p.window = window; p.sink = 0; p.scale_log2 = scale * 1.4426950408889634f; p.splits = splits;
+  p.window = window; p.chunked = 0; p.sink = 0; p.sinks = nullptr; p.scale_log2 = scale * 1.4426950408889634f; p.splits = splits;
   p.slopes = nullptr;
   p.part_o = scratch_floats;
   p.part_ml = scratch_floats ? scratch_floats + (int64_t)B * H * splits * D : nullptr;
@@ -860,12 +861,13 @@ DINFER_API int dinfer_attention_decode(const void* q, int64_t ldq, void* out, in
 // The TMA variant (pages of at least 8 tokens): no scratch (the splits fold inside a cluster, at most
 // 16 of them), plus the number of pages of the cache tensor (for the tensor map) and the device status
 // word that a bounded wait sets when it runs out.
-// sink != 0: the softmax has one more term of score 0 that carries no value.
+// chunked: window is the size of the chunks (see first_key).
+// sink != 0: the softmax has one more term that carries no value, of score sinks[h] (f32 [H]; null: 0).
 // slopes: f32 [H] or null; with them score_ij - slopes[h] * (i - j).
 DINFER_API int dinfer_attention_decode_tma_bias(const void* q, int64_t ldq, void* out, int64_t ldo, const void* cache,
                                                 int64_t num_blocks, const int* block_table, int max_blocks,
                                                 const int* cu_seqlens, const int* seq_lens, int B, int H, int Hkv, int D,
-                                                int block_size, float scale, int window, int sink, const float* slopes,
+                                                int block_size, float scale, int window, int chunked, int sink, const float* sinks, const float* slopes,
                                                 int splits, int* status, cudaStream_t stream);
 
 DINFER_API int dinfer_attention_decode_tma_sink(const void* q, int64_t ldq, void* out, int64_t ldo, const void* cache,
@@ -874,13 +876,13 @@ DINFER_API int dinfer_attention_decode_tma_sink(const void* q, int64_t ldq, void
                                                 int block_size, float scale, int window, int sink, int splits,
                                                 int* status, cudaStream_t stream) {
   return dinfer_attention_decode_tma_bias(q, ldq, out, ldo, cache, num_blocks, block_table, max_blocks, cu_seqlens, seq_lens,
-                                          B, H, Hkv, D, block_size, scale, window, sink, nullptr, splits, status, stream);
+                                          B, H, Hkv, D, block_size, scale, window, 0, sink, nullptr, nullptr, splits, status, stream);
 }
 
 DINFER_API int dinfer_attention_decode_tma_bias(const void* q, int64_t ldq, void* out, int64_t ldo, const void* cache,
                                                 int64_t num_blocks, const int* block_table, int max_blocks,
                                                 const int* cu_seqlens, const int* seq_lens, int B, int H, int Hkv, int D,
-                                                int block_size, float scale, int window, int sink, const float* slopes,
+                                                int block_size, float scale, int window, int chunked, int sink, const float* sinks, const float* slopes,
                                                 int splits, int* status, cudaStream_t stream) {
   if (B <= 0 || H <= 0 || Hkv <= 0 || H % Hkv || max_blocks <= 0 || num_blocks <= 0)
     return refuse(DINFER_BAD_ARGUMENT, "attention_decode_tma: bad sizes B=%d H=%d Hkv=%d", B, H, Hkv);
@@ -915,7 +917,7 @@ DINFER_API int dinfer_attention_decode_tma_bias(const void* q, int64_t ldq, void
   p.cu_seqlens = cu_seqlens; p.seq_lens = seq_lens; p.H = H; p.Hkv = Hkv; p.group = H / Hkv;
   p.block_size = block_size; p.bs_log2 = 0;
   while ((1 << p.bs_log2) < block_size) ++p.bs_log2;
-  p.window = window; p.sink = sink; p.scale_log2 = scale * 1.4426950408889634f; p.splits = splits;
+  p.window = window; p.chunked = chunked; p.sink = sink; p.sinks = sinks; p.scale_log2 = scale * 1.4426950408889634f; p.splits = splits;
   p.slopes = slopes;
   p.part_o = nullptr; p.part_ml = nullptr; p.counters = nullptr; p.status = status;
   const int nh8 = (p.group + 7) / 8;

@@ -5,9 +5,9 @@
 // One warp owns one (token, query head): the lanes split the head's D elements, keys are visited
 // four at a time in position order with an online softmax; scores, softmax and the output sum are
 // 32-bit (expf, not the fast intrinsic).  A query at position p sees the keys [max(0, p-window+1), p]
-// of its own request, read through the request's block table.  Values may be Dv wide where keys are D wide (the
+// of its own request (`chunked`: those of its own chunk of `window` positions), read through the request's block table.  Values may be Dv wide where keys are D wide (the
 // cache's rows are then Dc = max(D, Dv) wide); with `sink` the softmax has one more term of score 0 and no value:
-// p_j = exp(s_j) / (1 + sum exp(s_j)).  With `slopes` (one number per query head) a distance bias is taken off every
+// p_j = exp(s_j) / (1 + sum exp(s_j)); `sinks` gives that term a score of its own per query head.  With `slopes` (one number per query head) a distance bias is taken off every
 // score: s_ij - slopes[h] * (i - j).
 //
 // Counterpart in the reference: the any-D reference kernels crates/kernels/cuda/gqa.cu:956-1118.
@@ -26,7 +26,7 @@ attention_generic_kernel(const T* __restrict__ q, int64_t ldq, T* __restrict__ o
                          const T* __restrict__ cache, const int* __restrict__ block_table, int max_blocks,
                          const int* __restrict__ cu_seqlens, const int* __restrict__ positions,
                          int num_reqs, int H, int Hkv, int D, int Dv, int Dc, int block_size, float scale, int window,
-                         int sink, const float* __restrict__ slopes) {
+                         int chunked, int sink, const float* __restrict__ sinks, const float* __restrict__ slopes) {
   const int t = blockIdx.x;
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   const int h = blockIdx.y * WARPS + warp;
@@ -40,7 +40,7 @@ attention_generic_kernel(const T* __restrict__ q, int64_t ldq, T* __restrict__ o
   const int* table = block_table + (int64_t)lo * max_blocks;
   const int hk = h / (H / Hkv);
   const int pos = positions[t];
-  const int first = (window > 0 && pos - window + 1 > 0) ? pos - window + 1 : 0;
+  const int first = first_key(pos, window, chunked);
   const float slope = slopes ? slopes[h] : 0.f;
 
   float qv[C], acc[C];
@@ -96,10 +96,11 @@ attention_generic_kernel(const T* __restrict__ q, int64_t ldq, T* __restrict__ o
     }
     m = m_new;
   }
-  if (sink) {                                                     // one more term, exp(0 - m), in the denominator only
-    const float m_new = fmaxf(m, 0.f);
+  if (sink) {                                                     // one more term, exp(score - m), in the denominator only
+    const float extra = sinks ? sinks[h] : 0.f;
+    const float m_new = fmaxf(m, extra);
     const float alpha = m == -INFINITY ? 0.f : expf(m - m_new);
-    l = l * alpha + expf(-m_new);
+    l = l * alpha + expf(extra - m_new);
 #pragma unroll
     for (int c = 0; c < C; ++c) acc[c] *= alpha;
   }
@@ -114,12 +115,12 @@ attention_generic_kernel(const T* __restrict__ q, int64_t ldq, T* __restrict__ o
 template <typename T, int C>
 int launch(const void* q, int64_t ldq, void* out, int64_t ldo, const void* cache, const int* block_table,
            int max_blocks, const int* cu_seqlens, const int* positions, int T_, int B, int H, int Hkv,
-           int D, int Dv, int Dc, int block_size, float scale, int window, int sink, const float* slopes,
+           int D, int Dv, int Dc, int block_size, float scale, int window, int chunked, int sink, const float* sinks, const float* slopes,
            cudaStream_t stream) {
   dim3 grid(T_, (H + WARPS - 1) / WARPS);
   attention_generic_kernel<T, C><<<grid, WARPS * 32, 0, stream>>>(
       (const T*)q, ldq, (T*)out, ldo, (const T*)cache, block_table, max_blocks, cu_seqlens, positions,
-      B, H, Hkv, D, Dv, Dc, block_size, scale, window, sink, slopes);
+      B, H, Hkv, D, Dv, Dc, block_size, scale, window, chunked, sink, sinks, slopes);
   return cuda_status("attention_generic");
 }
 
@@ -130,8 +131,8 @@ DINFER_DEFINE_LAST_ERROR()
 DINFER_API int dinfer_attention_generic_bias(const void* q, int64_t ldq, void* out, int64_t ldo, const void* cache,
                                              const int* block_table, int max_blocks, const int* cu_seqlens,
                                              const int* positions, int T, int B, int H, int Hkv, int D, int Dv, int Dc,
-                                             int block_size, float scale, int window, int sink, const float* slopes,
-                                             int dtype, cudaStream_t stream);
+                                             int block_size, float scale, int window, int chunked, int sink, const float* sinks,
+                                             const float* slopes, int dtype, cudaStream_t stream);
 
 // q: [T, ...] rows of stride ldq, head h at h*D; out likewise with stride ldo.
 // cache [num_blocks, 2, Hkv, block_size, D]; block_table [B, max_blocks] int32;
@@ -143,7 +144,7 @@ DINFER_API int dinfer_attention_generic(const void* q, int64_t ldq, void* out, i
                                         int block_size, float scale, int window, int dtype,
                                         cudaStream_t stream) {
   return dinfer_attention_generic_bias(q, ldq, out, ldo, cache, block_table, max_blocks, cu_seqlens, positions, T, B, H,
-                                       Hkv, D, D, D, block_size, scale, window, 0, nullptr, dtype, stream);
+                                       Hkv, D, D, D, block_size, scale, window, 0, 0, nullptr, nullptr, dtype, stream);
 }
 
 // The same with values Dv wide in a cache whose rows are Dc wide (out: head h at h*Dv), and an optional sink.
@@ -153,15 +154,16 @@ DINFER_API int dinfer_attention_generic_ex(const void* q, int64_t ldq, void* out
                                            int block_size, float scale, int window, int sink, int dtype,
                                            cudaStream_t stream) {
   return dinfer_attention_generic_bias(q, ldq, out, ldo, cache, block_table, max_blocks, cu_seqlens, positions, T, B, H,
-                                       Hkv, D, Dv, Dc, block_size, scale, window, sink, nullptr, dtype, stream);
+                                       Hkv, D, Dv, Dc, block_size, scale, window, 0, sink, nullptr, nullptr, dtype, stream);
 }
 
-// The same with a distance bias: slopes [H] f32 or null.
+// The same with a distance bias (slopes [H] f32 or null), keys by chunks (chunked, see first_key) and a score per head
+// for the sink's term (sinks [H] f32 or null: 0).
 DINFER_API int dinfer_attention_generic_bias(const void* q, int64_t ldq, void* out, int64_t ldo, const void* cache,
                                              const int* block_table, int max_blocks, const int* cu_seqlens,
                                              const int* positions, int T, int B, int H, int Hkv, int D, int Dv, int Dc,
-                                             int block_size, float scale, int window, int sink, const float* slopes,
-                                             int dtype, cudaStream_t stream) {
+                                             int block_size, float scale, int window, int chunked, int sink, const float* sinks,
+                                             const float* slopes, int dtype, cudaStream_t stream) {
   if (Dv <= 0 || Dc < D || Dc < Dv) return refuse(DINFER_BAD_ARGUMENT, "attention_generic: bad sizes D=%d Dv=%d Dc=%d", D, Dv, Dc);
   if (T < 0 || B <= 0 || H <= 0 || Hkv <= 0 || D <= 0 || block_size <= 0 || max_blocks <= 0)
     return refuse(DINFER_BAD_ARGUMENT, "attention_generic: bad sizes T=%d B=%d H=%d Hkv=%d D=%d block=%d",
@@ -172,7 +174,7 @@ DINFER_API int dinfer_attention_generic_bias(const void* q, int64_t ldq, void* o
   if (T == 0) return 0;
   const int c = ((D > Dv ? D : Dv) + 31) / 32;
 #define GO(C) return launch<T_, C>(q, ldq, out, ldo, cache, block_table, max_blocks, cu_seqlens, positions, \
-                                   T, B, H, Hkv, D, Dv, Dc, block_size, scale, window, sink, slopes, stream)
+                                   T, B, H, Hkv, D, Dv, Dc, block_size, scale, window, chunked, sink, sinks, slopes, stream)
   DINFER_DISPATCH_DTYPE(dtype, T_, {
     if (c <= 1) GO(1);
     else if (c <= 2) GO(2);

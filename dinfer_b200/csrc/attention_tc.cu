@@ -37,8 +37,9 @@ struct Params {
   const __nv_bfloat16* cache;
   const int* block_table; int max_blocks;
   const int* cu_seqlens; const int* seq_lens;
-  int H, Hkv, group, block_size, window;
-  int sink;                    // one more softmax term of score 0 without a value
+  int H, Hkv, group, block_size, window, chunked;
+  int sink;                    // one more softmax term without a value, of score sinks[head] (null: 0)
+  const float* sinks;
   float scale_log2;            // scale * log2(e)
   const float* slopes;         // [H] or null: a distance bias, score - slopes[h] * (i - j)
   int splits;                  // decode shape only
@@ -135,7 +136,7 @@ __global__ void __launch_bounds__(DECODE ? NT_DECODE : NT_PROMPT, 2) attention_t
   const int last_row = min(row0 + (DECODE ? 16 : BM), rows_total) - 1;
   const int first_tok = row0 / p.group, last_tok = last_row / p.group;
   int hi = hist + last_tok + 1;
-  int lo = p.window > 0 ? max(0, hist + first_tok - p.window + 1) : 0;
+  int lo = first_key(hist + first_tok, p.window, p.chunked);
   int tile_begin = lo / BN, tile_end = (hi + BN - 1) / BN;
   if (DECODE) {
     const int n = tile_end - tile_begin;
@@ -179,10 +180,12 @@ __global__ void __launch_bounds__(DECODE ? NT_DECODE : NT_PROMPT, 2) attention_t
 
   const int wrow = DECODE ? 0 : warp * 16;                 // first row of this warp inside the CTA's rows
   int pos_r[2];                                            // position of the query of rows g, g + 8 (-1: no row)
+  int lo_r[2];                                             // the first key each of them sees
 #pragma unroll
   for (int i = 0; i < 2; ++i) {
     const int row = row0 + wrow + g + 8 * i;
     pos_r[i] = row < rows_total ? hist + row / p.group : -1;
+    lo_r[i] = pos_r[i] >= 0 ? first_key(pos_r[i], p.window, p.chunked) : 0;
   }
   float slope_r[2] = {0.f, 0.f};                           // the rows' slopes, in the exp2 domain
   if (p.slopes) {
@@ -243,7 +246,7 @@ __global__ void __launch_bounds__(DECODE ? NT_DECODE : NT_PROMPT, 2) attention_t
         if (need_mask) {
           const int j = jbase + i * 8 + tq * 2 + (e & 1);
           const int pr = pos_r[e >> 1];
-          const bool vis = j <= pr && j >= lo && (p.window <= 0 || j > pr - p.window);
+          const bool vis = j <= pr && j >= lo_r[e >> 1];
           if (!vis) v = -INFINITY;
         }
         s[i][e] = v;
@@ -303,7 +306,8 @@ __global__ void __launch_bounds__(DECODE ? NT_DECODE : NT_PROMPT, 2) attention_t
     for (int r = 0; r < 2; ++r) {
       const int row = row0 + wrow + g + 8 * r;
       if (row >= rows_total) continue;
-      const float l_all = l_run[r] + (p.sink ? exp2f(-m_run[r]) : 0.f);     // the sink: exp(0 - m), in the denominator only
+      const float extra = p.sink ? exp2f(sink_log2(p.sinks, hk * p.group + row % p.group) - m_run[r]) : 0.f;
+      const float l_all = l_run[r] + extra;                                 // the sink, in the denominator only
       const float inv = l_all > 0.f ? 1.f / l_all : 0.f;
       __nv_bfloat16* dst = p.out + (int64_t)(t0 + row / p.group) * p.ldo + (int64_t)(hk * p.group + row % p.group) * D;
 #pragma unroll
@@ -344,7 +348,7 @@ __global__ void __launch_bounds__(DECODE ? NT_DECODE : NT_PROMPT, 2) attention_t
     }
     const int head = hk * p.group + row;
     if (p.splits == 1) {
-      if (p.sink) L += exp2f(-M);
+      if (p.sink) L += exp2f(sink_log2(p.sinks, head) - M);
       p.out[(int64_t)t0 * p.ldo + (int64_t)head * D + d] = __float2bfloat16_rn(L > 0.f ? acc / L : 0.f);
     } else {
       const int64_t slot = ((int64_t)b * p.H + head) * p.splits + blockIdx.x;
@@ -371,7 +375,7 @@ __global__ void __launch_bounds__(D) attention_merge_kernel(const Params p) {
     L += p.part_ml[(base + s) * 2 + 1] * f;
     acc += p.part_o[(base + s) * D + d] * f;
   }
-  if (p.sink) L += exp2f(-M);
+  if (p.sink) L += exp2f(sink_log2(p.sinks, head) - M);
   p.out[(int64_t)t0 * p.ldo + (int64_t)head * D + d] = __float2bfloat16_rn(L > 0.f ? acc / L : 0.f);
 }
 
@@ -429,12 +433,15 @@ DINFER_API int64_t dinfer_attention_tc_scratch_floats(int B, int H, int D, int s
 // block_table [B, max_blocks]; cu_seqlens [B+1]; seq_lens [B] (length after this step).
 // any_decode / any_prefill: whether the batch holds requests with q_len == 1 / q_len > 1.
 // scratch: dinfer_attention_tc_scratch_floats() floats, or null when splits == 1.
-// sink != 0: the softmax has one more term of score 0 that carries no value (p_j = exp(s_j) / (1 + sum exp(s_j))).
+// chunked: window is the size of the chunks (see first_key).
+// sink != 0: the softmax has one more term that carries no value, of score sinks[h] (f32 [H]; null: 0, that is
+// p_j = exp(s_j) / (1 + sum exp(s_j))).
 // slopes: f32 [H] or null; with them score_ij - slopes[h] * (i - j).
 DINFER_API int dinfer_attention_tc_bias(const void* q, int64_t ldq, void* out, int64_t ldo, const void* cache,
                                         const int* block_table, int max_blocks, const int* cu_seqlens,
                                         const int* seq_lens, int B, int H, int Hkv, int D, int block_size,
-                                        float scale, int window, int sink, const float* slopes, int max_q_len,
+                                        float scale, int window, int chunked, int sink, const float* sinks,
+                                        const float* slopes, int max_q_len,
                                         int any_decode, int any_prefill, int splits, float* scratch, cudaStream_t stream) {
   if (B <= 0 || H <= 0 || Hkv <= 0 || H % Hkv || block_size <= 0 || max_blocks <= 0)
     return refuse(DINFER_BAD_ARGUMENT, "attention_tc: bad sizes B=%d H=%d Hkv=%d block=%d", B, H, Hkv, block_size);
@@ -448,7 +455,7 @@ DINFER_API int dinfer_attention_tc_bias(const void* q, int64_t ldq, void* out, i
   p.q = (const __nv_bfloat16*)q; p.ldq = ldq; p.out = (__nv_bfloat16*)out; p.ldo = ldo;
   p.cache = (const __nv_bfloat16*)cache; p.block_table = block_table; p.max_blocks = max_blocks;
   p.cu_seqlens = cu_seqlens; p.seq_lens = seq_lens; p.H = H; p.Hkv = Hkv; p.group = H / Hkv;
-  p.block_size = block_size; p.window = window; p.sink = sink; p.scale_log2 = scale * 1.4426950408889634f;
+  p.block_size = block_size; p.window = window; p.chunked = chunked; p.sink = sink; p.sinks = sinks; p.scale_log2 = scale * 1.4426950408889634f;
   p.slopes = slopes;
   p.splits = splits; p.part_o = scratch;
   p.part_ml = scratch ? scratch + (int64_t)B * H * splits * D : nullptr;
@@ -463,7 +470,7 @@ DINFER_API int dinfer_attention_tc_sink(const void* q, int64_t ldq, void* out, i
                                         float scale, int window, int sink, int max_q_len, int any_decode,
                                         int any_prefill, int splits, float* scratch, cudaStream_t stream) {
   return dinfer_attention_tc_bias(q, ldq, out, ldo, cache, block_table, max_blocks, cu_seqlens, seq_lens, B, H, Hkv, D,
-                                  block_size, scale, window, sink, nullptr, max_q_len, any_decode, any_prefill, splits,
+                                  block_size, scale, window, 0, sink, nullptr, nullptr, max_q_len, any_decode, any_prefill, splits,
                                   scratch, stream);
 }
 

@@ -45,8 +45,9 @@ struct Params {
   __nv_bfloat16* out; int64_t ldo;
   const int* block_table; int max_blocks;
   const int* cu_seqlens; const int* seq_lens;
-  int B, H, Hkv, group, block_size, bs_log2, window;
-  int sink;                    // one more softmax term of score 0 without a value
+  int B, H, Hkv, group, block_size, bs_log2, window, chunked;
+  int sink;                    // one more softmax term without a value, of score sinks[head] (null: 0)
+  const float* sinks;
   int ksplit;                          // CTAs of a cluster that share a row-tile pair's keys (1, 2, 4 or 8)
   float scale_log2;
   const float* slopes;                 // [H] or null: a distance bias, score - slopes[h] * (i - j)
@@ -127,7 +128,7 @@ attention_umma_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_co
   const int last_tok = (min(row0 + 2 * BM, rows_total) - 1) / p.group;
   const int hi = hist + last_tok + 1;
   const int hi_a = hist + last_tok_a + 1;
-  const int lo = p.window > 0 ? max(0, hist + first_tok - p.window + 1) : 0;
+  const int lo = first_key(hist + first_tok, p.window, p.chunked);
   // the key tiles of the pair, dealt out to the cluster's CTAs in runs of `per` (a CTA may get none)
   const int tile_first = lo / BN;
   const int n_all = (hi + BN - 1) / BN - tile_first;   // tiles of B (or of A when B does not exist)
@@ -326,6 +327,9 @@ attention_umma_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_co
     const float sl_raw = (p.slopes && row_ok) ? p.slopes[hk * p.group + row % p.group] * 1.4426950408889634f / p.scale_log2 : 0.f;
     const int n_w = w == 0 ? n_tiles_a : (b_on ? n_tiles : 0);
     const int first_tok_w = (row0 + w * BM) / p.group;
+    // keys below this one are masked for this row; tiles from lo_all on need no mask on that side
+    const int row_lo = row_ok ? first_key(pos, p.window, p.chunked) : 0;
+    const int lo_all = first_key(hist + (w == 0 ? last_tok_a : last_tok), p.window, p.chunked);
     const uint32_t lane_addr = tmem + ((uint32_t)(quarter * 32) << 16);
     const uint32_t s_addr = lane_addr + w * BN, o_addr = lane_addr + O_COL + w * 128 + h * (D / 2);
     const int pair_bar = 1 + w * 4 + quarter;                       // named barrier of the two warps on these 32 rows
@@ -337,7 +341,7 @@ attention_umma_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_co
       if (ok && !__all_sync(0xffffffffu, mbar_wait(smem_u32(&s_full[w]), j & 1))) { s_abort = 1; atomicExch(p.status, 15); ok = false; }
       tc_fence_after();
       const int jbase = (tile_begin + j) * BN;
-      const bool need_mask = (jbase + BN - 1 > hist + first_tok_w) || p.window > 0 || jbase < lo;
+      const bool need_mask = (jbase + BN - 1 > hist + first_tok_w) || jbase < lo_all;
       // this thread's 64 scores; their maximum (raw: the scale is positive), as eight short chains
       float v0[32], v1[32];
       float mx = -INFINITY;
@@ -357,8 +361,8 @@ attention_umma_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_co
 #pragma unroll
           for (int i = 0; i < 32; ++i) {
             const int ja = jbase + h * 64 + i, jc = ja + 32;
-            if (!(ja <= pos && ja >= lo && (p.window <= 0 || ja > pos - p.window))) v0[i] = -INFINITY;
-            if (!(jc <= pos && jc >= lo && (p.window <= 0 || jc > pos - p.window))) v1[i] = -INFINITY;
+            if (!(ja <= pos && ja >= row_lo)) v0[i] = -INFINITY;
+            if (!(jc <= pos && jc >= row_lo)) v1[i] = -INFINITY;
           }
         }
         float mq[8];
@@ -432,11 +436,12 @@ attention_umma_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_co
     s_sum[w][h][r] = l_run;
     asm volatile("bar.sync %0, 64;" ::"r"(pair_bar) : "memory");
     const float l_own = n_w > 0 ? s_sum[w][0][r] + s_sum[w][1][r] : 0.f;
-    __nv_bfloat16* dst = row_ok ? p.out + (int64_t)(t0 + row / p.group) * p.ldo + (int64_t)(hk * p.group + row % p.group) * D + h * (D / 2)
+    const int head = hk * p.group + row % p.group;
+    __nv_bfloat16* dst = row_ok ? p.out + (int64_t)(t0 + row / p.group) * p.ldo + (int64_t)head * D + h * (D / 2)
                                 : nullptr;
     if (ks == 1) {
       if (ok && n_w > 0) {
-        const float l_fin = l_own + (p.sink ? exp2f(-m_run) : 0.f);       // the sink: exp(0 - m), in the denominator only
+        const float l_fin = l_own + (p.sink ? exp2f(sink_log2(p.sinks, head) - m_run) : 0.f);       // the sink, in the denominator only
         const float inv = l_fin > 0.f ? 1.f / l_fin : 0.f;
 #pragma unroll
         for (int c = 0; c < D / 64; ++c) {
@@ -497,7 +502,7 @@ attention_umma_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_co
           const float l_p = x_sum[sl * rows_r + rloc];
           if (l_p > 0.f) l_all += l_p * fast_exp2(x_max[sl * rows_r + rloc] - m_all);
         }
-        if (p.sink) l_all += exp2f(-m_all);
+        if (p.sink) l_all += exp2f(sink_log2(p.sinks, head) - m_all);
         const float inv = l_all > 0.f ? 1.f / l_all : 0.f;
         const float4* recv = reinterpret_cast<const float4*>(smem_dyn + (sK - smem_u32(smem_dyn)));
 #pragma unroll
@@ -622,12 +627,13 @@ DINFER_API int dinfer_attention_umma_supports(int D, int group, int block_size) 
 // key_splits (1, 2, 4 or 8): that many CTAs of a cluster share the keys of a row-tile pair and fold their results
 // through distributed shared memory; for steps with fewer row tiles than the device has SMs.
 // q: [T, ...] rows of stride ldq with head h at h*D (all H heads); cache [num_blocks, 2, Hkv, block, D] bf16.
-// sink != 0: the softmax has one more term of score 0 that carries no value.
+// chunked: window is the size of the chunks (see first_key).
+// sink != 0: the softmax has one more term that carries no value, of score sinks[h] (f32 [H]; null: 0).
 // slopes: f32 [H] or null; with them score_ij - slopes[h] * (i - j).
 DINFER_API int dinfer_attention_umma_bias(const void* q, int64_t ldq, void* out, int64_t ldo, const void* cache,
                                           int64_t num_blocks, const int* block_table, int max_blocks,
                                           const int* cu_seqlens, const int* seq_lens, int T, int B, int H, int Hkv, int D,
-                                          int block_size, float scale, int window, int sink, const float* slopes,
+                                          int block_size, float scale, int window, int chunked, int sink, const float* sinks, const float* slopes,
                                           int max_q_len, int pair_bound, int key_splits, int* status, cudaStream_t stream);
 
 DINFER_API int dinfer_attention_umma_sink(const void* q, int64_t ldq, void* out, int64_t ldo, const void* cache,
@@ -636,14 +642,14 @@ DINFER_API int dinfer_attention_umma_sink(const void* q, int64_t ldq, void* out,
                                           int block_size, float scale, int window, int sink, int max_q_len,
                                           int pair_bound, int key_splits, int* status, cudaStream_t stream) {
   return dinfer_attention_umma_bias(q, ldq, out, ldo, cache, num_blocks, block_table, max_blocks, cu_seqlens, seq_lens, T, B,
-                                    H, Hkv, D, block_size, scale, window, sink, nullptr, max_q_len, pair_bound, key_splits,
+                                    H, Hkv, D, block_size, scale, window, 0, sink, nullptr, nullptr, max_q_len, pair_bound, key_splits,
                                     status, stream);
 }
 
 DINFER_API int dinfer_attention_umma_bias(const void* q, int64_t ldq, void* out, int64_t ldo, const void* cache,
                                           int64_t num_blocks, const int* block_table, int max_blocks,
                                           const int* cu_seqlens, const int* seq_lens, int T, int B, int H, int Hkv, int D,
-                                          int block_size, float scale, int window, int sink, const float* slopes,
+                                          int block_size, float scale, int window, int chunked, int sink, const float* sinks, const float* slopes,
                                           int max_q_len, int pair_bound, int key_splits, int* status, cudaStream_t stream) {
   if (T <= 0 || B <= 0 || H <= 0 || Hkv <= 0 || H % Hkv || max_blocks <= 0 || num_blocks <= 0)
     return refuse(DINFER_BAD_ARGUMENT, "attention_umma: bad sizes T=%d B=%d H=%d Hkv=%d", T, B, H, Hkv);
@@ -690,7 +696,7 @@ DINFER_API int dinfer_attention_umma_bias(const void* q, int64_t ldq, void* out,
   p.cu_seqlens = cu_seqlens; p.seq_lens = seq_lens; p.H = H; p.Hkv = Hkv; p.group = group; p.block_size = block_size;
   p.bs_log2 = 0;
   while ((1 << p.bs_log2) < block_size) ++p.bs_log2;
-  p.window = window; p.sink = sink; p.scale_log2 = scale * 1.4426950408889634f; p.status = status;
+  p.window = window; p.chunked = chunked; p.sink = sink; p.sinks = sinks; p.scale_log2 = scale * 1.4426950408889634f; p.status = status;
   p.slopes = slopes;
   p.ksplit = key_splits; p.B = B;
   // pairs of 128-row tiles in the batch: the caller's bound, or every request taken for the longest

@@ -43,8 +43,9 @@ struct Params {
   __nv_bfloat16* out; int64_t ldo;
   const int* block_table; int max_blocks;
   const int* cu_seqlens; const int* seq_lens;
-  int B, H, Hkv, group, block_size, bs_log2, window;
-  int sink;                    // one more softmax term of score 0 without a value
+  int B, H, Hkv, group, block_size, bs_log2, window, chunked;
+  int sink;                    // one more softmax term without a value, of score sinks[head] (null: 0)
+  const float* sinks;
   float scale_log2;
   const float* slopes;         // [H] or null: a distance bias, score - slopes[h] * (i - j)
   int* status;
@@ -122,7 +123,7 @@ attention_umma64_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_
   const int last_tok = (min(row0 + 2 * BM, rows_total) - 1) / p.group;
   const int hi = hist + last_tok + 1;
   const int hi_a = hist + last_tok_a + 1;
-  const int lo = p.window > 0 ? max(0, hist + first_tok - p.window + 1) : 0;
+  const int lo = first_key(hist + first_tok, p.window, p.chunked);
   const int tile_begin = lo / BN, tile_end = (hi + BN - 1) / BN;
   const int n_tiles = tile_end - tile_begin;           // tiles of B (or of A when B does not exist)
   const int n_tiles_a = (hi_a + BN - 1) / BN - tile_begin;
@@ -300,6 +301,9 @@ attention_umma64_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_
     const float sl_raw = (p.slopes && row_ok) ? p.slopes[hk * p.group + row % p.group] * 1.4426950408889634f / p.scale_log2 : 0.f;
     const int n_w = w == 0 ? n_tiles_a : (b_on ? n_tiles : 0);
     const int first_tok_w = (row0 + w * BM) / p.group;
+    // keys below this one are masked for this row; tiles from lo_all on need no mask on that side
+    const int row_lo = row_ok ? first_key(pos, p.window, p.chunked) : 0;
+    const int lo_all = first_key(hist + (w == 0 ? last_tok_a : last_tok), p.window, p.chunked);
     const uint32_t lane_addr = tmem + ((uint32_t)(quarter * 32) << 16);
     const uint32_t s_addr = lane_addr + 2 * w * BN, o_addr = lane_addr + O_COL + w * 128;
     unsigned char* prow = smem_dyn + (sP - smem_u32(smem_dyn)) + w * P_BYTES + r * 128;
@@ -321,13 +325,13 @@ attention_umma64_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_
           s1[i] = fmaf(sl_raw, d0 + (float)(i + 32), s1[i]);
         }
       }
-      const bool need_mask = (jbase + BN - 1 > hist + first_tok_w) || p.window > 0 || jbase < lo;
+      const bool need_mask = (jbase + BN - 1 > hist + first_tok_w) || jbase < lo_all;
       if (need_mask) {
 #pragma unroll
         for (int i = 0; i < 32; ++i) {
           const int ja = jbase + i, jc = jbase + 32 + i;
-          if (!(ja <= pos && ja >= lo && (p.window <= 0 || ja > pos - p.window))) s0[i] = -INFINITY;
-          if (!(jc <= pos && jc >= lo && (p.window <= 0 || jc > pos - p.window))) s1[i] = -INFINITY;
+          if (!(ja <= pos && ja >= row_lo)) s0[i] = -INFINITY;
+          if (!(jc <= pos && jc >= row_lo)) s1[i] = -INFINITY;
         }
       }
       // maximum of the raw scores (the scale is positive), as eight short chains instead of one long one
@@ -393,9 +397,10 @@ attention_umma64_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_
       tc_fence_after();
     }
     if (ok && n_w > 0) {
-      const float l_fin = l_run + (p.sink ? exp2f(-m_run) : 0.f);          // the sink: exp(0 - m), in the denominator only
+      const int head = hk * p.group + row % p.group;
+      const float l_fin = l_run + (p.sink ? exp2f(sink_log2(p.sinks, head) - m_run) : 0.f);          // the sink, in the denominator only
       const float inv = l_fin > 0.f ? 1.f / l_fin : 0.f;
-      __nv_bfloat16* dst = row_ok ? p.out + (int64_t)(t0 + row / p.group) * p.ldo + (int64_t)(hk * p.group + row % p.group) * D
+      __nv_bfloat16* dst = row_ok ? p.out + (int64_t)(t0 + row / p.group) * p.ldo + (int64_t)head * D
                                   : nullptr;
 #pragma unroll
       for (int c = 0; c < D / 32; ++c) {
@@ -465,12 +470,13 @@ DINFER_API int dinfer_attention_umma64_supports(int D, int group, int block_size
 
 // Prompt portions (q_len > 1) only; requests that bring one token are skipped.
 // q: [T, ...] rows of stride ldq with head h at h*D (all H heads); cache [num_blocks, 2, Hkv, block, D] bf16.
-// sink != 0: the softmax has one more term of score 0 that carries no value.
+// chunked: window is the size of the chunks (see first_key).
+// sink != 0: the softmax has one more term that carries no value, of score sinks[h] (f32 [H]; null: 0).
 // slopes: f32 [H] or null; with them score_ij - slopes[h] * (i - j).
 DINFER_API int dinfer_attention_umma64_bias(const void* q, int64_t ldq, void* out, int64_t ldo, const void* cache,
                                      int64_t num_blocks, const int* block_table, int max_blocks,
                                      const int* cu_seqlens, const int* seq_lens, int T, int B, int H, int Hkv, int D,
-                                     int block_size, float scale, int window, int sink, const float* slopes, int max_q_len,
+                                     int block_size, float scale, int window, int chunked, int sink, const float* sinks, const float* slopes, int max_q_len,
                                      int pair_bound, int* status, cudaStream_t stream);
 
 DINFER_API int dinfer_attention_umma64_sink(const void* q, int64_t ldq, void* out, int64_t ldo, const void* cache,
@@ -479,13 +485,13 @@ DINFER_API int dinfer_attention_umma64_sink(const void* q, int64_t ldq, void* ou
                                      int block_size, float scale, int window, int sink, int max_q_len, int pair_bound,
                                      int* status, cudaStream_t stream) {
   return dinfer_attention_umma64_bias(q, ldq, out, ldo, cache, num_blocks, block_table, max_blocks, cu_seqlens, seq_lens, T, B,
-                                      H, Hkv, D, block_size, scale, window, sink, nullptr, max_q_len, pair_bound, status, stream);
+                                      H, Hkv, D, block_size, scale, window, 0, sink, nullptr, nullptr, max_q_len, pair_bound, status, stream);
 }
 
 DINFER_API int dinfer_attention_umma64_bias(const void* q, int64_t ldq, void* out, int64_t ldo, const void* cache,
                                      int64_t num_blocks, const int* block_table, int max_blocks,
                                      const int* cu_seqlens, const int* seq_lens, int T, int B, int H, int Hkv, int D,
-                                     int block_size, float scale, int window, int sink, const float* slopes, int max_q_len,
+                                     int block_size, float scale, int window, int chunked, int sink, const float* sinks, const float* slopes, int max_q_len,
                                      int pair_bound, int* status, cudaStream_t stream) {
   if (T <= 0 || B <= 0 || H <= 0 || Hkv <= 0 || H % Hkv || max_blocks <= 0 || num_blocks <= 0)
     return refuse(DINFER_BAD_ARGUMENT, "attention_umma64: bad sizes T=%d B=%d H=%d Hkv=%d", T, B, H, Hkv);
@@ -530,7 +536,7 @@ DINFER_API int dinfer_attention_umma64_bias(const void* q, int64_t ldq, void* ou
   p.cu_seqlens = cu_seqlens; p.seq_lens = seq_lens; p.H = H; p.Hkv = Hkv; p.group = group; p.block_size = block_size;
   p.bs_log2 = 0;
   while ((1 << p.bs_log2) < block_size) ++p.bs_log2;
-  p.window = window; p.sink = sink; p.scale_log2 = scale * 1.4426950408889634f; p.status = status; p.B = B;
+  p.window = window; p.chunked = chunked; p.sink = sink; p.sinks = sinks; p.scale_log2 = scale * 1.4426950408889634f; p.status = status; p.B = B;
   p.slopes = slopes;
   // pairs of 128-row tiles in the batch: the caller's bound, or every request taken for the longest
   int64_t pairs = pair_bound > 0 ? pair_bound : (int64_t)B * (((int64_t)max_q_len * group + 2 * BM - 1) / (2 * BM));

@@ -48,6 +48,7 @@ LIBRARIES: Dict[str, tuple] = {
     "attention_diff_tc": ("attention_diff_tc.cu", []),
     "sandwich": ("sandwich.cu", []),
     "linear_state": ("linear_state.cu", []),
+    "token_side": ("token_side.cu", []),
     # host-side bookkeeping (page pools, cache manager, decode plans): plain C++, no CUDA
     "host_core": ("host_core.cpp", []),
 }

@@ -66,6 +66,26 @@ __device__ __forceinline__ float warp_max(float v) {
   return v;
 }
 
+// xIELU: quadratic above zero, exponential below, both with the slope 1/2 at zero; a_pos = softplus(p), a_neg = 1/2 +
+// softplus(q) of the two numbers that the model learns
+__device__ __forceinline__ float xielu(float z, float a_pos, float a_neg) {
+  return 0.5f * z + (z > 0.f ? a_pos * z * z : a_neg * (expm1f(z) - z));
+}
+
+// ---- which keys a query sees
+// The first key that a query at position pos (>= 0) sees: all of its request's (window <= 0), the last `window` ones
+// (itself included), or with `chunked` those of its own chunk (chunks of `window` positions, counted from the
+// sequence's first).  It never falls as pos rises.
+__device__ __forceinline__ int first_key(int pos, int window, int chunked) {
+  if (window <= 0) return 0;
+  return chunked ? pos / window * window : max(0, pos - window + 1);
+}
+// The softmax's extra term of a head (it has no key and no value): its score times log2(e); the score is sinks[head],
+// or 0 where no sinks are given.
+__device__ __forceinline__ float sink_log2(const float* sinks, int head) {
+  return sinks ? sinks[head] * 1.4426950408889634f : 0.f;
+}
+
 // Sum over a block of up to 1024 threads; every thread gets the result.  `scratch` holds 33 floats.
 __device__ __forceinline__ float block_sum(float v, float* scratch) {
   const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5, nwarp = (blockDim.x + 31) >> 5;

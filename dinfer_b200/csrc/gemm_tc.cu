@@ -67,7 +67,9 @@ struct GemmParams {
   const int* tile_expert = nullptr;
   const int* sorted = nullptr;
   const float* row_w = nullptr;
+  // grp_act also works outside the grouped mode: an activation on the product's result (5: xIELU with a_pos, a_neg)
   int pairs = 0, grp_epi = 0, grp_act = 0;
+  float a_pos = 0.f, a_neg = 0.f;
 };
 
 // ---- PTX wrappers
@@ -166,8 +168,9 @@ __device__ __forceinline__ float gelu_tanh_mul(float g, float u) {
   return 0.5f * g * (1.f + tanhf(0.7978845608028654f * (g + 0.044715f * g * g * g))) * u;
 }
 __device__ __forceinline__ float gate_mul(float g, float u, int act) { return act == 2 ? gelu_tanh_mul(g, u) : silu_mul(g, u); }
-__device__ __forceinline__ float grouped_act(float z, int act) {
-  switch (act) {
+__device__ __forceinline__ float grouped_act(float z, const GemmParams& p) {
+  switch (p.grp_act) {
+    case 5: return xielu(z, p.a_pos, p.a_neg);
     case 1: { const float r = fmaxf(z, 0.f); return r * r; }
     case 2: return z / (1.f + expf(-z));
     case 3: return gelu_tanh_mul(z, 1.f);
@@ -355,7 +358,7 @@ gemm_tc_kernel(const __grid_constant__ CUtensorMap map_a, const __grid_constant_
             if (n < p.N) {
 #pragma unroll
               for (int j = 0; j < 16; ++j)
-                if (b0 + c0 + j < p.tokens) out[(int64_t)(b0 + c0 + j) * p.ldc + n] = out_cast<OutT>(__uint_as_float(v[j]));
+                if (b0 + c0 + j < p.tokens) out[(int64_t)(b0 + c0 + j) * p.ldc + n] = out_cast<OutT>(grouped_act(__uint_as_float(v[j]), p));
             }
           } else {
             // recv[split][token column][row of the owner's share]: consecutive lanes, consecutive words
@@ -448,7 +451,7 @@ gemm_tc_kernel(const __grid_constant__ CUtensorMap map_a, const __grid_constant_
           for (int s = 0; s < p.splits; ++s) acc += recv[(s * N_TILE + c) * rows_per + rl];
           if (p.ss_in) acc *= s_rstd[c];
           const int n = a0 + rank * rows_per + rl;
-          if (n < p.N) out[(int64_t)(b0 + c) * p.ldc + n] = out_cast<OutT>(acc);
+          if (n < p.N) out[(int64_t)(b0 + c) * p.ldc + n] = out_cast<OutT>(grouped_act(acc, p));
         }
       }
     }
@@ -634,13 +637,13 @@ gemm_tc_pair_kernel(const __grid_constant__ CUtensorMap map_a, const __grid_cons
           for (int j = 0; j < 16; ++j) { v[0][j] = 0u; v[1][j] = 0u; }
         }
         if (t >= p.tokens || skip_row) continue;
-        if (p.tile_expert) {
+        if (p.tile_expert || p.grp_act) {
 #pragma unroll
           for (int h = 0; h < 2; ++h)
 #pragma unroll
             for (int j = 0; j < 16; ++j) {
               const float x = __uint_as_float(v[h][j]);
-              v[h][j] = __float_as_uint(p.grp_epi == 0 ? grouped_act(x, p.grp_act) : x * row_scale);
+              v[h][j] = __float_as_uint(p.grp_epi == 0 ? grouped_act(x, p) : x * row_scale);
             }
         }
 #pragma unroll
@@ -832,10 +835,13 @@ DINFER_DEFINE_LAST_ERROR()
 //                  ss_out[part * ss_stride + token] = sum of squares of the new residual over the part's rows,
 //                  for part < dinfer_gemm_tc_parts(tokens, N, K, splits);
 //   ss_in != null: out *= rsqrt(sum_{part < ss_parts} ss_in[part * ss_stride + token] * inv_size + eps).
-DINFER_API int dinfer_gemm_tc_fused(const void* x, int64_t ldx, const void* w, int64_t ldw, void* out, int64_t ldc,
-                                    int out_f32, int tokens, int N, int K, int splits, int act, float* resid, int64_t ldr,
-                                    const void* norm_w, int norm_w_f32, float* ss_out, const float* ss_in, int ss_parts,
-                                    int ss_stride, float inv_size, float eps, int* status, cudaStream_t stream) {
+// unary > 0 (no gate, no residual): an activation on the result, the codes of the grouped product's act and 5: xIELU with
+// a_pos, a_neg.
+DINFER_API int dinfer_gemm_tc_all(const void* x, int64_t ldx, const void* w, int64_t ldw, void* out, int64_t ldc,
+                                  int out_f32, int tokens, int N, int K, int splits, int act, int unary, float a_pos,
+                                  float a_neg, float* resid, int64_t ldr, const void* norm_w, int norm_w_f32, float* ss_out,
+                                  const float* ss_in, int ss_parts, int ss_stride, float inv_size, float eps, int* status,
+                                  cudaStream_t stream) {
   if (tokens < 0 || N <= 0 || K <= 0) return refuse(DINFER_BAD_ARGUMENT, "gemm_tc: bad sizes tokens=%d N=%d K=%d", tokens, N, K);
   if (tokens == 0) return 0;
   if ((K % 8) || (ldx % 8) || (ldw % 8) || (reinterpret_cast<uintptr_t>(x) & 15) || (reinterpret_cast<uintptr_t>(w) & 15))
@@ -850,7 +856,10 @@ DINFER_API int dinfer_gemm_tc_fused(const void* x, int64_t ldx, const void* w, i
     return refuse(DINFER_BAD_ARGUMENT, "gemm_tc: the residual epilogue needs the norm's weight and room for the sums, and no gate");
   if (ss_in && (ss_parts <= 0 || ss_stride < tokens))
     return refuse(DINFER_BAD_ARGUMENT, "gemm_tc: the scaled epilogue needs the parts of the sums (parts=%d stride=%d)", ss_parts, ss_stride);
+  if (unary < 0 || unary > 5 || (unary && (act || resid)))
+    return refuse(DINFER_BAD_ARGUMENT, "gemm_tc: activation %d (0 to 5) without a gate and a residual", unary);
   GemmParams p = {};
+  p.grp_act = unary; p.a_pos = a_pos; p.a_neg = a_neg;
   if (act < 0 || act > 2) return refuse(DINFER_BAD_ARGUMENT, "gemm_tc: unknown gate %d (0 none, 1 silu, 2 tanh-gelu)", act);
   p.act = act;
   p.resid = resid; p.ldr = ldr; p.norm_w = norm_w; p.norm_w_f32 = norm_w_f32; p.ss_out = ss_out;
@@ -889,6 +898,14 @@ DINFER_API int dinfer_gemm_tc_fused(const void* x, int64_t ldx, const void* w, i
   if ((rc = make_map(&mb, w, N, K, ldw, NT / 2))) return rc;
   if (act) return out_f32 ? launch_pair<float, true>(ma, mb, p, stream) : launch_pair<__nv_bfloat16, true>(ma, mb, p, stream);
   return out_f32 ? launch_pair<float, false>(ma, mb, p, stream) : launch_pair<__nv_bfloat16, false>(ma, mb, p, stream);
+}
+
+DINFER_API int dinfer_gemm_tc_fused(const void* x, int64_t ldx, const void* w, int64_t ldw, void* out, int64_t ldc,
+                                    int out_f32, int tokens, int N, int K, int splits, int act, float* resid, int64_t ldr,
+                                    const void* norm_w, int norm_w_f32, float* ss_out, const float* ss_in, int ss_parts,
+                                    int ss_stride, float inv_size, float eps, int* status, cudaStream_t stream) {
+  return dinfer_gemm_tc_all(x, ldx, w, ldw, out, ldc, out_f32, tokens, N, K, splits, act, 0, 0.f, 0.f, resid, ldr, norm_w,
+                            norm_w_f32, ss_out, ss_in, ss_parts, ss_stride, inv_size, eps, status, stream);
 }
 
 // Grouped product of a routed feed-forward's prompt-sized steps on the two-SM kernel: x [cap, K] holds the rows expert

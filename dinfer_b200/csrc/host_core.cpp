@@ -145,6 +145,7 @@ struct Held {
 struct Manager {
   std::vector<int> windows;                      // per group: 0 = every key is kept
   std::vector<int> keep_first;                   // per group: with a window, the first so many tokens stay
+  std::vector<char> chunked;                     // per group: the window is a chunk counted from the sequence's first token
   std::vector<int> block_sizes;                  // per group: tokens a page holds (one size for all with the prefix cache on)
   std::vector<Pool> pools;
   bool prefix = false;
@@ -160,6 +161,7 @@ struct Manager {
   }
   int first_needed_block(int g, int num_computed) const {
     if (!windows[g]) return 0;
+    if (chunked[g]) return num_computed / windows[g] * windows[g] / block_sizes[g];
     return std::max(0, num_computed - windows[g] + 1) / block_sizes[g];
   }
   int need(const Held* h, int g, int total) const {
@@ -239,6 +241,7 @@ DH_API void* dh_manager_new(int n_groups, const int* windows, const int* block_s
   auto* m = new Manager();
   m->windows.assign(windows, windows + n_groups);
   m->keep_first.assign(n_groups, 0);
+  m->chunked.assign(n_groups, 0);
   m->block_sizes.assign(block_sizes, block_sizes + n_groups);
   for (int g = 0; g < n_groups; ++g) {
     if (num_blocks[g] <= 0) { delete m; fail("a pool needs at least one block"); return nullptr; }
@@ -380,6 +383,13 @@ DH_API int dh_set_keep_first(void* mp, int g, int n) {
   auto* m = static_cast<Manager*>(mp);
   if (g < 0 || g >= (int)m->keep_first.size() || n < 0) return fail("group %lld / keep_first %lld out of range", (long long)g, n);
   m->keep_first[g] = n;
+  return 0;
+}
+// Group g's window is a chunk of positions (set before any request is admitted).
+DH_API int dh_set_chunked(void* mp, int g, int on) {
+  auto* m = static_cast<Manager*>(mp);
+  if (g < 0 || g >= (int)m->chunked.size()) return fail("group %lld out of range", (long long)g);
+  m->chunked[g] = on != 0;
   return 0;
 }
 DH_API int dh_resolve(void* mp, int64_t r, const int32_t* tokens, int n) {

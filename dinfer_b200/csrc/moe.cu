@@ -4,6 +4,9 @@
 //                  over all experts, or a sigmoid each), the `top` largest scores (ties to the lower index) -> expert
 //                  ids and weights (the scores, or the scores divided by their sum); optionally the gate of a shared
 //                  expert, the sigmoid of the logit in the column behind the experts' 
+//                  moe_route_choice instead chooses by the scores plus a correction per expert, among the experts of the
+//                  best groups of neighbours; experts behind those that have tensors are identity experts (their output
+//                  is their input): they get no row in the layout and moe_combine adds them
 //   moe_align      the (token, choice) pairs counted per expert and laid out expert by expert, each expert's run
 //                  padded to a multiple of the row tile, so that a row tile belongs to one expert
 //   moe_gemm       grouped product over those tiles: rows gathered by pair (first product, an activation in the
@@ -82,6 +85,91 @@ moe_route_kernel(const float* __restrict__ logits, int64_t ldz, int* __restrict_
       z[arg] = -INFINITY;
     }
     chosen_sum += best;
+    __syncwarp();
+  }
+  if (renorm && lane == 0) {
+    const float inv = 1.f / chosen_sum;
+    for (int k = 0; k < top; ++k) weights[(int64_t)t * top + k] *= inv;
+  }
+}
+
+// ---------------------------------------------------------------- router that chooses by corrected scores
+// The scores as above over all E experts; an expert is chosen by score + correction[e], its weight is the score alone
+// (divided by the chosen ones' sum with renorm).  The experts form `groups` equal runs of neighbours; a run's rank is its
+// largest choice score, and only experts of the `keep` best runs can be chosen.  Equal choice scores go to the lower index.
+__device__ __forceinline__ void warp_best(float& best, int& arg) {
+#pragma unroll
+  for (int o = 16; o > 0; o >>= 1) {
+    const float ob = __shfl_xor_sync(0xffffffffu, best, o);
+    const int oa = __shfl_xor_sync(0xffffffffu, arg, o);
+    if (ob > best || (ob == best && oa < arg)) { best = ob; arg = oa; }
+  }
+}
+
+__global__ void __launch_bounds__(RW * 32)
+moe_route_choice_kernel(const float* __restrict__ logits, int64_t ldz, const float* __restrict__ correction,
+                        int* __restrict__ ids, float* __restrict__ weights, int T, int E, int top, int sigmoid_scores,
+                        int renorm, int groups, int keep) {
+  extern __shared__ float sm[];                          // per warp: E scores, E choice scores, `groups` ranks
+  pdl_enter();
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+  const int t = blockIdx.x * RW + warp;
+  if (t >= T) return;
+  float* z = sm + (size_t)warp * (2 * E + groups);
+  float* c = z + E;
+  float* rank = c + E;
+  const float* row = logits + (int64_t)t * ldz;
+  float mx = -INFINITY;
+  for (int e = lane; e < E; e += 32) { z[e] = row[e]; mx = fmaxf(mx, z[e]); }
+  if (sigmoid_scores) {
+    for (int e = lane; e < E; e += 32) z[e] = 1.f / (1.f + expf(-z[e]));
+  } else {
+    mx = warp_max(mx);
+    float sum = 0.f;
+    for (int e = lane; e < E; e += 32) { const float p = expf(z[e] - mx); z[e] = p; sum += p; }
+    sum = warp_sum(sum);
+    for (int e = lane; e < E; e += 32) z[e] = z[e] / sum;
+  }
+  for (int e = lane; e < E; e += 32) c[e] = z[e] + (correction ? correction[e] : 0.f);
+  __syncwarp();
+  if (keep < groups) {
+    const int size = E / groups;
+    for (int g = lane; g < groups; g += 32) {
+      float m = -INFINITY;
+      for (int i = 0; i < size; ++i) m = fmaxf(m, c[g * size + i]);
+      rank[g] = m;
+    }
+    __syncwarp();
+    for (int k = 0; k < keep; ++k) {
+      float best = -INFINITY;
+      int arg = groups;
+      for (int g = lane; g < groups; g += 32)
+        if (rank[g] > best) { best = rank[g]; arg = g; }
+      warp_best(best, arg);
+      if (lane == 0 && arg < groups) rank[arg] = -INFINITY;
+      // the kept runs are marked by their rank, the others lose their choice scores below
+      __syncwarp();
+    }
+    for (int e = lane; e < E; e += 32)
+      if (rank[e / size] != -INFINITY) c[e] = -INFINITY;
+    __syncwarp();
+  }
+  float chosen_sum = 0.f;
+  for (int k = 0; k < top; ++k) {
+    float best = -INFINITY;
+    int arg = E;
+    for (int e = lane; e < E; e += 32) {
+      const float v = c[e];
+      if (v > best) { best = v; arg = e; }               // the lowest index of a lane's equal scores stays
+    }
+    warp_best(best, arg);
+    const float s = arg < E ? z[arg] : 0.f;              // (fewer open experts than choices: refused by the host)
+    if (lane == 0) {
+      ids[(int64_t)t * top + k] = arg;
+      weights[(int64_t)t * top + k] = s;
+      if (arg < E) c[arg] = -INFINITY;
+    }
+    chosen_sum += s;
     __syncwarp();
   }
   if (renorm && lane == 0) {
@@ -336,16 +424,21 @@ moe_gemm_mma_kernel(const __nv_bfloat16* __restrict__ A, int64_t lda, const __nv
 }
 
 // ---------------------------------------------------------------- combine
+// With `x` the choices of identity experts (an id of E or above) have no row in y: they add weights[t, k] * x[t].
 template <typename TA>
 __global__ void __launch_bounds__(256)
 moe_combine_kernel(const TA* __restrict__ y, const TA* __restrict__ shared, const float* __restrict__ gate,
-                   TA* __restrict__ out, int top, int h) {
+                   TA* __restrict__ out, int top, int h, const TA* __restrict__ x, int64_t ldx, const int* __restrict__ ids,
+                   const float* __restrict__ weights, int E) {
   pdl_enter();
   const int t = blockIdx.x;
   const float g = gate ? gate[t] : 1.f;
   for (int i = threadIdx.x; i < h; i += blockDim.x) {
     float a = 0.f;
-    for (int k = 0; k < top; ++k) a += to_f32<TA>(y[((int64_t)t * top + k) * h + i]);
+    for (int k = 0; k < top; ++k) {
+      const int64_t pair = (int64_t)t * top + k;
+      a += (x && ids[pair] >= E) ? weights[pair] * to_f32<TA>(x[t * ldx + i]) : to_f32<TA>(y[pair * h + i]);
+    }
     if (shared) a += g * to_f32<TA>(shared[(int64_t)t * h + i]);
     out[(int64_t)t * h + i] = from_f32<TA>(a);
   }
@@ -354,7 +447,9 @@ moe_combine_kernel(const TA* __restrict__ y, const TA* __restrict__ shared, cons
 // bfloat16 rows of a multiple of 8 elements: 16-byte loads, one thread per 8 columns, the token's rows independent loads
 __global__ void __launch_bounds__(256)
 moe_combine_bf16x8_kernel(const __nv_bfloat16* __restrict__ y, const __nv_bfloat16* __restrict__ shared,
-                          const float* __restrict__ gate, __nv_bfloat16* __restrict__ out, int top, int h) {
+                          const float* __restrict__ gate, __nv_bfloat16* __restrict__ out, int top, int h,
+                          const __nv_bfloat16* __restrict__ x, int64_t ldx, const int* __restrict__ ids,
+                          const float* __restrict__ weights, int E) {
   pdl_enter();
   const int t = blockIdx.x;
   const int i = (blockIdx.y * blockDim.x + threadIdx.x) * 8;
@@ -368,7 +463,11 @@ moe_combine_bf16x8_kernel(const __nv_bfloat16* __restrict__ y, const __nv_bfloat
 #pragma unroll
     for (int j = 0; j < 4; ++j) { const float2 f = __bfloat1622float2(p2[j]); a[2 * j] += w * f.x; a[2 * j + 1] += w * f.y; }
   };
-  for (int k = 0; k < top; ++k) add(y + ((int64_t)t * top + k) * h, 1.f);
+  for (int k = 0; k < top; ++k) {
+    const int64_t pair = (int64_t)t * top + k;
+    if (x && ids[pair] >= E) add(x + t * ldx, weights[pair]);
+    else add(y + pair * h, 1.f);
+  }
   if (shared) add(shared + (int64_t)t * h, gate ? gate[t] : 1.f);
   uint4 o;
   __nv_bfloat162* o2 = reinterpret_cast<__nv_bfloat162*>(&o);
@@ -405,6 +504,26 @@ __global__ void activation_kernel(const TA* __restrict__ x, TA* __restrict__ out
     out[i] = from_f32<TA>(activate(to_f32<TA>(x[i]), act));
 }
 
+template <typename TA>
+__global__ void xielu_kernel(const TA* __restrict__ x, TA* __restrict__ out, int64_t n, float a_pos, float a_neg) {
+  pdl_enter();
+  for (int64_t i = (int64_t)blockIdx.x * blockDim.x + threadIdx.x; i < n; i += (int64_t)gridDim.x * blockDim.x)
+    out[i] = from_f32<TA>(xielu(to_f32<TA>(x[i]), a_pos, a_neg));
+}
+__global__ void xielu_bf16x8_kernel(const uint4* __restrict__ x, uint4* __restrict__ out, int64_t n8, float a_pos, float a_neg) {
+  pdl_enter();
+  for (int64_t i = (int64_t)blockIdx.x * blockDim.x + threadIdx.x; i < n8; i += (int64_t)gridDim.x * blockDim.x) {
+    uint4 v = x[i];
+    __nv_bfloat162* p = reinterpret_cast<__nv_bfloat162*>(&v);
+#pragma unroll
+    for (int j = 0; j < 4; ++j) {
+      const float2 f = __bfloat1622float2(p[j]);
+      p[j] = __floats2bfloat162_rn(xielu(f.x, a_pos, a_neg), xielu(f.y, a_pos, a_neg));
+    }
+    out[i] = v;
+  }
+}
+
 }  // namespace
 
 DINFER_DEFINE_LAST_ERROR()
@@ -420,6 +539,22 @@ DINFER_API int dinfer_moe_route(const float* logits, int64_t ldz, int* ids, floa
   launch_pdl(moe_route_kernel, dim3((T + RW - 1) / RW), dim3(RW * 32), (size_t)RW * E * sizeof(float), stream, logits, ldz,
              ids, weights, gate, T, E, top, sigmoid_scores, renorm);
   return cuda_status("moe_route");
+}
+
+// logits [T, >= E] f32 rows of stride ldz; correction [E] f32 or null; groups divides E, keep <= groups, and the keep
+// best groups hold at least `top` experts; ids, weights [T, top].
+DINFER_API int dinfer_moe_route_choice(const float* logits, int64_t ldz, const float* correction, int* ids, float* weights,
+                                       int T, int E, int top, int sigmoid_scores, int renorm, int groups, int keep,
+                                       cudaStream_t stream) {
+  if (T < 0 || E <= 0 || top <= 0 || groups <= 0 || E % groups || keep <= 0 || keep > groups ||
+      (int64_t)top > (int64_t)keep * (E / groups) || ldz < E)
+    return refuse(DINFER_BAD_ARGUMENT, "moe_route_choice: bad sizes T=%d E=%d top=%d groups=%d keep=%d", T, E, top, groups, keep);
+  const size_t smem = (size_t)RW * (2 * E + groups) * sizeof(float);
+  if (smem > 48 * 1024) return refuse(DINFER_BAD_ARGUMENT, "moe_route_choice: %d experts in %d groups are too many", E, groups);
+  if (T == 0) return 0;
+  launch_pdl(moe_route_choice_kernel, dim3((T + RW - 1) / RW), dim3(RW * 32), smem, stream, logits, ldz, correction, ids, weights,
+             T, E, top, sigmoid_scores, renorm, groups, keep);
+  return cuda_status("moe_route_choice");
 }
 
 // tokens [T] int32 (negative: -(r + 1) names prev[r]); table [vocab, top] int32; ids, weights [T, top].
@@ -479,23 +614,31 @@ DINFER_API int dinfer_moe_gemm(const void* A, int64_t lda, const void* W, void* 
   return 0;
 }
 
-// y [T * top, h] by pair; shared [T, h] or null with gate [T] or null (1); out [T, h].
-DINFER_API int dinfer_moe_combine(const void* y, const void* shared, const float* gate, void* out, int T, int top,
-                                  int h, int act_dtype, cudaStream_t stream) {
+// y [T * top, h] by pair; shared [T, h] or null with gate [T] or null (1); out [T, h].  x (or null): the feed-forward's
+// input [T, h], rows of stride ldx, with ids and weights [T, top]: pairs whose id is E or above are identity experts.
+DINFER_API int dinfer_moe_combine_identity(const void* y, const void* shared, const float* gate, void* out, int T, int top,
+                                           int h, const void* x, int64_t ldx, const int* ids, const float* weights, int E,
+                                           int act_dtype, cudaStream_t stream) {
   if (T < 0 || top <= 0 || h <= 0) return refuse(DINFER_BAD_ARGUMENT, "moe_combine: bad sizes T=%d top=%d h=%d", T, top, h);
+  if (x && (!ids || !weights || ldx < h || E < 0)) return refuse(DINFER_BAD_ARGUMENT, "moe_combine: identity experts need the ids, the weights and rows of at least %d", h);
   if (T == 0) return 0;
   const auto al = [](const void* q) { return (reinterpret_cast<uintptr_t>(q) & 15) == 0; };
-  if (act_dtype == DINFER_BF16 && h % 8 == 0 && al(y) && al(shared) && al(out) && (h / 8 + 255) / 256 <= 65535) {
+  if (act_dtype == DINFER_BF16 && h % 8 == 0 && ldx % 8 == 0 && al(y) && al(shared) && al(out) && al(x) && (h / 8 + 255) / 256 <= 65535) {
     launch_pdl(moe_combine_bf16x8_kernel, dim3(T, (h / 8 + 255) / 256), dim3(256), 0, stream, (const __nv_bfloat16*)y,
-               (const __nv_bfloat16*)shared, gate, (__nv_bfloat16*)out, top, h);
+               (const __nv_bfloat16*)shared, gate, (__nv_bfloat16*)out, top, h, (const __nv_bfloat16*)x, ldx, ids, weights, E);
     return cuda_status("moe_combine");
   }
   DINFER_DISPATCH_DTYPE(act_dtype, TA, {
     launch_pdl(moe_combine_kernel<TA>, dim3(T), dim3(256), 0, stream, (const TA*)y, (const TA*)shared, gate, (TA*)out,
-               top, h);
+               top, h, (const TA*)x, ldx, ids, weights, E);
     return cuda_status("moe_combine");
   });
   return 0;
+}
+
+DINFER_API int dinfer_moe_combine(const void* y, const void* shared, const float* gate, void* out, int T, int top,
+                                  int h, int act_dtype, cudaStream_t stream) {
+  return dinfer_moe_combine_identity(y, shared, gate, out, T, top, h, nullptr, 0, nullptr, nullptr, 0, act_dtype, stream);
 }
 
 // out = act(x), element by element (1 relu^2, 2 silu, 3 tanh-gelu, 4 relu); out may be x.
@@ -506,6 +649,24 @@ DINFER_API int dinfer_activation(const void* x, void* out, int64_t n, int act, i
   DINFER_DISPATCH_DTYPE(act_dtype, TA, {
     launch_pdl(activation_kernel<TA>, dim3(blocks), dim3(256), 0, stream, (const TA*)x, (TA*)out, n, act);
     return cuda_status("activation");
+  });
+  return 0;
+}
+
+// out = xIELU(x) with a_pos, a_neg, element by element; out may be x.
+DINFER_API int dinfer_xielu(const void* x, void* out, int64_t n, float a_pos, float a_neg, int act_dtype, cudaStream_t stream) {
+  if (n < 0) return refuse(DINFER_BAD_ARGUMENT, "xielu: bad size");
+  if (n == 0) return 0;
+  const bool vec = act_dtype == DINFER_BF16 && n % 8 == 0 && !(reinterpret_cast<uintptr_t>(x) & 15) && !(reinterpret_cast<uintptr_t>(out) & 15);
+  const int64_t items = vec ? n / 8 : n;
+  const int blocks = (int)((items + 255) / 256 < 8192 ? (items + 255) / 256 : 8192);
+  if (vec) {
+    launch_pdl(xielu_bf16x8_kernel, dim3(blocks), dim3(256), 0, stream, (const uint4*)x, (uint4*)out, items, a_pos, a_neg);
+    return cuda_status("xielu");
+  }
+  DINFER_DISPATCH_DTYPE(act_dtype, TA, {
+    launch_pdl(xielu_kernel<TA>, dim3(blocks), dim3(256), 0, stream, (const TA*)x, (TA*)out, n, a_pos, a_neg);
+    return cuda_status("xielu");
   });
   return 0;
 }

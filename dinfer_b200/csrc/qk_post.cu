@@ -411,8 +411,22 @@ DINFER_API int dinfer_qk_post(void* qkv, int64_t ld, const int* positions, const
 // Two more steps, each off unless asked for.  A query temperature: q of a token at position p is multiplied by
 // 1 + temp_coef * ln(floor((p + 1) / temp_every) + 1), in 32-bit, last of all.  Mixed values: v <- (1 - lam) v +
 // lam v_first with v_first [T, Hkv * Dv] (row stride ld_first) the values another layer made of the same tokens;
-// the mixed v is what the cache gets (v in the projection's row is left as it was).
+// the mixed v is what the cache gets (v in the projection's row is left as it was).  And turned values: with v_cos_sin
+// (rows of Dv, like cos_sin) the cached v is rotated over its whole width by its position's row, in the layout of pairs
+// of q and k.
 namespace {
+
+// x[a], x[b] <- the pair turned by the angle whose cosine and sine are given
+__device__ __forceinline__ void turn_pairs(float* xs, const float* cs, int half, int interleaved, int lane) {
+  for (int i = lane; i < half; i += 32) {
+    const int a = interleaved ? 2 * i : i, b = interleaved ? 2 * i + 1 : i + half;
+    const float c = cs[i], s = cs[half + i];
+    const float u = xs[a], v = xs[b];
+    xs[a] = u * c - v * s;
+    xs[b] = v * c + u * s;
+  }
+  __syncwarp();
+}
 
 template <typename TA, typename TW>
 __global__ void __launch_bounds__(WARPS * 32)
@@ -421,7 +435,8 @@ qkv_post_general_kernel(TA* __restrict__ qkv, int64_t ld, const int* __restrict_
                         float eps, const float* __restrict__ cos_sin, int rot, int interleaved, TA* __restrict__ cache,
                         const int* __restrict__ slots, int block_size, int H, int Hkv, int D, int Dv, int Dc,
                         const float* __restrict__ bias, float temp_coef, int temp_every,
-                        const TA* __restrict__ v_first, int64_t ld_first, float v_lambda) {
+                        const TA* __restrict__ v_first, int64_t ld_first, float v_lambda,
+                        const float* __restrict__ v_cos_sin) {
   __shared__ float sm[WARPS][MAX_D];
   pdl_enter();
   const int t = blockIdx.x;
@@ -448,18 +463,7 @@ qkv_post_general_kernel(TA* __restrict__ qkv, int64_t ld, const int* __restrict_
       __syncwarp();
     };
     if (norm && norm_first) normalize();
-    if (cos_sin) {
-      const float* cs = cos_sin + (int64_t)positions[t] * rot;
-      const int half = rot >> 1;
-      for (int i = lane; i < half; i += 32) {
-        const int a = interleaved ? 2 * i : i, b = interleaved ? 2 * i + 1 : i + half;
-        const float c = cs[i], s = cs[half + i];
-        const float u = xs[a], v = xs[b];
-        xs[a] = u * c - v * s;
-        xs[b] = v * c + u * s;
-      }
-      __syncwarp();
-    }
+    if (cos_sin) turn_pairs(xs, cos_sin + (int64_t)positions[t] * rot, rot >> 1, interleaved, lane);
     if (norm && !norm_first) normalize();
     if (kind == 0 && temp_coef != 0.f) {
       const float f = 1.f + temp_coef * logf((float)((positions[t] + 1) / temp_every) + 1.f);
@@ -469,7 +473,9 @@ qkv_post_general_kernel(TA* __restrict__ qkv, int64_t ld, const int* __restrict_
   } else if (v_first) {
     const TA* vf = v_first + (int64_t)t * ld_first + (int64_t)(head - H - Hkv) * Dv;
     for (int e = lane; e < Dv; e += 32) xs[e] = (1.f - v_lambda) * xs[e] + v_lambda * to_f32<TA>(vf[e]);
+    __syncwarp();
   }
+  if (kind == 2 && v_cos_sin) turn_pairs(xs, v_cos_sin + (int64_t)positions[t] * Dv, Dv >> 1, interleaved, lane);
   if (kind != 0 && cache) {
     const int slot = slots[t];
     if (slot < 0) return;
@@ -480,12 +486,183 @@ qkv_post_general_kernel(TA* __restrict__ qkv, int64_t ld, const int* __restrict_
   }
 }
 
+// The usual case of it in bfloat16 without shared memory: keys and values D = 8 * LPH wide, weighted head norms ahead
+// of a rotation in halves, nothing else.  LPH lanes own a head, eight neighbouring elements each (one 16-byte load and
+// store); the partner of a rotated element is held by another lane of the head.  A thread keeps its cosines and sines
+// while it walks over the token's heads.
+template <typename TW, int LPH>
+__global__ void __launch_bounds__(256)
+qkv_post_turn_kernel(__nv_bfloat16* __restrict__ qkv, int64_t ld, const int* __restrict__ positions,
+                     const TW* __restrict__ q_weight, const TW* __restrict__ k_weight, float eps,
+                     const float* __restrict__ cos_sin, int rot, const float* __restrict__ v_cos_sin,
+                     __nv_bfloat16* __restrict__ cache, const int* __restrict__ slots, int block_size, int H, int Hkv) {
+  constexpr int D = LPH * 8, GROUPS = 256 / LPH;
+  pdl_launch_dependents();
+  const int t = blockIdx.x;
+  const int lane = threadIdx.x & 31, l = lane % LPH;
+  const int heads = H + 2 * Hkv;
+  const int pos = positions[t];
+  // this lane's place in a rotation over its head's first n elements: 0 none, 1 the first half, 2 the second
+  auto place = [&](int n) { return 8 * l < n / 2 ? 1 : (8 * l < n ? 2 : 0); };
+  const int pl_k = cos_sin ? place(rot) : 0, pl_v = v_cos_sin ? place(D) : 0;
+  float c_k[8], s_k[8];
+#pragma unroll
+  for (int j = 0; j < 8; ++j) { c_k[j] = 1.f; s_k[j] = 0.f; }
+  if (pl_k) {
+    const float* cs = cos_sin + (int64_t)pos * rot + 8 * l - (pl_k == 2 ? rot / 2 : 0);
+    load8<float>(cs, c_k);
+    load8<float>(cs + rot / 2, s_k);
+  }
+  const int slot = (cache && slots) ? slots[t] : -1;
+  pdl_wait();
+  const int step = gridDim.y * GROUPS;
+  const int rounds = (heads + step - 1) / step;
+  for (int r = 0; r < rounds; ++r) {
+    const int head = (r * gridDim.y + blockIdx.y) * GROUPS + threadIdx.x / LPH;
+    const bool live = head < heads;
+    const int kind = head < H ? 0 : (head < H + Hkv ? 1 : 2);
+    __nv_bfloat16* x = qkv + (int64_t)t * ld + (int64_t)head * D + 8 * l;
+    float a[8], c[8], s[8];
+#pragma unroll
+    for (int j = 0; j < 8; ++j) { a[j] = 0.f; c[j] = c_k[j]; s[j] = s_k[j]; }
+    int pl = pl_k, n = rot;
+    if (live) load8<__nv_bfloat16>(x, a);
+    if (kind == 2) {
+      pl = pl_v;
+      n = D;
+      if (pl) {
+        const float* cs = v_cos_sin + (int64_t)pos * D + 8 * l - (pl == 2 ? D / 2 : 0);
+        load8<float>(cs, c);
+        load8<float>(cs + D / 2, s);
+      }
+    }
+    __syncwarp();
+    float ss = 0.f;
+#pragma unroll
+    for (int j = 0; j < 8; ++j) ss += a[j] * a[j];
+#pragma unroll
+    for (int o = LPH / 2; o > 0; o >>= 1) ss += __shfl_xor_sync(0xffffffffu, ss, o);
+    const TW* w = kind == 0 ? q_weight : k_weight;
+    if (live && kind != 2 && w) {
+      const float rinv = rsqrtf(ss / (float)D + eps);
+      float wv[8];
+      load8<TW>(w + 8 * l, wv);
+#pragma unroll
+      for (int j = 0; j < 8; ++j) a[j] = a[j] * rinv * wv[j];
+    }
+    const int other = lane + (pl == 1 ? n / 16 : (pl == 2 ? -(n / 16) : 0));
+    float b[8];
+#pragma unroll
+    for (int j = 0; j < 8; ++j) b[j] = __shfl_sync(0xffffffffu, a[j], other);
+    if (pl) {
+      const float sign = pl == 1 ? -1.f : 1.f;
+#pragma unroll
+      for (int j = 0; j < 8; ++j) a[j] = a[j] * c[j] + sign * b[j] * s[j];
+    }
+    if (!live) continue;
+    if (kind != 2) store8<__nv_bfloat16>(x, a);
+    if (kind != 0 && slot >= 0) {
+      const int hk = kind == 1 ? head - H : head - H - Hkv;
+      const int64_t blk = slot / block_size, off = slot % block_size;
+      store8<__nv_bfloat16>(cache + (((blk * 2 + (kind == 2)) * Hkv + hk) * block_size + off) * D + 8 * l, a);
+    }
+  }
+}
+
+template <typename TW, int LPH>
+void launch_turn(void* qkv, int64_t ld, const int* positions, const void* qw, const void* kw, float eps, const float* cos_sin,
+                 int rot, const float* v_cos_sin, void* cache, const int* slots, int block_size, int T, int H, int Hkv,
+                 cudaStream_t stream) {
+  const int groups = 256 / LPH, all = (H + 2 * Hkv + groups - 1) / groups;
+  // few tokens: a head a thread group; many: a CTA walks over its token's heads
+  launch_pdl(qkv_post_turn_kernel<TW, LPH>, dim3(T, T >= 512 ? 1 : all), dim3(256), 0, stream, (__nv_bfloat16*)qkv, ld, positions,
+             (const TW*)qw, (const TW*)kw, eps, cos_sin, rot, v_cos_sin, (__nv_bfloat16*)cache, slots, block_size, H, Hkv);
+}
+
+// ---- what becomes of the heads' outputs: pair m of head h of a token at position p is turned by minus its angle, then
+// the head is multiplied by sigmoid(gate[t, h]); 32-bit, one rounding, in place.
+template <typename T>
+__global__ void __launch_bounds__(256)
+heads_out_kernel(T* __restrict__ x, int64_t ldx, const int* __restrict__ positions, const float* __restrict__ cos_sin,
+                 const T* __restrict__ gate, int64_t ldg, int H, int Dv, int interleaved) {
+  pdl_enter();
+  const int t = blockIdx.x;
+  const int half = (Dv + 1) / 2;                                  // an odd width has no pairs (and no table)
+  const float* cs = cos_sin ? cos_sin + (int64_t)positions[t] * Dv : nullptr;
+  for (int i = blockIdx.y * blockDim.x + threadIdx.x; i < H * half; i += gridDim.y * blockDim.x) {
+    const int h = i / half, m = i % half;
+    const float g = gate ? 1.f / (1.f + expf(-to_f32<T>(gate[(int64_t)t * ldg + h]))) : 1.f;
+    T* row = x + (int64_t)t * ldx + (int64_t)h * Dv;
+    const int a = interleaved ? 2 * m : m, b = interleaved ? 2 * m + 1 : m + half;
+    const float u = to_f32<T>(row[a]), v = b < Dv ? to_f32<T>(row[b]) : 0.f;
+    const float c = cs ? cs[m] : 1.f, s = cs ? cs[half + m] : 0.f;
+    row[a] = from_f32<T>((u * c + v * s) * g);
+    if (b < Dv) row[b] = from_f32<T>((v * c - u * s) * g);
+  }
+}
+
+// bfloat16, pairs in halves, a width of a multiple of 16: eight pairs a thread, which keeps its cosines and sines while
+// it walks over the token's heads
+__global__ void __launch_bounds__(256)
+heads_out_bf16x8_kernel(__nv_bfloat16* __restrict__ x, int64_t ldx, const int* __restrict__ positions,
+                        const float* __restrict__ cos_sin, const __nv_bfloat16* __restrict__ gate, int64_t ldg, int H, int Dv) {
+  pdl_launch_dependents();
+  const int t = blockIdx.x;
+  const int half = Dv / 2, per = Dv / 16, groups = 256 / per;
+  const int group = threadIdx.x / per, l = threadIdx.x % per;
+  float c[8], s[8];
+#pragma unroll
+  for (int j = 0; j < 8; ++j) { c[j] = 1.f; s[j] = 0.f; }
+  if (cos_sin) {
+    const float* cs = cos_sin + (int64_t)positions[t] * Dv + 8 * l;
+    load8<float>(cs, c);
+    load8<float>(cs + half, s);
+  }
+  pdl_wait();
+  if (group >= groups) return;
+  for (int h = blockIdx.y * groups + group; h < H; h += gridDim.y * groups) {
+    const float g = gate ? 1.f / (1.f + expf(-__bfloat162float(gate[(int64_t)t * ldg + h]))) : 1.f;
+    __nv_bfloat16* row = x + (int64_t)t * ldx + (int64_t)h * Dv + 8 * l;
+    float u[8], v[8], a[8], b[8];
+    load8<__nv_bfloat16>(row, u);
+    load8<__nv_bfloat16>(row + half, v);
+#pragma unroll
+    for (int j = 0; j < 8; ++j) { a[j] = (u[j] * c[j] + v[j] * s[j]) * g; b[j] = (v[j] * c[j] - u[j] * s[j]) * g; }
+    store8<__nv_bfloat16>(row, a);
+    store8<__nv_bfloat16>(row + half, b);
+  }
+}
+
 }  // namespace
 
-DINFER_API int dinfer_qkv_post_mixed(void* qkv, int64_t ld, const int* positions, const void* q_weight,
+// x [T, H * Dv] rows of stride ldx (in place); cos_sin f32 [max_pos, Dv] or null; gate [T, H] of x's type, rows of stride
+// ldg, or null; positions [T] int32.
+DINFER_API int dinfer_heads_out(void* x, int64_t ldx, const int* positions, const float* cos_sin, const void* gate, int64_t ldg,
+                                int T, int H, int Dv, int interleaved, int dtype, cudaStream_t stream) {
+  if (T < 0 || H <= 0 || Dv <= 0 || ldx < (int64_t)H * Dv || (gate && ldg < H) || (cos_sin && (Dv & 1)))
+    return refuse(DINFER_BAD_ARGUMENT, "heads_out: bad sizes T=%d H=%d Dv=%d", T, H, Dv);
+  if (T == 0) return 0;
+  const auto al = [](const void* q, int n) { return (reinterpret_cast<uintptr_t>(q) & (n - 1)) == 0; };
+  if (dtype == DINFER_BF16 && (!interleaved || !cos_sin) && Dv % 16 == 0 && Dv <= 4096 && ldx % 8 == 0 && al(x, 16) && al(cos_sin, 16)) {
+    const int groups = 256 / (Dv / 16), all = (H + groups - 1) / groups;
+    launch_pdl(heads_out_bf16x8_kernel, dim3(T, T >= 512 ? 1 : all), dim3(256), 0, stream, (__nv_bfloat16*)x, ldx, positions,
+               cos_sin, (const __nv_bfloat16*)gate, ldg, H, Dv);
+    return cuda_status("heads_out");
+  }
+  const int64_t pairs = (int64_t)H * ((Dv + 1) / 2);
+  const int by = (int)((pairs + 255) / 256 > 64 ? 64 : (pairs + 255) / 256);
+  DINFER_DISPATCH_DTYPE(dtype, TA, {
+    launch_pdl(heads_out_kernel<TA>, dim3(T, by), dim3(256), 0, stream, (TA*)x, ldx, positions, cos_sin, (const TA*)gate, ldg,
+               H, Dv, interleaved);
+    return cuda_status("heads_out");
+  });
+  return 0;
+}
+
+DINFER_API int dinfer_qkv_post_turned(void* qkv, int64_t ld, const int* positions, const void* q_weight,
                                      const void* k_weight, int norm, int norm_first, float eps, const float* cos_sin,
-                                     int rot, int interleaved, void* cache, const int* slots, int block_size, int T,
-                                     int H, int Hkv, int D, int Dv, int Dc, const float* bias, float temp_coef,
+                                      int rot, const float* v_cos_sin, int interleaved, void* cache, const int* slots,
+                                      int block_size, int T, int H, int Hkv, int D, int Dv, int Dc, const float* bias, float temp_coef,
                                      int temp_every, const void* v_first, int64_t ld_first, float v_lambda,
                                      int act_dtype, int w_dtype, cudaStream_t stream) {
   if (temp_coef != 0.f && temp_every <= 0)
@@ -499,13 +676,26 @@ DINFER_API int dinfer_qkv_post_mixed(void* qkv, int64_t ld, const int* positions
     return refuse(DINFER_BAD_ARGUMENT, "qkv_post_general: rotary dim %d must be even and at most head_dim %d", rot, D);
   if (ld < (int64_t)(H + Hkv) * D + (int64_t)Hkv * Dv) return refuse(DINFER_BAD_ARGUMENT, "qkv_post_general: row stride below the row's width");
   if (cache && block_size <= 0) return refuse(DINFER_BAD_ARGUMENT, "qkv_post_general: block_size %d", block_size);
+  if (v_cos_sin && (Dv & 1)) return refuse(DINFER_BAD_ARGUMENT, "qkv_post_general: turned values need an even width, got %d", Dv);
   if (T == 0) return 0;
+  const auto al16 = [](const void* q) { return (reinterpret_cast<uintptr_t>(q) & 15) == 0; };
+  // (a rotated half of a multiple of eight elements: the lanes of a pair hold whole runs of it)
+  if (act_dtype == DINFER_BF16 && D == Dv && (D == 64 || D == 128 || D == 256) && norm && norm_first && q_weight && k_weight && !interleaved &&
+      !bias && temp_coef == 0.f && !v_first && (!cos_sin || rot % 16 == 0) && ld % 8 == 0 && al16(qkv) && al16(cache) &&
+      al16(cos_sin) && al16(v_cos_sin) && al16(q_weight) && al16(k_weight)) {
+    DINFER_DISPATCH_DTYPE(w_dtype, TW, {
+      auto go = D == 64 ? launch_turn<TW, 8> : (D == 128 ? launch_turn<TW, 16> : launch_turn<TW, 32>);
+      go(qkv, ld, positions, q_weight, k_weight, eps, cos_sin, rot, v_cos_sin, cache, slots, block_size, T, H, Hkv, stream);
+      return cuda_status("qkv_post_turn");
+    });
+  }
   dim3 grid(T, (H + 2 * Hkv + WARPS - 1) / WARPS);
   DINFER_DISPATCH_DTYPE(act_dtype, TA,
     DINFER_DISPATCH_DTYPE(w_dtype, TW, {
       launch_pdl(qkv_post_general_kernel<TA, TW>, grid, dim3(WARPS * 32), 0, stream, (TA*)qkv, ld, positions,
                  (const TW*)q_weight, (const TW*)k_weight, norm, norm_first, eps, cos_sin, rot, interleaved, (TA*)cache,
-                 slots, block_size, H, Hkv, D, Dv, Dc, bias, temp_coef, temp_every, (const TA*)v_first, ld_first, v_lambda);
+                 slots, block_size, H, Hkv, D, Dv, Dc, bias, temp_coef, temp_every, (const TA*)v_first, ld_first, v_lambda,
+                 v_cos_sin);
       return cuda_status("qkv_post_general");
     }));
   return 0;
@@ -516,7 +706,7 @@ DINFER_API int dinfer_qkv_post_general(void* qkv, int64_t ld, const int* positio
                                        int rot, int interleaved, void* cache, const int* slots, int block_size, int T,
                                        int H, int Hkv, int D, int Dv, int Dc, const float* bias, int act_dtype,
                                        int w_dtype, cudaStream_t stream) {
-  return dinfer_qkv_post_mixed(qkv, ld, positions, q_weight, k_weight, norm, norm_first, eps, cos_sin, rot, interleaved,
+  return dinfer_qkv_post_turned(qkv, ld, positions, q_weight, k_weight, norm, norm_first, eps, cos_sin, rot, nullptr, interleaved,
                                cache, slots, block_size, T, H, Hkv, D, Dv, Dc, bias, 0.f, 1, nullptr, 0, 0.f, act_dtype,
                                w_dtype, stream);
 }

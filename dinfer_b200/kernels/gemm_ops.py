@@ -110,15 +110,19 @@ def decode_splits(tokens: int, N: int, K: int) -> int:
 
 # the gates the product's epilogue knows
 GATES = {False: 0, None: 0, True: 1, "silu": 1, "gelu_tanh": 2}
+# the activations it knows without a gate; an xIELU comes as ("xielu", a_pos, a_neg)
+UNARY = {None: 0, "relu2": 1, "silu": 2, "gelu_tanh": 3, "relu": 4, "xielu": 5}
 
 
 def gemm_tc(x: torch.Tensor, w: torch.Tensor, out: torch.Tensor, splits: Optional[int] = None,
             gated=False, residual: Optional[torch.Tensor] = None, norm_weight: Optional[torch.Tensor] = None,
-            sums: Optional[torch.Tensor] = None, row_scale=None) -> torch.Tensor:
+            sums: Optional[torch.Tensor] = None, row_scale=None, activation=None) -> torch.Tensor:
     """out[tokens, N] = x[tokens, K] @ w[N, K]^T.  out: bfloat16 or float32, last axis contiguous.
 
     ``gated`` (any number of rows; True or "silu", or "gelu_tanh"): the rows of w are (gate, up) pairs, out is
     [tokens, N / 2], out[t, j] = g(x w_2j) * (x w_2j+1) with that g.
+    ``activation`` (any number of rows; no gate, no residual): a key of ``UNARY`` or ("xielu", a_pos, a_neg), applied to
+    the result.
     Epilogues of the decode orientation (at most ``DECODE_MAX_TOKENS`` rows):
       ``residual`` [tokens, N] f32 with ``norm_weight`` [N] and ``sums`` [parts, stride >= tokens] f32
         (``parts = residual_parts(...)``): the product is added into the residual, out gets the new
@@ -134,6 +138,9 @@ def gemm_tc(x: torch.Tensor, w: torch.Tensor, out: torch.Tensor, splits: Optiona
         raise KernelError(f"gemm_tc: unknown gate {gated!r}")
     if (residual is not None or row_scale is not None) and tokens > DECODE_MAX_TOKENS:
         raise KernelError("gemm_tc: the norm epilogues take at most 64 rows")
+    unary, a_pos, a_neg = activation if isinstance(activation, (tuple, list)) else (activation, 0.0, 0.0)
+    if unary not in UNARY or (unary == "xielu") != isinstance(activation, (tuple, list)) or (unary and (gated or residual is not None)):
+        raise KernelError(f"gemm_tc: activation {activation!r}: one of {', '.join(str(k) for k in UNARY)}, without a gate or a residual")
     if gated and (N % 2 or residual is not None):
         raise KernelError("gemm_tc: the gated epilogue needs an even number of weight rows and no residual")
     if w.shape[1] != K or out.shape != (tokens, N // 2 if gated else N) or out.stride(1) != 1 \
@@ -166,12 +173,13 @@ def gemm_tc(x: torch.Tensor, w: torch.Tensor, out: torch.Tensor, splits: Optiona
         if residual is not None and s_in.stride(0) != stride:
             raise KernelError("gemm_tc: the sums read and written must have one row stride")
         si_ptr, stride, inv_size = ptr(s_in), s_in.stride(0), 1.0 / float(size)
-    lib, f = _fn("gemm_tc", "dinfer_gemm_tc_fused",
+    lib, f = _fn("gemm_tc", "dinfer_gemm_tc_all",
                  [c_void_p, c_int64, c_void_p, c_int64, c_void_p, c_int64, c_int, c_int, c_int, c_int, c_int, c_int,
+                  c_int, c_float, c_float,
                   c_void_p, c_int64, c_void_p, c_int, c_void_p, c_void_p, c_int, c_int, c_float, c_float,
                   c_void_p, c_void_p])
     check(lib, f(ptr(x), x.stride(0), ptr(w), w.stride(0), ptr(out), out.stride(0), int(out.dtype == torch.float32),
-                 tokens, N, K, int(splits), GATES[gated], r_ptr, ldr, nw_ptr, nw_f32, so_ptr, si_ptr, int(parts),
+                 tokens, N, K, int(splits), GATES[gated], UNARY[unary], float(a_pos), float(a_neg), r_ptr, ldr, nw_ptr, nw_f32, so_ptr, si_ptr, int(parts),
                  int(stride), float(inv_size), float(eps), ptr(st["status"]), stream_handle()), "gemm_tc")
     return out
 

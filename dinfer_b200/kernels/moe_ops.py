@@ -34,6 +34,30 @@ def route(logits: torch.Tensor, num_experts: int, top_k: int, scoring: str = "so
     return ids, weights, gate
 
 
+def route_choice(logits: torch.Tensor, num_experts: int, top_k: int, correction: Optional[torch.Tensor] = None,
+                 scoring: str = "softmax", renormalize: bool = False, groups: int = 1,
+                 keep: int = 1) -> Tuple[torch.Tensor, torch.Tensor]:
+    """(expert ids int32 [T, top_k], weights f32 [T, top_k]) of a router that chooses by ``score + correction[e]`` (f32
+    [num_experts]) and weighs by the score alone: the experts form ``groups`` equal runs of neighbours, a run ranks by
+    its largest choice score, and only the ``keep`` best runs' experts can be chosen."""
+    require_cuda(logits, correction)
+    _rows_contiguous(logits, "moe route_choice")
+    T = logits.shape[0]
+    if scoring not in ("softmax", "sigmoid"):
+        raise KernelError(f"moe route_choice: unknown scoring {scoring!r}")
+    if logits.dtype != torch.float32 or logits.dim() != 2 or logits.shape[1] < num_experts:
+        raise KernelError("moe route_choice: logits f32 [T, >= E]")
+    if correction is not None and (correction.dtype != torch.float32 or correction.numel() != num_experts or not correction.is_contiguous()):
+        raise KernelError("moe route_choice: correction f32 [E]")
+    ids = torch.empty((T, top_k), dtype=torch.int32, device=logits.device)
+    weights = torch.empty((T, top_k), dtype=torch.float32, device=logits.device)
+    lib, f = _fn("moe", "dinfer_moe_route_choice",
+                 [c_void_p, c_int64, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_void_p])
+    check(lib, f(ptr(logits), logits.stride(0), ptr(correction), ptr(ids), ptr(weights), T, num_experts, top_k,
+                 int(scoring == "sigmoid"), int(bool(renormalize)), int(groups), int(keep), stream_handle()), "moe_route_choice")
+    return ids, weights
+
+
 def route_table(tokens: torch.Tensor, table: torch.Tensor, num_experts: int,
                 prev: Optional[torch.Tensor] = None) -> Tuple[torch.Tensor, torch.Tensor]:
     """Routing without a router: ``table`` [vocab, top] int32 names each token id's experts, every choice weighs
@@ -160,8 +184,10 @@ def grouped_gemm(a: torch.Tensor, w: torch.Tensor, out: torch.Tensor, sorted_: t
 
 
 def combine(y: torch.Tensor, out: torch.Tensor, top_k: int, shared: Optional[torch.Tensor] = None,
-            gate: Optional[torch.Tensor] = None) -> torch.Tensor:
-    """out[t] = sum_k y[t * top_k + k] (+ gate[t] * shared[t]), summed in the order of the choices."""
+            gate: Optional[torch.Tensor] = None, identity=None) -> torch.Tensor:
+    """out[t] = sum_k y[t * top_k + k] (+ gate[t] * shared[t]), summed in the order of the choices.  ``identity`` = (x
+    [T, h], ids [T, top_k], weights, E): the choices with an id of E or above have no row in y and add
+    ``weights[t, k] * x[t]``."""
     require_cuda(y, out, shared, gate)
     T, h = out.shape
     if tuple(y.shape) != (T * top_k, h) or not y.is_contiguous() or not out.is_contiguous() or y.dtype != out.dtype:
@@ -170,9 +196,20 @@ def combine(y: torch.Tensor, out: torch.Tensor, top_k: int, shared: Optional[tor
         raise KernelError("moe combine: shared [T, h] contiguous")
     if gate is not None and (gate.dtype != torch.float32 or gate.numel() != T):
         raise KernelError("moe combine: gate f32 [T]")
-    lib, f = _fn("moe", "dinfer_moe_combine", [c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_void_p])
-    check(lib, f(ptr(y), ptr(shared), ptr(gate), ptr(out), T, top_k, h, dtype_code(out.dtype), stream_handle()),
-          "moe_combine")
+    x = ids = weights = None
+    E = 0
+    if identity is not None:
+        x, ids, weights, E = identity
+        require_cuda(x, ids, weights)
+        if tuple(x.shape) != (T, h) or x.stride(1) != 1 or x.dtype != out.dtype or ids.dtype != torch.int32 \
+                or weights.dtype != torch.float32 or ids.numel() != T * top_k or weights.numel() != T * top_k \
+                or not ids.is_contiguous() or not weights.is_contiguous():
+            raise KernelError("moe combine: identity experts take x [T, h] of the outputs' dtype, ids int32 and weights f32 [T, top_k]")
+    lib, f = _fn("moe", "dinfer_moe_combine_identity",
+                 [c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_void_p, c_int64, c_void_p, c_void_p, c_int,
+                  c_int, c_void_p])
+    check(lib, f(ptr(y), ptr(shared), ptr(gate), ptr(out), T, top_k, h, ptr(x), x.stride(0) if x is not None else 0, ptr(ids),
+                 ptr(weights), int(E), dtype_code(out.dtype), stream_handle()), "moe_combine")
     return out
 
 
@@ -183,4 +220,14 @@ def activation(x: torch.Tensor, out: torch.Tensor, kind: str) -> torch.Tensor:
         raise KernelError("activation: contiguous tensors of one shape and dtype")
     lib, f = _fn("moe", "dinfer_activation", [c_void_p, c_void_p, c_int64, c_int, c_int, c_void_p])
     check(lib, f(ptr(x), ptr(out), x.numel(), ACTIVATIONS[kind], dtype_code(x.dtype), stream_handle()), "activation")
+    return out
+
+
+def xielu(x: torch.Tensor, out: torch.Tensor, a_pos: float, a_neg: float) -> torch.Tensor:
+    """``out = z / 2 + (a_pos z^2 if z > 0 else a_neg (exp(z) - 1 - z))`` element by element (``out`` may be ``x``)."""
+    require_cuda(x, out)
+    if not x.is_contiguous() or not out.is_contiguous() or x.shape != out.shape or x.dtype != out.dtype:
+        raise KernelError("xielu: contiguous tensors of one shape and dtype")
+    lib, f = _fn("moe", "dinfer_xielu", [c_void_p, c_void_p, c_int64, c_float, c_float, c_int, c_void_p])
+    check(lib, f(ptr(x), ptr(out), x.numel(), float(a_pos), float(a_neg), dtype_code(x.dtype), stream_handle()), "xielu")
     return out

@@ -262,15 +262,19 @@ def qk_post(qkv: torch.Tensor, positions: torch.Tensor, num_heads: int, num_kv_h
 def attention_generic(q: torch.Tensor, out: torch.Tensor, cache: torch.Tensor, block_table: torch.Tensor,
                       cu_seqlens: torch.Tensor, positions: torch.Tensor, num_heads: int, num_kv_heads: int,
                       head_dim: int, scale: float, window: int = 0, v_dim: Optional[int] = None,
-                      sink: bool = False, slopes: Optional[torch.Tensor] = None) -> torch.Tensor:
+                      sink: bool = False, slopes: Optional[torch.Tensor] = None, chunked: bool = False,
+                      sinks: Optional[torch.Tensor] = None) -> torch.Tensor:
     """Paged causal attention, plain arithmetic, any head size.  ``q`` may be a strided view (for
     instance the q columns of the qkv rows).  ``v_dim``: the values' width where it differs from the keys' (the
     cache's rows are then ``max(head_dim, v_dim)`` wide, ``out`` holds head h at ``h * v_dim``); ``sink``: one more
-    term of score 0 and no value in the softmax's denominator; ``slopes`` (f32 [H]): a distance bias,
-    ``score_ij - slopes[h] * (i - j)``."""
-    require_cuda(q, out, cache, block_table, cu_seqlens, positions, slopes)
-    if slopes is not None and (slopes.dtype != torch.float32 or slopes.numel() != num_heads or not slopes.is_contiguous()):
-        raise KernelError("attention: slopes float32 [H]")
+    term without a value in the softmax's denominator, of score 0 or, where ``sinks`` (f32 [H]) is given, ``sinks[h]``;
+    ``slopes`` (f32 [H]): a distance bias, ``score_ij - slopes[h] * (i - j)``; ``chunked``: a token sees the keys of its
+    own chunk of ``window`` positions, counted from the sequence's first."""
+    require_cuda(q, out, cache, block_table, cu_seqlens, positions, slopes, sinks)
+    for t, n in ((slopes, "slopes"), (sinks, "sinks")):
+        if t is not None and (t.dtype != torch.float32 or t.numel() != num_heads or not t.is_contiguous()):
+            raise KernelError(f"attention: {n} float32 [H]")
+    sink = sink or sinks is not None
     _rows_contiguous(q, "attention q")
     _rows_contiguous(out, "attention out")
     T = q.shape[0]
@@ -289,11 +293,12 @@ def attention_generic(q: torch.Tensor, out: torch.Tensor, cache: torch.Tensor, b
         raise KernelError(f"attention: cache shape {tuple(cache.shape)} is not [blocks, 2, Hkv, block, {row}]")
     lib, f = _fn("attention_generic", "dinfer_attention_generic_bias",
                  [c_void_p, c_int64, c_void_p, c_int64, c_void_p, c_void_p, c_int, c_void_p, c_void_p,
-                  c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_float, c_int, c_int, c_void_p, c_int, c_void_p])
+                  c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_float, c_int, c_int, c_int, c_void_p, c_void_p,
+                  c_int, c_void_p])
     check(lib, f(ptr(q), q.stride(0), ptr(out), out.stride(0), ptr(cache), ptr(block_table),
                  block_table.shape[1], ptr(cu_seqlens), ptr(positions), T, B, num_heads, num_kv_heads,
-                 head_dim, v_dim, row, cache.shape[3], float(scale), int(window), int(bool(sink)), ptr(slopes),
-                 dtype_code(q.dtype), stream_handle()), "attention_generic")
+                 head_dim, v_dim, row, cache.shape[3], float(scale), int(window), int(bool(chunked)), int(bool(sink)),
+                 ptr(sinks), ptr(slopes), dtype_code(q.dtype), stream_handle()), "attention_generic")
     return out
 
 
@@ -302,14 +307,19 @@ def qkv_post_general(qkv: torch.Tensor, positions: torch.Tensor, num_heads: int,
                      norm: bool, norm_first: bool, cos_sin: Optional[torch.Tensor], cache: Optional[torch.Tensor],
                      slots: Optional[torch.Tensor], block_size: int, interleaved: bool = False,
                      bias: Optional[torch.Tensor] = None, q_temperature=None, v_first: Optional[torch.Tensor] = None,
-                     v_lambda: float = 0.0) -> None:
+                     v_lambda: float = 0.0, v_cos_sin: Optional[torch.Tensor] = None) -> None:
     """The general q/k/v post-processing: per-head RMS norm of q and k (``norm``; the weights may be None: a norm
     without a weight) before or behind (``norm_first``) the rotation, q and k written back in place, k and v (v of
     width ``v_dim``) into a paged cache whose rows are ``max(head_dim, v_dim)`` wide.  ``bias``: f32, one per column of
     the q, k, v projections, added first (a projection whose bias has no kernel of its own).  ``q_temperature`` =
     (coef, every): q at position p times ``1 + coef * ln(floor((p + 1) / every) + 1)``.  ``v_first`` [T, Hkv * v_dim]
-    (rows with a stride are fine) and ``v_lambda``: the cache gets ``(1 - v_lambda) v + v_lambda v_first``."""
-    require_cuda(qkv, positions, q_weight, k_weight, cos_sin, cache, slots, bias, v_first)
+    (rows with a stride are fine) and ``v_lambda``: the cache gets ``(1 - v_lambda) v + v_lambda v_first``.
+    ``v_cos_sin`` (f32 [max_pos, v_dim], laid out like ``cos_sin``): the cached v is turned by it over its whole width,
+    in the same layout of pairs."""
+    require_cuda(qkv, positions, q_weight, k_weight, cos_sin, cache, slots, bias, v_first, v_cos_sin)
+    if v_cos_sin is not None and (v_cos_sin.dtype != torch.float32 or v_cos_sin.dim() != 2 or v_dim % 2
+                                  or v_cos_sin.shape[1] != v_dim or not v_cos_sin.is_contiguous()):
+        raise KernelError("qkv_post_general: v_cos_sin contiguous float32 [max_pos, v_dim]")
     coef, every = (float(q_temperature[0]), int(q_temperature[1])) if q_temperature else (0.0, 1)
     if v_first is not None and (v_first.dtype != qkv.dtype or v_first.stride(1) != 1 or v_first.shape[0] != qkv.shape[0]
                                 or v_first.shape[1] != num_kv_heads * v_dim):
@@ -337,15 +347,37 @@ def qkv_post_general(qkv: torch.Tensor, positions: torch.Tensor, num_heads: int,
                 or slots.numel() != T or tuple(cache.shape[1:]) != (2, num_kv_heads, block_size, row):
             raise KernelError(f"qkv_post_general: cache [blocks, 2, {num_kv_heads}, {block_size}, {row}] of the "
                               f"activations' dtype, contiguous; slots int32 [T]")
-    lib, f = _fn("qk_post", "dinfer_qkv_post_mixed",
-                 [c_void_p, c_int64, c_void_p, c_void_p, c_void_p, c_int, c_int, c_float, c_void_p, c_int, c_int,
+    lib, f = _fn("qk_post", "dinfer_qkv_post_turned",
+                 [c_void_p, c_int64, c_void_p, c_void_p, c_void_p, c_int, c_int, c_float, c_void_p, c_int, c_void_p, c_int,
                   c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_void_p, c_float, c_int, c_void_p,
                   c_int64, c_float, c_int, c_int, c_void_p])
     check(lib, f(ptr(qkv), qkv.stride(0), ptr(positions), ptr(q_weight), ptr(k_weight), int(bool(norm)),
-                 int(bool(norm_first)), float(eps), ptr(cos_sin), rot, int(bool(interleaved)), ptr(cache), ptr(slots),
+                 int(bool(norm_first)), float(eps), ptr(cos_sin), rot, ptr(v_cos_sin), int(bool(interleaved)), ptr(cache), ptr(slots),
                  block_size, T, num_heads, num_kv_heads, head_dim, v_dim, row, ptr(bias), coef, every, ptr(v_first),
                  v_first.stride(0) if v_first is not None else 0, float(v_lambda), dtype_code(qkv.dtype), dtype_code(w_dt),
                  stream_handle()), "qkv_post_general")
+
+
+def heads_out(x: torch.Tensor, positions: torch.Tensor, num_heads: int, v_dim: int, cos_sin: Optional[torch.Tensor] = None,
+              gate: Optional[torch.Tensor] = None, interleaved: bool = False) -> torch.Tensor:
+    """The heads' outputs [T, H * v_dim], in place and in 32-bit with one rounding: turned back by their position's row
+    of ``cos_sin`` (f32 [max_pos, v_dim]: pair m by minus its angle), then multiplied by ``sigmoid(gate[t, h])`` (rows of
+    ``gate`` may have a stride)."""
+    require_cuda(x, positions, cos_sin, gate)
+    _rows_contiguous(x, "heads_out")
+    T = x.shape[0]
+    if x.shape[1] != num_heads * v_dim or positions.dtype != torch.int32 or positions.numel() != T:
+        raise KernelError("heads_out: x [T, H * v_dim], positions int32 [T]")
+    if cos_sin is not None and (cos_sin.dtype != torch.float32 or cos_sin.dim() != 2 or cos_sin.shape[1] != v_dim
+                                or v_dim % 2 or not cos_sin.is_contiguous()):
+        raise KernelError("heads_out: cos_sin contiguous float32 [max_pos, v_dim]")
+    if gate is not None and (tuple(gate.shape) != (T, num_heads) or gate.stride(1) != 1 or gate.dtype != x.dtype):
+        raise KernelError("heads_out: gate [T, H] of x's dtype")
+    lib, f = _fn("qk_post", "dinfer_heads_out", [c_void_p, c_int64, c_void_p, c_void_p, c_void_p, c_int64, c_int, c_int, c_int,
+                                                 c_int, c_int, c_void_p])
+    check(lib, f(ptr(x), x.stride(0), ptr(positions), ptr(cos_sin), ptr(gate), gate.stride(0) if gate is not None else 0, T,
+                 num_heads, v_dim, int(bool(interleaved)), dtype_code(x.dtype), stream_handle()), "heads_out")
+    return x
 
 
 def branch_norm(a: torch.Tensor, weight: Optional[torch.Tensor], eps: float, residual: Optional[torch.Tensor] = None,

@@ -164,3 +164,34 @@ def retention(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, decay: torch.Te
                  ptr(cu_seqlens), ptr(slots), ptr(fresh), ptr(out), B, H, dk, dv, float(k_scale),
                  int(single), stream_handle()), "retention")
     return out
+
+
+def branch_join(x: torch.Tensor, a: torch.Tensor, f: Optional[torch.Tensor] = None, cast: Optional[torch.Tensor] = None) -> None:
+    """``x += a (+ f)`` in place (x float32 [T, h], branches of one dtype); ``cast`` (their dtype) gets the sums rounded."""
+    require_cuda(x, a, f, cast)
+    if x.dtype != torch.float32 or not x.is_contiguous():
+        raise KernelError("branch_join: the stream is contiguous float32")
+    for t in (a, f, cast):
+        if t is not None and (t.shape != x.shape or not t.is_contiguous() or t.dtype != a.dtype):
+            raise KernelError("branch_join: branches and the rounded copy are contiguous, of the stream's shape and one dtype")
+    lib, fn = _fn("token_side", "dinfer_branch_join", [c_void_p, c_void_p, c_void_p, c_void_p, c_int64, c_int, c_void_p])
+    check(lib, fn(ptr(x), ptr(a), ptr(f), ptr(cast), x.numel(), dtype_code(a.dtype), stream_handle()), "branch_join")
+
+
+def token_gate(g: torch.Tensor, ids: torch.Tensor, table: torch.Tensor, at: int, prev: Optional[torch.Tensor] = None) -> torch.Tensor:
+    """``gelu_tanh(g[t, j]) * table[ids[t], at + j]`` [T, dim]; an id -(r + 1) stands for ``prev[r]``."""
+    require_cuda(g, ids, table, prev)
+    _rows_contiguous(g, "token_gate")
+    _rows_contiguous(table, "token_gate table")
+    _ints(ids)
+    T, dim = g.shape
+    if ids.numel() != T or table.dim() != 2 or at < 0 or table.shape[1] < at + dim:
+        raise KernelError("token_gate: ids int32 [T], table [vocab, >= at + dim]")
+    out = torch.empty((T, dim), dtype=g.dtype, device=g.device)
+    lib, f = _fn("token_side", "dinfer_token_gate",
+                 [c_void_p, c_int64, c_void_p, c_void_p, c_int, c_void_p, c_int64, c_int, c_int, c_void_p, c_int, c_int, c_int,
+                  c_int, c_void_p])
+    check(lib, f(ptr(g), g.stride(0), ptr(ids), ptr(prev), prev.numel() if prev is not None else 0, ptr(table), table.stride(0),
+                 table.shape[0], int(at), ptr(out), T, dim, dtype_code(g.dtype), dtype_code(table.dtype), stream_handle()),
+          "token_gate")
+    return out

@@ -19,6 +19,7 @@ from ..kernels import attention_ops, ops
 from .base import (MIXERS, POSITION_ENCODINGS, BuildEnv, CacheBinding, KvCacheNeed, Mixer, StepContext,
                    build_part)
 from .linear import Linear
+from .rope import rope_table
 from .spec import PartSpec, TensorDecl
 
 
@@ -37,7 +38,12 @@ class GQAttention(Mixer):
     H)``) or one number per head.  ``value_mix`` = {"weight": tensor name of one number lambda, "key": any name}: the
     first layer of a model with this key keeps its values of the step's tokens, every later one caches
     ``(1 - lambda) v + lambda v_first`` instead of its own v (the first one's tensor is not used).  ``gate_proj``: the
-    heads are multiplied by ``sigmoid(W_g x)`` before the output projection."""
+    heads are multiplied by ``sigmoid(W_g x)`` before the output projection, one gate per element or, with ``gate_per`` =
+    "head", one per head.  ``sink`` may also be a tensor's name: the extra term's score is then learned, one number per head.
+    ``chunked``: ``window`` is the size of chunks of positions, counted from the sequence's first, and a token sees the
+    tokens of its own chunk.  ``value_turn`` (a rotation's base): the value of position j is cached turned by j over its
+    whole width, pair m by ``j * base^(-2m / v_dim)`` in the position encoding's layout of pairs, and every head's output at
+    position i is turned back by i, ahead of the gate."""
 
     def __init__(self, params, env: BuildEnv, prefix=""):
         super().__init__(params, env, prefix)
@@ -57,7 +63,20 @@ class GQAttention(Mixer):
         self.bias_suffix = p.get("bias_suffix")
         self.out_float32 = bool(p.get("out_float32", False))     # the output projection's result stays 32-bit
         self.Dv = int(p.get("v_dim", self.D))
-        self.sink = bool(p.get("sink", False))
+        sink = p.get("sink", False)
+        self.sink_name = prefix + sink if isinstance(sink, str) else None
+        self.sink = bool(sink)
+        self.sinks = None
+        self.chunked = bool(p.get("chunked", False))
+        if self.chunked and not self.window:
+            raise ValueError("attention: chunks need their size (window)")
+        self.gate_per_head = p.get("gate_per", "element") == "head"
+        if p.get("gate_per", "element") not in ("element", "head"):
+            raise ValueError("attention: gate_per is element or head")
+        self.value_turn = float(p["value_turn"]) if p.get("value_turn") else None
+        self.v_table = None                                  # made at the first step
+        if self.value_turn and self.Dv % 2:
+            raise ValueError("attention: turned values need an even width")
         self.norm_after = p.get("qk_norm_order", "before") == "after"
         self.norm_weight = bool(p.get("qk_norm_weight", True))
         if p.get("qk_norm_order", "before") not in ("before", "after") or self.Dv <= 0:
@@ -75,7 +94,7 @@ class GQAttention(Mixer):
         self.gate_name = prefix + p["gate_proj"] if p.get("gate_proj") else None
         # the q/k kernel with lane paths takes the usual order and equal widths; anything else takes the general one
         self.general = (self.Dv != self.D or (self.qk_norm and (self.norm_after or not self.norm_weight))
-                        or self.q_temperature is not None or self.value_mix is not None)
+                        or self.q_temperature is not None or self.value_mix is not None or self.value_turn is not None)
         pos: PartSpec = p.get("position") or PartSpec("none")
         self.position = build_part(POSITION_ENCODINGS, pos, env, prefix)
         n = lambda key, default: prefix + p.get(key, default)
@@ -103,7 +122,9 @@ class GQAttention(Mixer):
         if self.value_mix:
             d.append(TensorDecl(self.names["vmix"], ()))
         if self.gate_name:
-            d.append(TensorDecl(self.gate_name, (H * Dv, h)))
+            d.append(TensorDecl(self.gate_name, (H if self.gate_per_head else H * Dv, h)))
+        if self.sink_name:
+            d.append(TensorDecl(self.sink_name, (H,)))
         return d
 
     def _bias_name(self, which: str) -> str:
@@ -133,6 +154,8 @@ class GQAttention(Mixer):
                 rows.append(q.new_zeros((self.gate_col - used, q.shape[1]), dtype=dt))
             rows.append(tensors[self.gate_name].to(dt))
         self.qkv = Linear(torch.cat(rows, dim=0), None if self.general else qkv_bias)
+        if self.sink_name:
+            self.sinks = tensors[self.sink_name].to(torch.float32).contiguous()
         if self.slope_values is not None:
             self.slopes = torch.tensor(self.slope_values, dtype=torch.float32, device=q.device)
         if self.value_mix:
@@ -143,7 +166,8 @@ class GQAttention(Mixer):
             self.k_norm_w = tensors[self.names["kn"]].to(self.q_norm_w.dtype).contiguous()
 
     def cache_need(self):
-        return KvCacheNeed(self.Hkv, max(self.D, self.Dv), self.window, int(self.page_size) if self.page_size else None)
+        return KvCacheNeed(self.Hkv, max(self.D, self.Dv), self.window, int(self.page_size) if self.page_size else None,
+                           chunked=self.chunked)
 
     def _fast(self, dtype) -> bool:
         """Whether the tensor-core kernels take this attention: keys and values of one width."""
@@ -170,6 +194,10 @@ class GQAttention(Mixer):
         qkv = self.qkv(x)
         kv = cache.kv if cache.write else None
         table = self.position.fused_table()
+        interleaved = getattr(self.position, "interleaved", False)
+        if self.value_turn and self.v_table is None:
+            self.v_table = rope_table(self.Dv, self.value_turn, int(self.env.max_positions), self.env.device)
+        v_table = self.v_table
         if self.general:
             if not self.position.fused:
                 raise NotImplementedError("attention: a head norm behind the rotation, or values of another width, "
@@ -185,11 +213,12 @@ class GQAttention(Mixer):
                     v_first = None
             ops.qkv_post_general(qkv, ctx.positions, H, Hkv, D, self.Dv, self.eps, self.q_norm_w, self.k_norm_w,
                                  self.qk_norm, not self.norm_after, table, kv, g.slot_mapping, g.block_size,
-                                 interleaved=getattr(self.position, "interleaved", False), bias=self.qkv_bias32,
-                                 q_temperature=self.q_temperature, v_first=v_first, v_lambda=self.v_lambda)
+                                 interleaved=interleaved, bias=self.qkv_bias32,
+                                 q_temperature=self.q_temperature, v_first=v_first, v_lambda=self.v_lambda,
+                                 v_cos_sin=v_table)
         elif self.position.fused:
             ops.qk_post(qkv, ctx.positions, H, Hkv, D, self.eps, self.q_norm_w, self.k_norm_w, table,
-                        kv, g.slot_mapping, g.block_size, interleaved=getattr(self.position, "interleaved", False))
+                        kv, g.slot_mapping, g.block_size, interleaved=interleaved)
         else:
             if self.qk_norm:
                 ops.qk_post(qkv, ctx.positions, H, Hkv, D, self.eps, self.q_norm_w, self.k_norm_w, None,
@@ -202,7 +231,10 @@ class GQAttention(Mixer):
                             g.slot_mapping, g.block_size)
         out = torch.empty((qkv.shape[0], H * self.Dv), dtype=qkv.dtype, device=qkv.device)
         self.attend(qkv[:, :H * D], out, cache.kv, g, ctx)
-        if self.gate_name:
+        if v_table is not None or (self.gate_name and self.gate_per_head):
+            gate = qkv[:, self.gate_col:self.gate_col + H] if self.gate_name and self.gate_per_head else None
+            ops.heads_out(out, ctx.positions, H, self.Dv, v_table, gate, interleaved=interleaved)
+        if self.gate_name and not self.gate_per_head:
             ops.sigmoid_gate(out, qkv[:, self.gate_col:self.gate_col + H * self.Dv])
         if sink is not None:                               # (residual, the norm behind this mixer)
             return self.o.into_residual(out, sink[0], sink[1])
@@ -212,15 +244,17 @@ class GQAttention(Mixer):
         """Tensor-core kernels where they take the head size (bfloat16; 32, 64, 128), else the
         plain-arithmetic kernel, which takes every size."""
         window = int(self.window or 0)
+        seen = dict(sink=self.sink, slopes=self.slopes, chunked=self.chunked, sinks=self.sinks)
         if self._fast(q.dtype):
             splits = ctx.decode_splits or attention_ops.decode_splits(ctx.num_reqs, self.Hkv, ctx.max_seq_len)
+            if self.chunked:                                # a decoded token sees its chunk at most: no more splits than that fills
+                splits = min(splits, attention_ops.decode_splits(ctx.num_reqs, self.Hkv, min(window, ctx.max_seq_len)))
             tc_decode = ctx.any_decode
             if ctx.any_decode and attention_ops.decode_supported(q.dtype, self.D, self.H // self.Hkv, g.block_size) \
-                    and (g.block_size >= 8 or not (self.sink or self.slopes is not None)):
+                    and (g.block_size >= 8 or not (self.sink or self.slopes is not None or self.chunked)):
                 # decoded tokens: the kernel made for them (keys on the tile's rows, in-kernel fold)
                 attention_ops.attention_decode(q, out, kv, g.block_table, ctx.cu_seqlens, ctx.seq_lens, self.H,
-                                               self.Hkv, self.D, self.scale, window, splits, sink=self.sink,
-                                               slopes=self.slopes)
+                                               self.Hkv, self.D, self.scale, window, splits, **seen)
                 tc_decode = False
             tc_prefill = ctx.any_prefill
             if ctx.any_prefill and attention_ops.umma_supported(q.dtype, self.D, self.H // self.Hkv, g.block_size):
@@ -238,16 +272,16 @@ class GQAttention(Mixer):
                         and attention_ops.umma64_supported(q.dtype, self.D, self.H // self.Hkv, g.block_size)):
                     attention_ops.attention_umma64(q, out, kv, g.block_table, ctx.cu_seqlens, ctx.seq_lens, self.H,
                                                    self.Hkv, self.D, self.scale, window, ctx.max_q_len, shape[1],
-                                                   sink=self.sink, slopes=self.slopes)
+                                                   **seen)
                 else:
                     attention_ops.attention_umma(q, out, kv, g.block_table, ctx.cu_seqlens, ctx.seq_lens, self.H,
                                                  self.Hkv, self.D, self.scale, window, ctx.max_q_len, shape[0], shape[1],
-                                                 sink=self.sink, slopes=self.slopes)
+                                                 **seen)
                 tc_prefill = False
             if tc_decode or tc_prefill:
                 attention_ops.attention_tc(q, out, kv, g.block_table, ctx.cu_seqlens, ctx.seq_lens, self.H,
                                            self.Hkv, self.D, self.scale, window, ctx.max_q_len, tc_decode,
-                                           tc_prefill, splits, sink=self.sink, slopes=self.slopes)
+                                           tc_prefill, splits, **seen)
         else:
             ops.attention_generic(q, out, kv, g.block_table, ctx.cu_seqlens, ctx.positions, self.H, self.Hkv,
-                                  self.D, self.scale, window, v_dim=self.Dv, sink=self.sink, slopes=self.slopes)
+                                  self.D, self.scale, window, v_dim=self.Dv, **seen)

@@ -28,17 +28,20 @@ class KvCacheNeed:
     """Keys and values of every token (``window`` None) or of the last ``window`` tokens, in pages of
     ``block_size`` tokens (None: the engine's page size).  ``planes``: 2 = keys and values apart
     (``[pages, 2, Hkv, page, D]``); 1 = one row per token that serves as both (a latent cache:
-    ``[pages, 1, Hkv, page, D]``)."""
+    ``[pages, 1, Hkv, page, D]``).  ``chunked``: the window is a chunk of so many positions, counted from the
+    sequence's first: a token sees the tokens of its own chunk, and a chunk's pages go back when the next one begins."""
     num_kv_heads: int
     head_dim: int
     window: Optional[int] = None
     block_size: Optional[int] = None
     planes: int = 2
     keep_first: int = 0        # with a window: the first so many tokens of a request stay (their pages are not given back)
+    chunked: bool = False
 
     def group_key(self):
         # layers whose pages live and die together: same span of tokens, same page size
-        return ("kv", self.window, self.block_size, self.keep_first if self.window is not None else 0)
+        windowed = self.window is not None
+        return ("kv", self.window, self.block_size, self.keep_first if windowed else 0, windowed and self.chunked)
 
 
 @dataclass(frozen=True)

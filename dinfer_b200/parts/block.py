@@ -175,6 +175,17 @@ class PostNormResidual(Block):
             self._join(stream, branch, norm)
 
 
+def _gain_of(norm):
+    """One number, or the norm's weight vector in 32-bit (what ``gain_norm_join`` takes)."""
+    if isinstance(norm, RMSNorm) and norm.gain is not None:
+        return norm.gain
+    if isinstance(norm, RMSNorm) and norm.weight is not None:
+        if norm.weight.dtype != torch.float32:
+            norm.weight = norm.weight.to(torch.float32).contiguous()
+        return norm.weight
+    raise TypeError("the norms are RMS norms with a weight")
+
+
 @BLOCKS.register("sandwich_residual")
 class SandwichResidual(Block):
     """``x += norm1b(mixer(norm1(x))); x += norm2b(ffn(norm2(x)))``: every sublayer has a norm on its input and one on
@@ -217,16 +228,6 @@ class SandwichResidual(Block):
 
     def _no_feed_forward(self) -> bool:
         return bool(getattr(self.feed_forward, "absent", False))
-
-    def _gain(self, norm):
-        """One number, or the norm's weight vector in 32-bit."""
-        if isinstance(norm, RMSNorm) and norm.gain is not None:
-            return norm.gain
-        if isinstance(norm, RMSNorm) and norm.weight is not None:
-            if norm.weight.dtype != torch.float32:
-                norm.weight = norm.weight.to(torch.float32).contiguous()
-            return norm.weight
-        raise TypeError("sandwich_residual: the norms are RMS norms with a weight")
 
     def forward(self, stream: ResidualStream, ctx: StepContext, cache: CacheBinding,
                 next_block: Optional[Block] = None) -> None:
@@ -274,9 +275,9 @@ class SandwichResidual(Block):
         def join(branch, norm, x_from, final: bool):
             follow = nxt if final else self.feed_forward_norm
             out = torch.empty((T, h), dtype=act, device=branch.device) if follow is not None else None
-            stream_ops.gain_norm_join(branch, self._gain(norm), eps, x_from, x_work,
+            stream_ops.gain_norm_join(branch, _gain_of(norm), eps, x_from, x_work,
                                       average=average if final else None,
-                                      next_gain=self._gain(follow) if follow is not None else None, next_out=out)
+                                      next_gain=_gain_of(follow) if follow is not None else None, next_out=out)
             return out
 
         out = join(a, self.mixer_norm_out, x_in, last)
@@ -285,5 +286,59 @@ class SandwichResidual(Block):
             out = join(f, self.feed_forward_norm_out, x_work, True)
         stream.x = average[4] if average is not None else x_work
         stream.cast = None
+        if nxt is not None:
+            stream.normed, stream.normed_by = out, nxt
+
+
+@BLOCKS.register("shared_norm_residual")
+class SharedNormResidual(Block):
+    """``h = norm1(x); x += mixer(h) + ffn(h)``: the sublayers side by side behind one norm (the second norm's place is
+    kind "none"; a layer may have no feed-forward).  extras: ``token_side`` (the params of a ``TokenSide``, or absent): the
+    layer's token input, ``x += norm_s(token_side(x))``, behind the sublayers.
+
+    With a token side two kernels touch the stream: ``branch_join`` adds both branches and leaves the rounded stream that
+    the token side's product reads, ``gain_norm_join`` norms and adds the token side and norms the result for the next
+    block of this kind.  Without one the branches stay pending until the next norm."""
+
+    def configure(self, extras, env, prefix) -> None:
+        from .token_side import TokenSide
+        super().configure(extras, env, prefix)
+        side = self.extras.get("token_side")
+        self.side = TokenSide(side, env, prefix) if side else None
+
+    def parts(self):
+        return super().parts() + ([self.side] if self.side is not None else [])
+
+    def kernel_libraries(self):
+        return ["sandwich", "norm", "token_side"]
+
+    def forward(self, stream: ResidualStream, ctx: StepContext, cache: CacheBinding,
+                next_block: Optional[Block] = None) -> None:
+        from ..kernels import stream_ops
+        from .base import ScaledDeltas
+        if stream.half is not None:
+            raise RuntimeError("a block with one norm does not take half-normed rows")
+        if stream.normed is not None and stream.normed_by is self.mixer_norm:
+            hin = stream.normed
+        else:
+            hin = self.mixer_norm.forward(stream.x, delta=stream.pending)
+            stream.pending = None
+        stream.normed = stream.normed_by = stream.cast = None
+        a = self.mixer.forward(hin, ctx, cache)
+        f = None if getattr(self.feed_forward, "absent", False) else self.feed_forward.forward(hin, ctx)
+        if self.side is None:
+            stream.pending = ScaledDeltas([(a, None)] + ([(f, None)] if f is not None else []))
+            return
+        act = self.env.act_dtype
+        T, h = stream.x.shape
+        cast = torch.empty((T, h), dtype=act, device=a.device) if act != torch.float32 else None
+        stream_ops.branch_join(stream.x, a, f, cast)
+        y = self.side.forward(cast if cast is not None else stream.x, ctx)
+        nxt = None
+        if isinstance(next_block, SharedNormResidual) and next_block.mixer_norm.eps == self.side.norm.eps:
+            nxt = next_block.mixer_norm
+        out = torch.empty((T, h), dtype=act, device=a.device) if nxt is not None else None
+        stream_ops.gain_norm_join(y, _gain_of(self.side.norm), self.side.norm.eps, stream.x, stream.x,
+                                  next_gain=_gain_of(nxt) if nxt is not None else None, next_out=out)
         if nxt is not None:
             stream.normed, stream.normed_by = out, nxt

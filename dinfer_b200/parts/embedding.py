@@ -37,11 +37,13 @@ class TableEmbedding(Embedding):
         return ops.embedding(ids, self.table, x, prev=ctx.prev_tokens, scale=self.scale)
 
 
+@EMBEDDINGS.register("positioned_table")
 @EMBEDDINGS.register("hashed_bigram")
 class HashedBigramEmbedding(Embedding):
     """params: ``tensor``, ``vocab_size``; ``bigram`` (the second table's name; None: none) with ``buckets``,
     ``mul_prev``, ``mul_cur``: row ``(before * mul_prev + token * mul_cur) mod buckets``, and row ``buckets`` (the
-    table's last) for a request's first token; ``positions`` (the name of a learned position table
+    table's last) for a request's first token; without it the embedding is a token's row plus its position's
+    (``positioned_table``) and keeps nothing per request; ``positions`` (the name of a learned position table
     [``max_positions``, h]; None: none)."""
 
     def __init__(self, params, env, prefix=""):

@@ -79,6 +79,20 @@ class Linear:
             return gemm_ops.gemm_tc(x, self.weight, act, gated=True)
         return ops.silu_mul(self(x), act, pairs=True)
 
+    def activated(self, x: torch.Tensor, activation) -> torch.Tensor:
+        """``act(x W^T)`` with an activation of ``gemm_ops.UNARY`` (an xIELU as ("xielu", a_pos, a_neg)): in the product's
+        epilogue where ``fuses_gate`` would fuse a gate, else the product followed by the activation's kernel."""
+        from ..kernels import moe_ops
+        rows = x.shape[0]
+        if (self.bias is None and x.dtype == torch.bfloat16 and self.weight.dtype == torch.bfloat16
+                and (rows <= TC_MAX_DECODE_TOKENS or rows >= TC_MIN_GATED_PROMPT_TOKENS) and gemm_ops.supported(x, self.weight)):
+            out = torch.empty((rows, self.out_features), dtype=x.dtype, device=x.device)
+            return gemm_ops.gemm_tc(x, self.weight, out, activation=activation)
+        y = self(x)
+        if isinstance(activation, (tuple, list)):
+            return moe_ops.xielu(y, y, activation[1], activation[2])
+        return moe_ops.activation(y, y, activation)
+
     def into_residual(self, x: torch.Tensor, residual: torch.Tensor, norm) -> HalfNormed:
         """``residual += x W^T`` and the half-normed rows for the product behind ``norm`` (an RMSNorm over
         ``out_features``), in one kernel.  Only where ``fuses_norm``."""

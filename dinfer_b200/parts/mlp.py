@@ -1,4 +1,4 @@
-"""Dense gated feed-forward: ``down( silu(gate(x)) * up(x) )``.
+"""Dense feed-forwards: the gated one, ``down( silu(gate(x)) * up(x) )``, and one without a gate (``PlainMLP``).
 
 gate and up are stacked once at load into one ``[2I, h]`` matrix whose rows are (gate_j, up_j) pairs, so
 that one product feeds the gate (the reference stacks them as two halves and runs the gate as its own
@@ -7,6 +7,8 @@ product applies the gate in its epilogue; prompts run the product and then the g
 from __future__ import annotations
 
 from typing import Dict, List, Optional
+
+import math
 
 import torch
 
@@ -73,3 +75,44 @@ class SwiGLU(FeedForward):
         if sink is not None:                               # (residual, the norm behind this feed-forward)
             return self.down.into_residual(act, sink[0], sink[1])
         return self.down(act, out_dtype=torch.float32 if self.out_float32 else None)
+
+
+@FEED_FORWARDS.register("plain_mlp")
+class PlainMLP(FeedForward):
+    """``down( act(up(x)) )``, no gate.  params: ``intermediate_size``, ``activation`` (relu, relu2, silu, gelu_tanh, or
+    xielu, whose two learned numbers are the tensor ``act``: with a_pos = softplus(act[0]) and a_neg = 1/2 + softplus(act[1]),
+    ``z / 2 + a_pos z^2`` above zero and ``z / 2 + a_neg (exp(z) - 1 - z)`` below), tensor names ``up_proj``, ``down_proj``,
+    ``act``.  The activation is 32-bit, in the epilogue of the up product where that is this package's own."""
+
+    def __init__(self, params, env, prefix=""):
+        super().__init__(params, env, prefix)
+        self.hidden = env.hidden_size
+        self.inter = int(params["intermediate_size"])
+        self.activation = str(params.get("activation", "relu2"))
+        from ..kernels.gemm_ops import UNARY
+        if self.activation not in UNARY:
+            raise ValueError(f"feed-forward: unknown activation {self.activation!r}")
+        n = lambda key, default: prefix + params.get(key, default)
+        self.names = {"u": n("up_proj", "up_proj.weight"), "d": n("down_proj", "down_proj.weight"), "a": n("act", "act")}
+        self.up: Optional[Linear] = None
+        self.down: Optional[Linear] = None
+
+    def declare(self) -> List[TensorDecl]:
+        d = [TensorDecl(self.names["u"], (self.inter, self.hidden)), TensorDecl(self.names["d"], (self.hidden, self.inter))]
+        if self.activation == "xielu":
+            d.append(TensorDecl(self.names["a"], (2,)))
+        return d
+
+    def bind(self, tensors: Dict[str, torch.Tensor]) -> None:
+        self.up, self.down = Linear(tensors[self.names["u"]]), Linear(tensors[self.names["d"]])
+        self.act = self.activation
+        if self.activation == "xielu":
+            p, q = (float(v) for v in tensors[self.names["a"]].double().cpu())
+            softplus = lambda v: max(v, 0.0) + math.log1p(math.exp(-abs(v)))
+            self.act = ("xielu", softplus(p), 0.5 + softplus(q))
+
+    def kernel_libraries(self):
+        return ["moe"] + self.up.kernel_libraries() + self.down.kernel_libraries()
+
+    def forward(self, x, ctx=None, sink=None):
+        return self.down(self.up.activated(x, self.act))

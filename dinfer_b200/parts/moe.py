@@ -38,7 +38,11 @@ class MoE(FeedForward):
     ``shared_gate_proj``.  ``routing`` ("router", the default, or "table": tensor name ``table``), ``gated`` (experts
     and the shared expert have a gate matrix: names ``expert_gate``, ``shared_gate_up``).  ``weight_on`` ("output", the
     default: ``sum_k w_k expert_k(x)``; "input": ``sum_k expert_k(w_k x)``, gated experts only: the weight is applied
-    to the first product's result, in 32-bit, ahead of the activation)."""
+    to the first product's result, in 32-bit, ahead of the activation).  ``identity`` (so many experts behind the
+    ``num_experts`` that have tensors: the router scores and chooses them too, their output is their input, times the
+    weight), ``correction`` (tensor name of one number per expert, identity experts included, added to the scores for the
+    choice only), ``groups`` = (count, keep): the experts in ``count`` equal runs of neighbours, of which only the ``keep``
+    with the largest choice scores in them take part."""
 
     def __init__(self, params, env, prefix=""):
         super().__init__(params, env, prefix)
@@ -58,10 +62,23 @@ class MoE(FeedForward):
         if p.get("weight_on", "output") not in ("output", "input") or (self.weight_on_input and not self.gated):
             raise ValueError("moe: weight_on is output or input, and input needs gated experts")
         self._ones = {}
+        self.identity = int(p.get("identity", 0) or 0)
+        self.E_all = self.E + self.identity                 # what the router scores
+        self.correction_name = prefix + p["correction"] if p.get("correction") else None
+        self.groups = tuple(int(v) for v in p["groups"]) if p.get("groups") else (1, 1)
+        self.by_choice = bool(self.identity or self.correction_name or p.get("groups"))
+        self.correction = None
+        if self.by_choice:
+            count, keep = self.groups
+            if self.routing != "router" or self.shared_gate or self.weight_on_input:
+                raise ValueError("moe: identity experts, a correction and groups need a router, the weight on the output and "
+                                 "no gate on the shared expert")
+            if count <= 0 or self.E_all % count or not (0 < keep <= count) or self.top > keep * (self.E_all // count):
+                raise ValueError(f"moe: groups {self.groups} do not divide {self.E_all} experts, or keep fewer than top_k {self.top}")
         if self.routing not in ("router", "table") or (self.routing == "table" and (self.vocab <= 0 or self.shared_gate)):
             raise ValueError("moe: routing is router or table; a table needs vocab_size and takes no gate on the shared expert")
-        if not (0 < self.top <= self.E):
-            raise ValueError(f"moe: top_k {self.top} must be between 1 and num_experts {self.E}")
+        if not (0 < self.top <= self.E_all):
+            raise ValueError(f"moe: top_k {self.top} must be between 1 and the {self.E_all} experts")
         if self.activation not in moe_ops.ACTIVATIONS or self.activation == "none":
             raise ValueError(f"moe: unknown activation {self.activation!r}")
         if self.scoring not in ("softmax", "sigmoid") or self.shared_gate not in (None, "sigmoid"):
@@ -82,7 +99,9 @@ class MoE(FeedForward):
         if self.routing == "table":
             d = [TensorDecl(self.names["table"], (self.vocab, self.top), kind="int", init="choices", init_arg=self.E)]
         else:
-            d = [TensorDecl(self.names["router"], (self.E, h))]
+            d = [TensorDecl(self.names["router"], (self.E_all, h))]
+            if self.correction_name:
+                d.append(TensorDecl(self.correction_name, (self.E_all,)))
         for e in range(self.E):
             if self.gated:
                 d.append(TensorDecl(self.names["gate"].format(e=e), (self.ff, h)))
@@ -108,6 +127,8 @@ class MoE(FeedForward):
             if pad:
                 router_w = torch.cat([router_w, router_w.new_zeros((pad, router_w.shape[1]))])
             self.router = Linear(router_w)
+            if self.correction_name:
+                self.correction = tensors[self.correction_name].to(torch.float32).contiguous()
         ups = [tensors[self.names["up"].format(e=e)] for e in range(self.E)]
         downs = [tensors[self.names["down"].format(e=e)] for e in range(self.E)]
         gates = [tensors[self.names["gate"].format(e=e)] for e in range(self.E)] if self.gated else []
@@ -145,8 +166,15 @@ class MoE(FeedForward):
         else:
             # 32-bit logits: products of the stored values summed in 32-bit (the same product that makes the model's logits)
             z = self.router(x, out_dtype=torch.float32)
-            ids, weights, gate = moe_ops.route(z, self.E, self.top, self.scoring, self.renormalize,
-                                               bool(self.shared_ff and self.shared_gate))
+            if self.by_choice:
+                gate = None
+                ids, weights = moe_ops.route_choice(z, self.E_all, self.top, self.correction, self.scoring, self.renormalize,
+                                                    *self.groups)
+            else:
+                ids, weights, gate = moe_ops.route(z, self.E, self.top, self.scoring, self.renormalize,
+                                                   bool(self.shared_ff and self.shared_gate))
+        # identity experts: their pairs get no row below, the last kernel adds them from the input
+        identity = (x, ids, weights, self.E) if self.identity else None
         pairs = T * self.top
         wide = self.w_up.shape[1]                            # ff, or 2 ff with a gate
         first_act = "none" if self.gated else self.activation
@@ -159,7 +187,7 @@ class MoE(FeedForward):
             u, weights = self._gate(u, order, weights)
             y = torch.empty((pairs, self.hidden), dtype=x.dtype, device=x.device)
             moe_ops.grouped_gemm_tc(u, self.w_down, y, order, tile_expert, pairs, 1, weights=weights)
-            return self._combine(x, y, gate)
+            return self._combine(x, y, gate, identity)
         tile = moe_ops.row_tile(pairs, self.E)
         order, tile_expert = moe_ops.align(ids, self.E, tile)
         u = torch.empty((order.numel(), wide), dtype=x.dtype, device=x.device)
@@ -167,7 +195,7 @@ class MoE(FeedForward):
         u, weights = self._gate(u, order, weights)
         y = torch.empty((pairs, self.hidden), dtype=x.dtype, device=x.device)
         moe_ops.grouped_gemm(u, self.w_down, y, order, tile_expert, pairs, self.top, tile, 1, weights=weights)
-        return self._combine(x, y, gate)
+        return self._combine(x, y, gate, identity)
 
     def _gate(self, u, order, weights):
         """With a gate: the (gate, up) column pairs of the first product become act(gate) * up.  Where the routing weight
@@ -187,7 +215,7 @@ class MoE(FeedForward):
             ones = self._ones[flat.numel()] = torch.ones_like(flat)
         return ops.gated_act_scaled(u, out, flat, order, self.activation, pairs=True), ones
 
-    def _combine(self, x, y, gate):
+    def _combine(self, x, y, gate, identity=None):
         shared = None
         if self.shared_ff and self.gated:
             shared = self.shared_down(self.shared_up.gated_pairs(x, self.activation))
@@ -196,4 +224,4 @@ class MoE(FeedForward):
             moe_ops.activation(s, s, self.activation)
             shared = self.shared_down(s)
         out = torch.empty((x.shape[0], self.hidden), dtype=x.dtype, device=x.device)
-        return moe_ops.combine(y, out, self.top, shared, gate)
+        return moe_ops.combine(y, out, self.top, shared, gate, identity)

@@ -10,6 +10,14 @@ from .base import NORMS, Norm
 from .spec import TensorDecl
 
 
+@NORMS.register("none")
+class NoNorm(Norm):
+    """The place of a norm that an arrangement does not have (a layer whose sublayers share one)."""
+
+    def forward(self, residual, delta=None, rows=None):
+        raise RuntimeError("this layer has no such norm")
+
+
 @NORMS.register("rmsnorm")
 class RMSNorm(Norm):
     """params: ``size``, ``eps``, ``weight`` (tensor name after the prefix), ``optional`` (the weight may be absent
