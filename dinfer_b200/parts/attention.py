@@ -153,6 +153,9 @@ class GQAttention(Mixer):
             if self.gate_col > used:
                 rows.append(q.new_zeros((self.gate_col - used, q.shape[1]), dtype=dt))
             rows.append(tensors[self.gate_name].to(dt))
+            pad = -sum(t.shape[0] for t in rows) % 8         # rows of whole 16-byte pieces, for TMA and vector loads
+            if pad:
+                rows.append(q.new_zeros((pad, q.shape[1]), dtype=dt))
         self.qkv = Linear(torch.cat(rows, dim=0), None if self.general else qkv_bias)
         if self.sink_name:
             self.sinks = tensors[self.sink_name].to(torch.float32).contiguous()

@@ -84,7 +84,7 @@ class Bench:
         assert names == set(W), (sorted(names), sorted(W))
         self.part.bind({k: dev(v, self.dt) for k, v in W.items()})
         kv, st = split_needs(self.part.cache_need())
-        group = GroupSpec(window=kv.window, keep_first=kv.keep_first) if kv is not None else GroupSpec()
+        group = GroupSpec(window=kv.window, keep_first=kv.keep_first, chunked=kv.chunked) if kv is not None else GroupSpec()
         self.m = CacheManager([group], block_size, num_blocks, slots)
         self.binding = CacheBinding(group=0)
         if kv is not None:
