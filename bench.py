@@ -429,7 +429,33 @@ POROVIK_SIZES = {
     "medium": (_porovik_cfg(2048, 16, 4, 128, 64, 6, 1408, 7680), ZASIPEL_SIZES["medium"][0]),
     "large": (_porovik_cfg(4096, 32, 8, 128, 64, 6, 2048, 12288), ZASIPEL_SIZES["large"][0]),
 }
-DESIGNS = {"dobedra": DESIGN_SIZES, "zasipel": ZASIPEL_SIZES, "sobivik": SOBIVIK_SIZES, "porovik": POROVIK_SIZES}
+
+
+# ---------------------------------------------------------------- Datozen beside Qwen3 at equal layer sizes
+def _datozen_cfg(width, heads, kv_heads, dim, experts, identity, groups, keep, top, ff_expert, shared, ff_dense, side, vocab=32768):
+    def att(chunk):
+        return {"type": "attention",
+                "mixer": {"heads": heads, "kv_heads": kv_heads, "dim": dim, "vdim": dim, "scale": dim ** -0.5, "mask": {"size": chunk},
+                          "rot": {"base": 1e6, "dims": dim // 2,
+                                  "scaling": {"factor": 4.0, "original": 4096, "fast": 32.0, "slow": 1.0}}}}
+    dense = {"kind": "dense", "ff": ff_dense}
+    moe = {"kind": "moe", "expert": {"ff": ff_expert}, "shared": {"ff": shared},
+           "router": {"experts": experts, "identity": identity, "top": top, "groups": {"count": groups, "keep": keep}}}
+    return {"architecture": "Datozen", "vocab": vocab, "width": width, "norm": {"eps": 1e-6}, "max_positions": 8192,
+            "token_side": {"dim": side},
+            "layers": [dict(att(1024), mlp=dense), dict(att(8192), mlp=moe), dict(att(1024), mlp=dense), dict(att(8192), mlp=moe)]}
+
+
+# four layers (chunks of 1024 and 8192 positions in turn; a dense feed-forward behind the first and third, 16 or 64 experts
+# and a quarter as many identity experts, of which a token uses 2 or 6, with a shared expert behind the others), heads of 64
+# or 128, a token input of 64 to 256; no loop, so that four layers run; beside each the dense Qwen3 layers of the same width
+# and heads, whose feed-forward has as many weights as the dense one here
+DATOZEN_SIZES = {
+    "small": (_datozen_cfg(1024, 16, 4, 64, 16, 4, 4, 2, 2, 512, 1024, 3072, 64), _qwen3_cfg(1024, 16, 4, 64, 2048)),
+    "medium": (_datozen_cfg(2048, 16, 4, 128, 64, 16, 8, 4, 6, 1408, 2816, 11520, 128), _qwen3_cfg(2048, 16, 4, 128, 7680)),
+    "large": (_datozen_cfg(4096, 32, 8, 128, 64, 16, 8, 4, 6, 2048, 4096, 18432, 256), _qwen3_cfg(4096, 32, 8, 128, 12288)),
+}
+DESIGNS = {"datozen": DATOZEN_SIZES, "dobedra": DESIGN_SIZES, "zasipel": ZASIPEL_SIZES, "sobivik": SOBIVIK_SIZES, "porovik": POROVIK_SIZES}
 # the model a design stands beside (the closest one this package has)
 BESIDE = {"porovik": "zasipel"}
 
@@ -493,7 +519,7 @@ def _time_model(cfg, batch, context, prefill_tokens, steps, seed=5, profile=None
 
 
 def design_run(a) -> int:
-    """``--design dobedra|zasipel|sobivik|porovik``: prefill and decode throughput of four layers of the design beside four
+    """``--design dobedra|zasipel|sobivik|porovik|datozen``: prefill and decode throughput of four layers of the design beside four
     layers of the model it is compared with (Qwen3, or ``BESIDE``) at the same width and head count, at the sizes of
     ``DESIGNS``; one JSON line."""
     rows = {}
@@ -538,11 +564,11 @@ def main() -> int:
     ap.add_argument("--closed-loop", default=None, metavar="C,P,O",
                     help="the reference's serving measurement at engine level instead: C clients, each sending its "
                          "next request when the last has ended, prompts of P tokens, O generated tokens (--shape applies)")
-    ap.add_argument("--design", choices=["dobedra", "zasipel", "sobivik", "porovik"], default=None,
+    ap.add_argument("--design", choices=["dobedra", "zasipel", "sobivik", "porovik", "datozen"], default=None,
                     help="instead of the benchmark: four layers of this design beside four Qwen3 layers of equal width, "
                          "prefill and decode, at a few layer sizes")
     ap.add_argument("--design-size", choices=["small", "medium", "large"], default=None, help="only this size")
-    ap.add_argument("--design-model", choices=["dobedra", "zasipel", "sobivik", "porovik", "qwen3"], default=None, help="with --profile: which of the two")
+    ap.add_argument("--design-model", choices=["dobedra", "zasipel", "sobivik", "porovik", "datozen", "qwen3"], default=None, help="with --profile: which of the two")
     a = ap.parse_args()
     if a.impl == "reference":
         print(json.dumps({"impl": "reference", "unavailable":
