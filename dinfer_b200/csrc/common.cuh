@@ -72,6 +72,15 @@ __device__ __forceinline__ float xielu(float z, float a_pos, float a_neg) {
   return 0.5f * z + (z > 0.f ? a_pos * z * z : a_neg * (expm1f(z) - z));
 }
 
+// The same for results that are rounded to bfloat16, without a branch: e^t - 1 - t by its Taylor polynomial near zero
+// (where the difference would cancel), else through the fast exponential.
+__device__ __forceinline__ float xielu_fast(float z, float a_pos, float a_neg) {
+  const float p = fmaxf(z, 0.f), t = fminf(z, 0.f);
+  const float near = t * t * (0.5f + t * (1.f / 6.f + t * (1.f / 24.f + t * (1.f / 120.f + t * (1.f / 720.f)))));
+  const float e = t > -0.3f ? near : __expf(t) - 1.f - t;
+  return fmaf(0.5f, z, fmaf(a_pos * p, p, a_neg * e));
+}
+
 // ---- which keys a query sees
 // The first key that a query at position pos (>= 0) sees: all of its request's (window <= 0), the last `window` ones
 // (itself included), or with `chunked` those of its own chunk (chunks of `window` positions, counted from the

@@ -170,7 +170,7 @@ __device__ __forceinline__ float gelu_tanh_mul(float g, float u) {
 __device__ __forceinline__ float gate_mul(float g, float u, int act) { return act == 2 ? gelu_tanh_mul(g, u) : silu_mul(g, u); }
 __device__ __forceinline__ float grouped_act(float z, const GemmParams& p) {
   switch (p.grp_act) {
-    case 5: return xielu(z, p.a_pos, p.a_neg);
+    case 5: return xielu_fast(z, p.a_pos, p.a_neg);
     case 1: { const float r = fmaxf(z, 0.f); return r * r; }
     case 2: return z / (1.f + expf(-z));
     case 3: return gelu_tanh_mul(z, 1.f);
@@ -475,10 +475,12 @@ gemm_tc_kernel(const __grid_constant__ CUtensorMap map_a, const __grid_constant_
 // accumulators back to both CTAs at once.  No load is multicast.
 // CTAs are persistent: a pair walks over tiles (token tile fastest, so that pairs running at the same time read the
 // same few weight tiles from L2), the shared-memory ring runs on across tiles, and the accumulator is double-buffered
-// in tensor memory (2 x 256 columns): the epilogue warps drain tile i while the MMAs of tile i + 1 run.  With GATED
-// the weight rows are (gate, up) pairs and the epilogue writes silu(gate) * up, half as wide.
+// in tensor memory (2 x 256 columns): the epilogue warps drain tile i while the MMAs of tile i + 1 run.  With
+// EPI_GATED the weight rows are (gate, up) pairs and the epilogue writes silu(gate) * up, half as wide; with EPI_ACT it
+// applies the activation grp_act, with EPI_XIELU that one.
 // (Narrower tiles, chosen so that the last round of tiles leaves fewer SMs idle, were measured and are slower at
 // every shape.)
+constexpr int EPI_PLAIN = 0, EPI_GATED = 1, EPI_ACT = 2, EPI_XIELU = 3;
 constexpr int NT = 256;                                                       // columns of the pair's tile
 constexpr int C_STAGES = 6, C_ACC_BUFS = 2, C_TMEM_COLS = NT * C_ACC_BUFS;
 constexpr uint32_t C_A_BYTES = TILE_M * BLOCK_K * 2, C_B_BYTES = (NT / 2) * BLOCK_K * 2;   // this CTA's rows of both operands
@@ -517,7 +519,7 @@ __device__ __forceinline__ void tcgen05_mma_f16_pair(uint32_t d_tmem, uint64_t a
                ::"r"(d_tmem), "l"(a_desc), "l"(b_desc), "r"(idesc), "r"(accumulate) : "memory");
 }
 
-template <typename OutT, bool GATED>
+template <typename OutT, int EPI>
 __global__ void __launch_bounds__(NTHREADS)
 gemm_tc_pair_kernel(const __grid_constant__ CUtensorMap map_a, const __grid_constant__ CUtensorMap map_b, const GemmParams p) {
   extern __shared__ unsigned char smem_dyn[];
@@ -602,7 +604,7 @@ gemm_tc_pair_kernel(const __grid_constant__ CUtensorMap map_a, const __grid_cons
     const int r = quarter * 32 + lane;
     OutT* out = reinterpret_cast<OutT*>(p.out);
     const bool vec = sizeof(OutT) == 2 && (p.ldc % 8 == 0) && ((reinterpret_cast<uintptr_t>(p.out) & 15) == 0);
-    const int n_out = GATED ? p.N / 2 : p.N;
+    const int n_out = EPI == EPI_GATED ? p.N / 2 : p.N;
     uint32_t lt = 0;
     for (int tile = pair; tile < tiles; tile += pairs, ++lt) {
       if (p.tile_expert && p.tile_expert[tile % m_tiles] < 0) { --lt; continue; }         // a tile without rows
@@ -637,18 +639,24 @@ gemm_tc_pair_kernel(const __grid_constant__ CUtensorMap map_a, const __grid_cons
           for (int j = 0; j < 16; ++j) { v[0][j] = 0u; v[1][j] = 0u; }
         }
         if (t >= p.tokens || skip_row) continue;
-        if (p.tile_expert || p.grp_act) {
+        if constexpr (EPI == EPI_ACT || EPI == EPI_XIELU) {
 #pragma unroll
           for (int h = 0; h < 2; ++h)
 #pragma unroll
             for (int j = 0; j < 16; ++j) {
               const float x = __uint_as_float(v[h][j]);
-              v[h][j] = __float_as_uint(p.grp_epi == 0 ? grouped_act(x, p) : x * row_scale);
+              v[h][j] = __float_as_uint(EPI == EPI_XIELU ? xielu_fast(x, p.a_pos, p.a_neg) : grouped_act(x, p));
             }
+        }
+        if (EPI == EPI_PLAIN && p.row_w) {                      // grouped, second product: times the row's weight
+#pragma unroll
+          for (int h = 0; h < 2; ++h)
+#pragma unroll
+            for (int j = 0; j < 16; ++j) v[h][j] = __float_as_uint(__uint_as_float(v[h][j]) * row_scale);
         }
 #pragma unroll
         for (int h = 0; h < 2; ++h) {
-          if constexpr (GATED) {
+          if constexpr (EPI == EPI_GATED) {
             const int o0 = (n0 + c0 + h * 16) >> 1;
             OutT* dst = out + (int64_t)t * p.ldc + o0;
             float y[8];
@@ -801,9 +809,9 @@ int cluster_pairs_resident(const void* kernel, size_t smem) {
   return n;
 }
 
-template <typename OutT, bool GATED>
+template <typename OutT, int EPI>
 int launch_pair(const CUtensorMap& ma, const CUtensorMap& mb, const GemmParams& p, cudaStream_t stream) {
-  auto k = gemm_tc_pair_kernel<OutT, GATED>;
+  auto k = gemm_tc_pair_kernel<OutT, EPI>;
   static int max_pairs = 0;
   if (!max_pairs) {
     cudaError_t e = cudaFuncSetAttribute(k, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)C_SMEM_BYTES);
@@ -896,8 +904,11 @@ DINFER_API int dinfer_gemm_tc_all(const void* x, int64_t ldx, const void* w, int
   p.splits = 1;
   if ((rc = make_map(&ma, x, tokens, K, ldx, TILE_M))) return rc;
   if ((rc = make_map(&mb, w, N, K, ldw, NT / 2))) return rc;
-  if (act) return out_f32 ? launch_pair<float, true>(ma, mb, p, stream) : launch_pair<__nv_bfloat16, true>(ma, mb, p, stream);
-  return out_f32 ? launch_pair<float, false>(ma, mb, p, stream) : launch_pair<__nv_bfloat16, false>(ma, mb, p, stream);
+#define GO(EPI) (out_f32 ? launch_pair<float, EPI>(ma, mb, p, stream) : launch_pair<__nv_bfloat16, EPI>(ma, mb, p, stream))
+  if (act) return GO(EPI_GATED);
+  if (unary == 5) return GO(EPI_XIELU);
+  return unary ? GO(EPI_ACT) : GO(EPI_PLAIN);
+#undef GO
 }
 
 DINFER_API int dinfer_gemm_tc_fused(const void* x, int64_t ldx, const void* w, int64_t ldw, void* out, int64_t ldc,
@@ -911,13 +922,15 @@ DINFER_API int dinfer_gemm_tc_fused(const void* x, int64_t ldx, const void* w, i
 // Grouped product of a routed feed-forward's prompt-sized steps on the two-SM kernel: x [cap, K] holds the rows expert
 // by expert, every expert's run padded to a multiple of 256 (cap a multiple of 256), tile_expert [cap / 256] names the
 // expert of each 256-row tile (-1: none); w [E * N, K] holds the experts' matrices one behind the other.
-// epi 0: out [cap, N] = act(x w_e^T) row for row (act: 0 none, 1 relu squared, 2 silu, 3 tanh-gelu, 4 relu);
+// epi 0: out [cap, N] = act(x w_e^T) row for row (act: 0 none, 1 relu squared, 2 silu, 3 tanh-gelu, 4 relu), or with gate
+// (1 silu, 2 tanh-gelu; N even, act 0) the expert's rows are (gate, up) pairs and out [cap, N / 2] = g(gate) * up;
 // epi 1: out [pairs, N]: row t of the product, times row_w[sorted[t]], goes to row sorted[t] (sorted[t] >= pairs: padding).
 DINFER_API int dinfer_gemm_tc_grouped(const void* x, int64_t ldx, const void* w, void* out, int64_t ldc,
                                       const int* tile_expert, const int* sorted, const float* row_w, int cap, int pairs,
-                                      int E, int N, int K, int epi, int act, int* status, cudaStream_t stream) {
+                                      int E, int N, int K, int epi, int act, int gate, int* status, cudaStream_t stream) {
   if (cap <= 0 || cap % 256 || pairs < 0 || E <= 0 || N <= 0 || K <= 0 || !tile_expert || (epi != 0 && epi != 1) ||
-      (epi == 1 && (!sorted || !row_w)) || act < 0 || act > 4)
+      (epi == 1 && (!sorted || !row_w)) || act < 0 || act > 4 || gate < 0 || gate > 2 || (gate && (epi || act || (N & 1))) ||
+      (epi == 1 && act))
     return refuse(DINFER_BAD_ARGUMENT, "gemm_tc_grouped: bad arguments cap=%d pairs=%d E=%d N=%d K=%d epi=%d", cap, pairs, E, N, K, epi);
   if ((K % 8) || (ldx % 8) || (reinterpret_cast<uintptr_t>(x) & 15) || (reinterpret_cast<uintptr_t>(w) & 15))
     return refuse(DINFER_BAD_ARGUMENT, "gemm_tc_grouped: K and the row stride must be multiples of 8 and the bases 16-byte aligned (TMA)");
@@ -925,12 +938,14 @@ DINFER_API int dinfer_gemm_tc_grouped(const void* x, int64_t ldx, const void* w,
   GemmParams p = {};
   p.out = out; p.ldc = ldc; p.tokens = cap; p.N = N; p.K = K; p.status = status;
   p.k_blocks_per_split = (K + BLOCK_K - 1) / BLOCK_K; p.splits = 1;
-  p.tile_expert = tile_expert; p.sorted = sorted; p.row_w = row_w; p.pairs = pairs; p.grp_epi = epi; p.grp_act = act;
+  p.tile_expert = tile_expert; p.sorted = sorted; p.row_w = epi == 1 ? row_w : nullptr; p.pairs = pairs; p.grp_epi = epi; p.grp_act = act;
+  p.act = gate;
   CUtensorMap ma, mb;
   int rc;
   if ((rc = make_map(&ma, x, cap, K, ldx, TILE_M))) return rc;
   if ((rc = make_map(&mb, w, (int64_t)E * N, K, K, NT / 2))) return rc;
-  return launch_pair<__nv_bfloat16, false>(ma, mb, p, stream);
+  if (gate) return launch_pair<__nv_bfloat16, EPI_GATED>(ma, mb, p, stream);
+  return act ? launch_pair<__nv_bfloat16, EPI_ACT>(ma, mb, p, stream) : launch_pair<__nv_bfloat16, EPI_PLAIN>(ma, mb, p, stream);
 }
 
 DINFER_API int dinfer_gemm_tc(const void* x, int64_t ldx, const void* w, int64_t ldw, void* out, int64_t ldc,

@@ -476,8 +476,8 @@ moe_combine_bf16x8_kernel(const __nv_bfloat16* __restrict__ y, const __nv_bfloat
   *reinterpret_cast<uint4*>(out + (int64_t)t * h + i) = o;
 }
 
-// a[pos] = x[sorted[pos] / top] (zeros for padding): the rows of a step laid out expert by expert, for products that
-// want every expert's rows side by side in memory
+// a[pos] = x[sorted[pos] / top]: the rows of a step laid out expert by expert, for products that want every expert's rows
+// side by side in memory.  Rows that pad a run are left as they are: a product's rows do not depend on one another.
 template <typename TA>
 __global__ void __launch_bounds__(256)
 moe_gather_kernel(const TA* __restrict__ x, int64_t ldx, const int* __restrict__ sorted, TA* __restrict__ a, int pairs,
@@ -485,15 +485,16 @@ moe_gather_kernel(const TA* __restrict__ x, int64_t ldx, const int* __restrict__
   pdl_enter();
   const int pos = blockIdx.x;
   const int pr = sorted[pos];
+  if (pr >= pairs) return;
   TA* dst = a + (int64_t)pos * h;
-  const TA* src = pr < pairs ? x + (int64_t)(pr / top) * ldx : nullptr;
+  const TA* src = x + (int64_t)(pr / top) * ldx;
   const bool vec = sizeof(TA) == 2 && h % 8 == 0 && ldx % 8 == 0 && !(reinterpret_cast<uintptr_t>(x) & 15) &&
                    !(reinterpret_cast<uintptr_t>(a) & 15);
   if (vec) {
     for (int i = threadIdx.x * 8; i < h; i += blockDim.x * 8)
-      *reinterpret_cast<uint4*>(dst + i) = src ? *reinterpret_cast<const uint4*>(src + i) : make_uint4(0, 0, 0, 0);
+      *reinterpret_cast<uint4*>(dst + i) = *reinterpret_cast<const uint4*>(src + i);
   } else {
-    for (int i = threadIdx.x; i < h; i += blockDim.x) dst[i] = src ? src[i] : from_f32<TA>(0.f);
+    for (int i = threadIdx.x; i < h; i += blockDim.x) dst[i] = src[i];
   }
 }
 
@@ -518,7 +519,7 @@ __global__ void xielu_bf16x8_kernel(const uint4* __restrict__ x, uint4* __restri
 #pragma unroll
     for (int j = 0; j < 4; ++j) {
       const float2 f = __bfloat1622float2(p[j]);
-      p[j] = __floats2bfloat162_rn(xielu(f.x, a_pos, a_neg), xielu(f.y, a_pos, a_neg));
+      p[j] = __floats2bfloat162_rn(xielu_fast(f.x, a_pos, a_neg), xielu_fast(f.y, a_pos, a_neg));
     }
     out[i] = v;
   }

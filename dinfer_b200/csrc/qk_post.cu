@@ -488,8 +488,8 @@ qkv_post_general_kernel(TA* __restrict__ qkv, int64_t ld, const int* __restrict_
 
 // The usual case of it in bfloat16 without shared memory: keys and values D = 8 * LPH wide, weighted head norms ahead
 // of a rotation in halves, nothing else.  LPH lanes own a head, eight neighbouring elements each (one 16-byte load and
-// store); the partner of a rotated element is held by another lane of the head.  A thread keeps its cosines and sines
-// while it walks over the token's heads.
+// store); the partner of a rotated element is held by another lane of the head.  (Two or three
+// heads a thread, with their loads ahead of the work, measured slower: fewer CTAs fit an SM.)
 template <typename TW, int LPH>
 __global__ void __launch_bounds__(256)
 qkv_post_turn_kernel(__nv_bfloat16* __restrict__ qkv, int64_t ld, const int* __restrict__ positions,
@@ -515,57 +515,52 @@ qkv_post_turn_kernel(__nv_bfloat16* __restrict__ qkv, int64_t ld, const int* __r
   }
   const int slot = (cache && slots) ? slots[t] : -1;
   pdl_wait();
-  const int step = gridDim.y * GROUPS;
-  const int rounds = (heads + step - 1) / step;
-  for (int r = 0; r < rounds; ++r) {
-    const int head = (r * gridDim.y + blockIdx.y) * GROUPS + threadIdx.x / LPH;
-    const bool live = head < heads;
-    const int kind = head < H ? 0 : (head < H + Hkv ? 1 : 2);
-    __nv_bfloat16* x = qkv + (int64_t)t * ld + (int64_t)head * D + 8 * l;
-    float a[8], c[8], s[8];
+  const int head = blockIdx.y * GROUPS + threadIdx.x / LPH;
+  const bool live = head < heads;
+  const int kind = head < H ? 0 : (head < H + Hkv ? 1 : 2);
+  __nv_bfloat16* x = qkv + (int64_t)t * ld + (int64_t)head * D + 8 * l;
+  float a[8], c[8], s[8];
 #pragma unroll
-    for (int j = 0; j < 8; ++j) { a[j] = 0.f; c[j] = c_k[j]; s[j] = s_k[j]; }
-    int pl = pl_k, n = rot;
-    if (live) load8<__nv_bfloat16>(x, a);
-    if (kind == 2) {
-      pl = pl_v;
-      n = D;
-      if (pl) {
-        const float* cs = v_cos_sin + (int64_t)pos * D + 8 * l - (pl == 2 ? D / 2 : 0);
-        load8<float>(cs, c);
-        load8<float>(cs + D / 2, s);
-      }
-    }
-    __syncwarp();
-    float ss = 0.f;
-#pragma unroll
-    for (int j = 0; j < 8; ++j) ss += a[j] * a[j];
-#pragma unroll
-    for (int o = LPH / 2; o > 0; o >>= 1) ss += __shfl_xor_sync(0xffffffffu, ss, o);
-    const TW* w = kind == 0 ? q_weight : k_weight;
-    if (live && kind != 2 && w) {
-      const float rinv = rsqrtf(ss / (float)D + eps);
-      float wv[8];
-      load8<TW>(w + 8 * l, wv);
-#pragma unroll
-      for (int j = 0; j < 8; ++j) a[j] = a[j] * rinv * wv[j];
-    }
-    const int other = lane + (pl == 1 ? n / 16 : (pl == 2 ? -(n / 16) : 0));
-    float b[8];
-#pragma unroll
-    for (int j = 0; j < 8; ++j) b[j] = __shfl_sync(0xffffffffu, a[j], other);
+  for (int j = 0; j < 8; ++j) { a[j] = 0.f; c[j] = c_k[j]; s[j] = s_k[j]; }
+  if (live) load8<__nv_bfloat16>(x, a);
+  int pl = pl_k, n = rot;
+  if (kind == 2) {
+    pl = pl_v;
+    n = D;
     if (pl) {
-      const float sign = pl == 1 ? -1.f : 1.f;
+      const float* cs = v_cos_sin + (int64_t)pos * D + 8 * l - (pl == 2 ? D / 2 : 0);
+      load8<float>(cs, c);
+      load8<float>(cs + D / 2, s);
+    }
+  }
+  __syncwarp();
+  float ss = 0.f;
 #pragma unroll
-      for (int j = 0; j < 8; ++j) a[j] = a[j] * c[j] + sign * b[j] * s[j];
-    }
-    if (!live) continue;
-    if (kind != 2) store8<__nv_bfloat16>(x, a);
-    if (kind != 0 && slot >= 0) {
-      const int hk = kind == 1 ? head - H : head - H - Hkv;
-      const int64_t blk = slot / block_size, off = slot % block_size;
-      store8<__nv_bfloat16>(cache + (((blk * 2 + (kind == 2)) * Hkv + hk) * block_size + off) * D + 8 * l, a);
-    }
+  for (int j = 0; j < 8; ++j) ss += a[j] * a[j];
+#pragma unroll
+  for (int o = LPH / 2; o > 0; o >>= 1) ss += __shfl_xor_sync(0xffffffffu, ss, o);
+  const TW* w = kind == 0 ? q_weight : k_weight;
+  if (live && kind != 2 && w) {
+    const float rinv = rsqrtf(ss / (float)D + eps);
+    float wv[8];
+    load8<TW>(w + 8 * l, wv);
+#pragma unroll
+    for (int j = 0; j < 8; ++j) a[j] = a[j] * rinv * wv[j];
+  }
+  const int other = lane + (pl == 1 ? n / 16 : (pl == 2 ? -(n / 16) : 0));
+  float b[8];
+#pragma unroll
+  for (int j = 0; j < 8; ++j) b[j] = __shfl_sync(0xffffffffu, a[j], other);
+  if (pl) {
+    const float sign = pl == 1 ? -1.f : 1.f;
+#pragma unroll
+    for (int j = 0; j < 8; ++j) a[j] = a[j] * c[j] + sign * b[j] * s[j];
+  }
+  if (live && kind != 2) store8<__nv_bfloat16>(x, a);
+  if (live && kind != 0 && slot >= 0) {
+    const int hk = kind == 1 ? head - H : head - H - Hkv;
+    const int64_t blk = slot / block_size, off = slot % block_size;
+    store8<__nv_bfloat16>(cache + (((blk * 2 + (kind == 2)) * Hkv + hk) * block_size + off) * D + 8 * l, a);
   }
 }
 
@@ -573,9 +568,8 @@ template <typename TW, int LPH>
 void launch_turn(void* qkv, int64_t ld, const int* positions, const void* qw, const void* kw, float eps, const float* cos_sin,
                  int rot, const float* v_cos_sin, void* cache, const int* slots, int block_size, int T, int H, int Hkv,
                  cudaStream_t stream) {
-  const int groups = 256 / LPH, all = (H + 2 * Hkv + groups - 1) / groups;
-  // few tokens: a head a thread group; many: a CTA walks over its token's heads
-  launch_pdl(qkv_post_turn_kernel<TW, LPH>, dim3(T, T >= 512 ? 1 : all), dim3(256), 0, stream, (__nv_bfloat16*)qkv, ld, positions,
+  constexpr int groups = 256 / LPH;
+  launch_pdl(qkv_post_turn_kernel<TW, LPH>, dim3(T, (H + 2 * Hkv + groups - 1) / groups), dim3(256), 0, stream, (__nv_bfloat16*)qkv, ld, positions,
              (const TW*)qw, (const TW*)kw, eps, cos_sin, rot, v_cos_sin, (__nv_bfloat16*)cache, slots, block_size, H, Hkv);
 }
 

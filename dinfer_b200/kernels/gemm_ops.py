@@ -104,7 +104,9 @@ def decode_splits(tokens: int, N: int, K: int) -> int:
     tiles = (N + 127) // 128
     k_blocks = (K + 63) // 64
     sms = num_sms()
-    slots = 3 * sms if tokens <= 16 else 2 * sms - 16
+    # a tile's CTAs are one cluster and a cluster stays inside a part of the chip, so not every slot can be filled:
+    # 384 CTAs in clusters of 8 run as one wave of 3 an SM, 392 do not, nor do 432 in clusters of 3
+    slots = 3 * sms - 58 if tokens <= 16 else 2 * sms - 16
     return max(1, min(slots // tiles, k_blocks // 8, MAX_SPLITS))
 
 

@@ -107,7 +107,8 @@ def tc_grouped_supported(x: torch.Tensor, w_up: torch.Tensor, w_down: torch.Tens
 
 
 def gather_rows(x: torch.Tensor, sorted_: torch.Tensor, pairs: int, top_k: int) -> torch.Tensor:
-    """The step's rows laid out expert by expert: a[pos] = x[sorted[pos] // top_k], zeros where the layout pads."""
+    """The step's rows laid out expert by expert: a[pos] = x[sorted[pos] // top_k]; rows where the
+    layout pads are left as they are (no row of a product depends on another, and the last product drops theirs)."""
     require_cuda(x, sorted_)
     _rows_contiguous(x, "moe gather")
     cap, h = sorted_.numel(), x.shape[1]
@@ -119,16 +120,20 @@ def gather_rows(x: torch.Tensor, sorted_: torch.Tensor, pairs: int, top_k: int) 
 
 
 def grouped_gemm_tc(a: torch.Tensor, w: torch.Tensor, out: torch.Tensor, sorted_: torch.Tensor, tile_expert: torch.Tensor,
-                    pairs: int, mode: int, activation: str = "none", weights: Optional[torch.Tensor] = None) -> torch.Tensor:
+                    pairs: int, mode: int, activation: str = "none", weights: Optional[torch.Tensor] = None,
+                    gate: Optional[str] = None) -> torch.Tensor:
     """The grouped product on the two-SM tcgen05 kernel (bfloat16; the layout padded to ``TC_ROW_TILE`` rows per
     expert run).  a [cap, K] by position.  mode 0: ``out[pos] = act(a[pos] @ w[e]^T)`` (out [cap, N]); mode 1:
-    ``out[pair] = (a[pos] @ w[e]^T) * weights[pair]`` (out [pairs, N])."""
+    ``out[pair] = (a[pos] @ w[e]^T) * weights[pair]`` (out [pairs, N]).  ``gate`` (mode 0; "silu" or "gelu_tanh"): the rows
+    of w[e] are (gate, up) pairs and out is [cap, N / 2], act(gate) * up."""
     from . import gemm_ops
     require_cuda(a, w, out, sorted_, tile_expert, weights)
     E, N, K = w.shape
     cap = sorted_.numel()
+    if gate is not None and (gate not in gemm_ops.GATES or mode != 0 or activation != "none" or N % 2):
+        raise KernelError("moe grouped_gemm_tc: a gate belongs to mode 0, (gate, up) row pairs and no other activation")
     if a.dtype != torch.bfloat16 or w.dtype != torch.bfloat16 or out.dtype != torch.bfloat16 or not w.is_contiguous() \
-            or tuple(a.shape) != (cap, K) or a.stride(1) != 1 or out.stride(1) != 1 or out.shape[1] != N \
+            or tuple(a.shape) != (cap, K) or a.stride(1) != 1 or out.stride(1) != 1 or out.shape[1] != (N // 2 if gate else N) \
             or cap % TC_ROW_TILE or tile_expert.numel() != cap // TC_ROW_TILE:
         raise KernelError("moe grouped_gemm_tc: bfloat16 a [cap, K], w [E, N, K], out [*, N]; cap in whole tiles")
     if (mode == 0 and out.shape[0] != cap) or (mode == 1 and (out.shape[0] != pairs or weights is None
@@ -137,9 +142,9 @@ def grouped_gemm_tc(a: torch.Tensor, w: torch.Tensor, out: torch.Tensor, sorted_
     st = gemm_ops._state(a.device)
     lib, f = _fn("gemm_tc", "dinfer_gemm_tc_grouped",
                  [c_void_p, c_int64, c_void_p, c_void_p, c_int64, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int,
-                  c_int, c_int, c_int, c_void_p, c_void_p])
+                  c_int, c_int, c_int, c_int, c_void_p, c_void_p])
     check(lib, f(ptr(a), a.stride(0), ptr(w), ptr(out), out.stride(0), ptr(tile_expert), ptr(sorted_), ptr(weights), cap,
-                 pairs, E, N, K, int(mode), ACTIVATIONS[activation], ptr(st["status"]), stream_handle()), "gemm_tc_grouped")
+                 pairs, E, N, K, int(mode), ACTIVATIONS[activation], gemm_ops.GATES[gate], ptr(st["status"]), stream_handle()), "gemm_tc_grouped")
     return out
 
 

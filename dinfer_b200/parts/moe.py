@@ -22,7 +22,7 @@ from typing import Dict, List, Optional
 
 import torch
 
-from ..kernels import moe_ops
+from ..kernels import gemm_ops, moe_ops
 from .base import FEED_FORWARDS, FeedForward
 from .linear import Linear
 from .spec import TensorDecl
@@ -182,9 +182,13 @@ class MoE(FeedForward):
             # prompt-sized steps: rows laid out expert by expert in whole 256-row tiles, both products on tcgen05
             order, tile_expert = moe_ops.align(ids, self.E, moe_ops.TC_ROW_TILE)
             a = moe_ops.gather_rows(x, order, pairs, self.top)
-            u = torch.empty((order.numel(), wide), dtype=x.dtype, device=x.device)
-            moe_ops.grouped_gemm_tc(a, self.w_up, u, order, tile_expert, pairs, 0, first_act)
-            u, weights = self._gate(u, order, weights)
+            if self.gated and not self.weight_on_input and self.activation in gemm_ops.GATES:
+                u = torch.empty((order.numel(), self.ff), dtype=x.dtype, device=x.device)      # the gate in the epilogue
+                moe_ops.grouped_gemm_tc(a, self.w_up, u, order, tile_expert, pairs, 0, gate=self.activation)
+            else:
+                u = torch.empty((order.numel(), wide), dtype=x.dtype, device=x.device)
+                moe_ops.grouped_gemm_tc(a, self.w_up, u, order, tile_expert, pairs, 0, first_act)
+                u, weights = self._gate(u, order, weights)
             y = torch.empty((pairs, self.hidden), dtype=x.dtype, device=x.device)
             moe_ops.grouped_gemm_tc(u, self.w_down, y, order, tile_expert, pairs, 1, weights=weights)
             return self._combine(x, y, gate, identity)
