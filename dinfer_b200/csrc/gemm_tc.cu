@@ -531,6 +531,10 @@ gemm_tc_pair_kernel(const __grid_constant__ CUtensorMap map_a, const __grid_cons
   const uint32_t rank = cluster_ctarank();                      // 0 = leader
   const int m_tiles = (p.tokens + 255) / 256, n_tiles = (p.N + NT - 1) / NT;
   const int tiles = m_tiles * n_tiles;
+  // the order of the tiles: token tile fastest, so that pairs running at the same time read the same few weight tiles; in
+  // grouped mode weight tile fastest, because a row tile has an expert's weights to itself and its rows are what is shared
+  const auto m_of = [&](int tile) { return p.tile_expert ? tile / n_tiles : tile % m_tiles; };
+  const auto n_of = [&](int tile) { return p.tile_expert ? tile % n_tiles : tile / m_tiles; };
   const int total_kb = (p.K + BLOCK_K - 1) / BLOCK_K;
   const int pair = blockIdx.x >> 1, pairs = gridDim.x >> 1;
   pdl_enter();
@@ -560,9 +564,9 @@ gemm_tc_pair_kernel(const __grid_constant__ CUtensorMap map_a, const __grid_cons
       bool ok = true;
       for (int tile = pair; tile < tiles && ok; tile += pairs) {
         int expert = 0;
-        if (p.tile_expert) { expert = p.tile_expert[tile % m_tiles]; if (expert < 0) continue; }
-        const int m0 = (tile % m_tiles) * 256 + (int)rank * 128;
-        const int n0 = expert * p.N + (tile / m_tiles) * NT + (int)rank * (NT / 2);
+        if (p.tile_expert) { expert = p.tile_expert[m_of(tile)]; if (expert < 0) continue; }
+        const int m0 = m_of(tile) * 256 + (int)rank * 128;
+        const int n0 = expert * p.N + n_of(tile) * NT + (int)rank * (NT / 2);
         for (int kb = 0; kb < total_kb; ++kb, ++it) {
           const uint32_t s = it % C_STAGES;
           if (!mbar_wait(smem_u32(&empty_bar[s]), ((it / C_STAGES) & 1) ^ 1)) { s_abort = 1; atomicExch(p.status, 1); ok = false; break; }
@@ -580,7 +584,7 @@ gemm_tc_pair_kernel(const __grid_constant__ CUtensorMap map_a, const __grid_cons
       uint32_t it = 0, lt = 0;
       bool ok = true;
       for (int tile = pair; tile < tiles && ok; tile += pairs, ++lt) {
-        if (p.tile_expert && p.tile_expert[tile % m_tiles] < 0) { --lt; continue; }       // a tile without rows
+        if (p.tile_expert && p.tile_expert[m_of(tile)] < 0) { --lt; continue; }       // a tile without rows
         const uint32_t b = lt % C_ACC_BUFS;
         if (!mbar_wait_cluster(smem_u32(&acc_empty_bar[b]), ((lt / C_ACC_BUFS) & 1) ^ 1)) { s_abort = 1; atomicExch(p.status, 2); break; }
         tcgen05_fence_after();
@@ -607,9 +611,9 @@ gemm_tc_pair_kernel(const __grid_constant__ CUtensorMap map_a, const __grid_cons
     const int n_out = EPI == EPI_GATED ? p.N / 2 : p.N;
     uint32_t lt = 0;
     for (int tile = pair; tile < tiles; tile += pairs, ++lt) {
-      if (p.tile_expert && p.tile_expert[tile % m_tiles] < 0) { --lt; continue; }         // a tile without rows
+      if (p.tile_expert && p.tile_expert[m_of(tile)] < 0) { --lt; continue; }         // a tile without rows
       const uint32_t b = lt % C_ACC_BUFS;
-      const int m0 = (tile % m_tiles) * 256 + (int)rank * 128, n0 = (tile / m_tiles) * NT;
+      const int m0 = m_of(tile) * 256 + (int)rank * 128, n0 = n_of(tile) * NT;
       if (total_kb > 0) {
         if (!mbar_wait(smem_u32(&acc_full_bar[b]), (lt / C_ACC_BUFS) & 1)) {
           if (lane == 0) { s_abort = 1; atomicExch(p.status, 3); }
