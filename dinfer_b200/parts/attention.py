@@ -251,7 +251,8 @@ class GQAttention(Mixer):
         if self._fast(q.dtype):
             splits = ctx.decode_splits or attention_ops.decode_splits(ctx.num_reqs, self.Hkv, ctx.max_seq_len)
             if self.chunked:                                # a decoded token sees its chunk at most: no more splits than that fills
-                splits = min(splits, attention_ops.decode_splits(ctx.num_reqs, self.Hkv, min(window, ctx.max_seq_len)))
+                longest = int(self.env.max_positions) if ctx.decode_splits else ctx.max_seq_len    # (a captured graph's bound)
+                splits = min(splits, attention_ops.decode_splits(ctx.num_reqs, self.Hkv, min(window, longest)))
             tc_decode = ctx.any_decode
             if ctx.any_decode and attention_ops.decode_supported(q.dtype, self.D, self.H // self.Hkv, g.block_size) \
                     and (g.block_size >= 8 or not (self.sink or self.slopes is not None or self.chunked)):
