@@ -191,7 +191,8 @@ template <int N_TILE, int STAGES> constexpr size_t gemm_smem_bytes(bool with_rec
 }
 
 // grid: (tiles of the 128-row operand, tiles of the N_TILE-row operand, K splits)
-template <int N_TILE, int STAGES, typename OutT>
+// UNARY: the activation grp_act on the result (kernels of their own: its code slows the plain product down)
+template <int N_TILE, int STAGES, typename OutT, bool UNARY>
 __global__ void __launch_bounds__(NTHREADS)
 gemm_tc_kernel(const __grid_constant__ CUtensorMap map_a, const __grid_constant__ CUtensorMap map_b, const GemmParams p) {
   extern __shared__ unsigned char smem_dyn[];
@@ -358,7 +359,7 @@ gemm_tc_kernel(const __grid_constant__ CUtensorMap map_a, const __grid_constant_
             if (n < p.N) {
 #pragma unroll
               for (int j = 0; j < 16; ++j)
-                if (b0 + c0 + j < p.tokens) out[(int64_t)(b0 + c0 + j) * p.ldc + n] = out_cast<OutT>(grouped_act(__uint_as_float(v[j]), p));
+                if (b0 + c0 + j < p.tokens) out[(int64_t)(b0 + c0 + j) * p.ldc + n] = out_cast<OutT>(UNARY ? grouped_act(__uint_as_float(v[j]), p) : __uint_as_float(v[j]));
             }
           } else {
             // recv[split][token column][row of the owner's share]: consecutive lanes, consecutive words
@@ -451,7 +452,7 @@ gemm_tc_kernel(const __grid_constant__ CUtensorMap map_a, const __grid_constant_
           for (int s = 0; s < p.splits; ++s) acc += recv[(s * N_TILE + c) * rows_per + rl];
           if (p.ss_in) acc *= s_rstd[c];
           const int n = a0 + rank * rows_per + rl;
-          if (n < p.N) out[(int64_t)(b0 + c) * p.ldc + n] = out_cast<OutT>(grouped_act(acc, p));
+          if (n < p.N) out[(int64_t)(b0 + c) * p.ldc + n] = out_cast<OutT>(UNARY ? grouped_act(acc, p) : acc);
         }
       }
     }
@@ -752,9 +753,9 @@ int make_map(CUtensorMap* map, const void* base, int64_t rows, int64_t K, int64_
   return 0;
 }
 
-template <int N_TILE, int STAGES, typename OutT>
-int launch(const CUtensorMap& ma, const CUtensorMap& mb, const GemmParams& p, dim3 grid, cudaStream_t stream) {
-  auto k = gemm_tc_kernel<N_TILE, STAGES, OutT>;
+template <int N_TILE, int STAGES, typename OutT, bool UNARY>
+int launch_decode(const CUtensorMap& ma, const CUtensorMap& mb, const GemmParams& p, dim3 grid, cudaStream_t stream) {
+  auto k = gemm_tc_kernel<N_TILE, STAGES, OutT, UNARY>;
   const size_t sm = gemm_smem_bytes<N_TILE, STAGES>(p.splits > 1 || p.resid != nullptr);
   static bool opted = false;
   if (!opted) {
@@ -765,6 +766,11 @@ int launch(const CUtensorMap& ma, const CUtensorMap& mb, const GemmParams& p, di
   cudaError_t e = launch_pdl_cluster(k, grid, dim3(NTHREADS), dim3(1, 1, p.splits), sm, stream, ma, mb, p);
   if (e != cudaSuccess) return refuse((int)e, "gemm_tc: launch failed: %s", cudaGetErrorString(e));
   return cuda_status("gemm_tc");
+}
+template <int N_TILE, int STAGES, typename OutT>
+int launch(const CUtensorMap& ma, const CUtensorMap& mb, const GemmParams& p, dim3 grid, cudaStream_t stream) {
+  return p.grp_act ? launch_decode<N_TILE, STAGES, OutT, true>(ma, mb, p, grid, stream)
+                   : launch_decode<N_TILE, STAGES, OutT, false>(ma, mb, p, grid, stream);
 }
 
 // What every bounded wait of this file does when it runs out, on its own: one CTA allocates tensor memory, waits

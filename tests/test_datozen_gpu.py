@@ -349,6 +349,20 @@ def test_xielu_feed_forward(dtype, ff, width, T):
     close(part.forward(dev(x, DT[dtype])).double().cpu(), P.dense_ff(x.double(), W), dtype)
 
 
+@pytest.mark.parametrize("act", ["relu", "relu2", "silu", "gelu_tanh"])
+@pytest.mark.parametrize("T, width, ff", [(5, 128, 96), (9, 1024, 256), (600, 64, 136)])
+def test_other_activations_without_a_gate(act, T, width, ff):
+    """The same epilogues with the other activations (few rows with and without split K, prompt rows)."""
+    import dinfer_b200.models.decoder  # noqa: F401
+    from dinfer_b200.parts.base import FEED_FORWARDS
+    part = FEED_FORWARDS.get("plain_mlp")({"intermediate_size": ff, "activation": act}, env(width, torch.bfloat16), "")
+    W = weights_for(part.declare(), "bfloat16", ff, std=1.0 / width ** 0.5)
+    part.bind({k: dev(v, torch.bfloat16) for k, v in W.items()})
+    x = torch.randn(T, width, generator=torch.Generator().manual_seed(T)).to(torch.bfloat16).float()
+    f = {"relu": lambda z: z.clamp(min=0), "relu2": lambda z: z.clamp(min=0) ** 2, "silu": P.silu, "gelu_tanh": P.gelu_tanh}[act]
+    close(part.forward(dev(x, torch.bfloat16)).double().cpu(), P.lin(f(P.lin(x.double(), W["up_proj.weight"])), W["down_proj.weight"]), "bfloat16")
+
+
 @pytest.mark.parametrize("dtype", ["float32", "bfloat16"])
 def test_xielu_values(dtype):
     from dinfer_b200.kernels import moe_ops
