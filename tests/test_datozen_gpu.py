@@ -201,7 +201,7 @@ def test_plain_kernel_windows_and_sinks(dtype, chunked, window):
 
 @pytest.mark.parametrize("dtype", ["float32", "bfloat16"])
 @pytest.mark.parametrize("H_, G, D, V, rot, T", [(4, 2, 64, 64, 32, 9), (32, 8, 128, 128, 64, 600), (3, 3, 128, 128, 128, 3), (6, 2, 256, 256, 16, 5),
-                                                 (4, 2, 64, 64, 20, 7), (4, 2, 12, 20, 8, 11), (2, 1, 96, 96, 48, 4), (5, 1, 64, 32, 64, 6)])
+                                                 (4, 2, 64, 64, 20, 7), (4, 2, 12, 20, 8, 11), (2, 1, 80, 80, 40, 4), (5, 1, 64, 32, 64, 6)])
 def test_keys_and_values_turned(dtype, H_, G, D, V, rot, T):
     """Head norm, rotation and the turned values in the cache: sizes of the kernel without shared memory (a token's heads
     walked over, or a thread group each) and of the general one; slots all over the cache, tokens that are not stored."""
@@ -242,7 +242,7 @@ def test_keys_and_values_turned(dtype, H_, G, D, V, rot, T):
 
 
 @pytest.mark.parametrize("dtype", ["float32", "bfloat16"])
-@pytest.mark.parametrize("H_, V, T", [(4, 64, 5), (32, 128, 600), (6, 96, 3), (3, 20, 7), (2, 6, 4), (1, 256, 2), (5, 7, 3)])
+@pytest.mark.parametrize("H_, V, T", [(4, 64, 5), (32, 128, 600), (6, 112, 3), (3, 20, 7), (2, 6, 4), (1, 256, 2), (5, 7, 3)])
 @pytest.mark.parametrize("turned, gated", [(True, True), (True, False), (False, True)])
 def test_heads_out(dtype, H_, V, T, turned, gated):
     from dinfer_b200.kernels import ops
