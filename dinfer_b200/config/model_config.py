@@ -1072,3 +1072,216 @@ class DatozenConfig:
         if self.eos_token_ids:
             d["eos_token_id"] = list(self.eos_token_ids)
         return d
+
+
+# ---------------------------------------------------------------- Rorutar
+
+@dataclass(frozen=True)
+class KeptWindowAttentionSizes:
+    """The left half of a ``parallel`` mixer of Rorutar: grouped heads (queries and keys of ``dim``, values of ``vdim``
+    elements) over the last ``window`` tokens (None: all) and a request's ``keep_first`` first ones; the first ``rot_dims``
+    elements rotate in halves, positions divided by ``rot_factor``; ``softcap`` > 0: soft-capped scores."""
+    heads: int
+    kv_heads: int
+    dim: int
+    vdim: int
+    scale: float
+    rot_base: float
+    rot_dims: int
+    rot_factor: float = 1.0
+    softcap: float = 0.0
+    window: Optional[int] = None
+    keep_first: int = 0
+
+    @classmethod
+    def from_dict(cls, m: Dict[str, Any], where: str) -> "KeptWindowAttentionSizes":
+        heads, dim = _take(m, "heads", int), _take(m, "dim", int)
+        rot = _section(m, "rot", where)
+        scaling = _section(rot, "scaling", where, optional=True)
+        mask = _section(m, "mask", where, optional=True) or {}
+        window = _take(mask, "size", int, None)
+        s = cls(heads=heads, kv_heads=_take(m, "kv_heads", int, heads), dim=dim, vdim=_take(m, "vdim", int, dim),
+                scale=_take(m, "scale", float), rot_base=_take(rot, "base", float), rot_dims=_take(rot, "dims", int),
+                rot_factor=_take(scaling, "factor", float) if scaling else 1.0, softcap=_take(m, "softcap", float, 0.0),
+                window=window, keep_first=_take(mask, "keep_first", int, 0))
+        _positive(s, ("heads", "kv_heads", "dim", "vdim", "scale", "rot_base", "rot_factor"), where)
+        if s.heads % s.kv_heads:
+            raise ConfigError(f"config.json: {where}heads {s.heads} must be a multiple of kv_heads {s.kv_heads}")
+        if s.rot_dims <= 0 or s.rot_dims % 2 or s.rot_dims > s.dim:
+            raise ConfigError(f"config.json: {where}rot.dims {s.rot_dims} must be even and at most dim {s.dim}")
+        if s.softcap < 0 or s.keep_first < 0 or (s.window is not None and s.window <= 0):
+            raise ConfigError(f"config.json: {where}mask.size must be positive, softcap and mask.keep_first not negative")
+        return s
+
+    def to_dict(self) -> Dict[str, Any]:
+        rot = {"base": self.rot_base, "dims": self.rot_dims}
+        if self.rot_factor != 1.0:
+            rot["scaling"] = {"factor": self.rot_factor}
+        d = {"heads": self.heads, "kv_heads": self.kv_heads, "dim": self.dim, "vdim": self.vdim, "scale": self.scale, "rot": rot}
+        if self.softcap:
+            d["softcap"] = self.softcap
+        if self.window is not None:
+            d["mask"] = {"size": self.window, "keep_first": self.keep_first}
+        return d
+
+
+@dataclass(frozen=True)
+class StateSpaceSizes:
+    """The right half of a ``parallel`` mixer of Rorutar: ``heads`` states of ``state`` x ``vdim``, ``groups`` of heads that
+    share what is written and read, ``conv`` taps, an output norm in ``norm_groups`` equal parts."""
+    heads: int
+    vdim: int
+    state: int
+    groups: int
+    conv: int
+    norm_groups: int
+
+    @classmethod
+    def from_dict(cls, m: Dict[str, Any], where: str) -> "StateSpaceSizes":
+        s = cls(heads=_take(m, "heads", int), vdim=_take(m, "vdim", int), state=_take(m, "state", int),
+                groups=_take(m, "groups", int, 1), conv=_take(m, "conv", int), norm_groups=_take(m, "norm_groups", int, 1))
+        _positive(s, ("heads", "vdim", "state", "groups", "conv", "norm_groups"), where)
+        if s.heads % s.groups:
+            raise ConfigError(f"config.json: {where}heads {s.heads} must be a multiple of groups {s.groups}")
+        if (s.heads * s.vdim) % s.norm_groups:
+            raise ConfigError(f"config.json: {where}norm_groups {s.norm_groups} must divide heads * vdim {s.heads * s.vdim}")
+        return s
+
+    def to_dict(self) -> Dict[str, Any]:
+        return {"heads": self.heads, "vdim": self.vdim, "state": self.state, "groups": self.groups, "conv": self.conv,
+                "norm_groups": self.norm_groups}
+
+
+@dataclass(frozen=True)
+class ParallelSizes:
+    """A ``parallel`` mixer of Rorutar: ``left_scale * left + right_scale * right``."""
+    left: KeptWindowAttentionSizes
+    right: StateSpaceSizes
+    left_scale: float
+    right_scale: float
+
+    @classmethod
+    def from_dict(cls, m: Dict[str, Any], where: str) -> "ParallelSizes":
+        return cls(left=KeptWindowAttentionSizes.from_dict(_section(m, "left", where), where + "left: "),
+                   right=StateSpaceSizes.from_dict(_section(m, "right", where), where + "right: "),
+                   left_scale=_take(m, "left_scale", float, 1.0), right_scale=_take(m, "right_scale", float, 1.0))
+
+    def to_dict(self) -> Dict[str, Any]:
+        return {"left": self.left.to_dict(), "right": self.right.to_dict(), "left_scale": self.left_scale,
+                "right_scale": self.right_scale}
+
+
+@dataclass(frozen=True)
+class ClampedExpertSizes:
+    """A ``moe`` feed-forward of Rorutar: ``experts`` gated experts ``ff`` wide, gate and up sides clamped at ``limit``, of
+    which a token uses ``top`` out of the ``keep`` best of ``groups`` groups."""
+    ff: int
+    limit: float
+    experts: int
+    top: int
+    groups: int = 1
+    keep: int = 1
+    kind: str = "moe"
+
+    @classmethod
+    def from_dict(cls, m: Dict[str, Any], where: str) -> "ClampedExpertSizes":
+        if m.get("kind", "moe") != "moe":
+            raise ConfigError(f"config.json: {where}mlp.kind {m.get('kind')!r}: the design's feed-forward is a mixture of experts")
+        expert, router = _section(m, "expert", where), _section(m, "router", where)
+        groups = _section(router, "groups", where, optional=True)
+        s = cls(ff=_take(expert, "ff", int), limit=_take(expert, "limit", float), experts=_take(router, "experts", int),
+                top=_take(router, "top", int), groups=_take(groups, "count", int) if groups else 1,
+                keep=_take(groups, "keep", int) if groups else 1)
+        _positive(s, ("ff", "limit", "experts", "top", "groups", "keep"), where)
+        if s.experts % s.groups or s.keep > s.groups:
+            raise ConfigError(f"config.json: {where}router.groups: {s.groups} must divide the {s.experts} experts and keep "
+                              f"{s.keep} be at most as many")
+        if s.top > s.keep * (s.experts // s.groups):
+            raise ConfigError(f"config.json: {where}router.top {s.top} is more than the kept groups hold")
+        return s
+
+    def to_dict(self) -> Dict[str, Any]:
+        return {"kind": "moe", "expert": {"ff": self.ff, "limit": self.limit},
+                "router": {"experts": self.experts, "top": self.top, "groups": {"count": self.groups, "keep": self.keep}}}
+
+
+@dataclass(frozen=True)
+class RorutarLayer:
+    type: str
+    mixer: ParallelSizes
+    mlp: Optional[ClampedExpertSizes]
+
+
+@dataclass(frozen=True)
+class RorutarConfig:
+    """``config.json`` of a Rorutar model: ``vocab``, ``width``, ``norm.eps``, ``embedding.scale``, ``loop`` (layers that run
+    several times) and the list ``layers``, each entry with its ``type`` (``parallel``), the mixer's sizes and its
+    feed-forward (``mlp``: a mixture of experts, or null).  ``max_positions`` is optional: the design has no longest
+    sequence of its own."""
+    vocab: int
+    width: int
+    norm_eps: float
+    layers: Tuple[RorutarLayer, ...]
+    embedding_scale: float = 1.0
+    loop: Optional[LayerLoop] = None
+    max_positions: int = 1 << 20
+    eos_token_ids: Tuple[int, ...] = ()
+    architecture: str = "Rorutar"
+
+    MIXER_TYPES = {"parallel": ParallelSizes}
+
+    @classmethod
+    def from_dict(cls, d: Dict[str, Any]) -> "RorutarConfig":
+        raw = d.get("layers")
+        if not isinstance(raw, list) or not raw:
+            raise ConfigError("config.json: 'layers' must be a non-empty list")
+        layers = []
+        for i, l in enumerate(raw):
+            where = f"layers[{i}]: "
+            if not isinstance(l, dict):
+                raise ConfigError(f"config.json: {where}must be an object")
+            kind = _take(l, "type", str)
+            if kind not in cls.MIXER_TYPES:
+                raise ConfigError(f"config.json: {where}unknown type {kind!r} ({', '.join(cls.MIXER_TYPES)})")
+            mixer = cls.MIXER_TYPES[kind].from_dict(_section(l, "mixer", where), where)
+            mlp = _section(l, "mlp", where, optional=True)
+            layers.append(RorutarLayer(kind, mixer, ClampedExpertSizes.from_dict(mlp, where) if mlp else None))
+        emb = _section(d, "embedding", "", optional=True) or {}
+        lp = _section(d, "loop", "", optional=True)
+        loop = LayerLoop(*(_take(lp, k, int) for k in ("start", "stop", "times"))) if lp else None
+        if loop is not None and not (0 <= loop.start < loop.stop <= len(layers) and loop.times >= 1):
+            raise ConfigError(f"config.json: loop: layers {loop.start} to {loop.stop} of {len(layers)}, {loop.times} times")
+        eos = d.get("eos_token_id")
+        eos_ids = (eos,) if isinstance(eos, int) and not isinstance(eos, bool) else \
+            tuple(int(x) for x in eos) if isinstance(eos, (list, tuple)) else ()
+        cfg = cls(vocab=_take(d, "vocab", int), width=_take(d, "width", int),
+                  norm_eps=_take(_section(d, "norm", ""), "eps", float), layers=tuple(layers),
+                  embedding_scale=_take(emb, "scale", float, 1.0), loop=loop,
+                  max_positions=_take(d, "max_positions", int, 1 << 20), eos_token_ids=eos_ids,
+                  architecture=str(d.get("architecture") or (d.get("architectures") or ["Rorutar"])[0]))
+        if cfg.vocab <= 0 or cfg.width <= 0 or cfg.max_positions <= 1:
+            raise ConfigError("config.json: vocab, width and max_positions must be positive")
+        if not cfg.norm_eps > 0:
+            raise ConfigError(f"config.json: norm.eps must be positive, got {cfg.norm_eps}")
+        return cfg
+
+    def schedule(self) -> Tuple[int, ...]:
+        """The layers in the order in which they run."""
+        n = len(self.layers)
+        if self.loop is None:
+            return tuple(range(n))
+        lp = self.loop
+        return tuple(range(lp.start)) + tuple(range(lp.start, lp.stop)) * lp.times + tuple(range(lp.stop, n))
+
+    def to_dict(self) -> Dict[str, Any]:
+        d = {"architecture": self.architecture, "vocab": self.vocab, "width": self.width, "norm": {"eps": self.norm_eps},
+             "embedding": {"scale": self.embedding_scale},
+             "layers": [{"type": l.type, "mixer": l.mixer.to_dict(), "mlp": None if l.mlp is None else l.mlp.to_dict()}
+                        for l in self.layers]}
+        if self.loop is not None:
+            d["loop"] = {"start": self.loop.start, "stop": self.loop.stop, "times": self.loop.times}
+        if self.max_positions != 1 << 20:
+            d["max_positions"] = self.max_positions
+        if self.eos_token_ids:
+            d["eos_token_id"] = list(self.eos_token_ids)
+        return d

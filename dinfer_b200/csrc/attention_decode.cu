@@ -40,6 +40,8 @@ struct Params {
   int H, Hkv, group, block_size, bs_log2, window, chunked;
   int sink;          // one more softmax term without a value, of score sinks[head] (null: 0) (the TMA variant)
   const float* sinks;
+  int keep;          // with a window: the keys below it are seen too (the TMA variant)
+  float cap_in, cap_out;   // a soft cap on the scores, see softcap_log2 (the TMA variant with CAP)
   float scale_log2;
   const float* slopes;   // [H] or null: a distance bias, score - slopes[h] * (i - j) (the TMA variant)
   int splits;
@@ -435,7 +437,7 @@ __device__ __forceinline__ uint32_t sw128(int row, int c) {
   return (uint32_t)((c >> 3) * (BN * 128) + row * 128 + (((c & 7) ^ (row & 7)) << 4));
 }
 
-template <int D, int NH8>
+template <int D, int NH8, bool CAP>
 __global__ void __launch_bounds__(NT_TMA, 2)
 attention_decode_tma_kernel(const __grid_constant__ CUtensorMap map_kv, const Params p) {
   constexpr int NHF = D / 64;                                 // 64-wide halves of the head
@@ -458,18 +460,17 @@ attention_decode_tma_kernel(const __grid_constant__ CUtensorMap map_kv, const Pa
   const int pos = seq_len - 1;
   const int lo = first_key(pos, p.window, p.chunked), hi = seq_len;
   const int* table = p.block_table + (int64_t)b * p.max_blocks;
-  int tile_begin = lo / BN, tile_end = (hi + BN - 1) / BN;
-  {
-    const int per = (tile_end - tile_begin + p.splits - 1) / p.splits;
-    tile_begin += split * per;
-    tile_end = min(tile_end, tile_begin + per);
-  }
-  const int n_tiles = max(0, tile_end - tile_begin);
+  // the visits: kept tiles in front of the window, then the window's; this CTA's run of them starts at visit v0
+  const int tile_first = lo / BN, kept = kept_tiles(p.keep, BN, tile_first);
+  const int visits = kept + (hi + BN - 1) / BN - tile_first;
+  const int per = (visits + p.splits - 1) / p.splits;
+  const int v0 = split * per, n_tiles = max(0, min(per, visits - v0));
   const uint32_t base = (smem_u32(smem_raw) + 1023u) & ~1023u;
   unsigned char* gbase = smem_raw + (base - smem_u32(smem_raw));
-  const int table_first = (tile_begin * BN) >> p.bs_log2;
+  // page-table entries of this CTA's part of the window (those of kept tiles are read as they come)
+  const int table_first = (tile_of(max(v0, kept), kept, tile_first) * BN) >> p.bs_log2;
   {
-    const int last = (min(tile_end * BN, hi) - 1) >> p.bs_log2;
+    const int last = (min(tile_of(max(v0 + n_tiles, kept), kept, tile_first) * BN, hi) - 1) >> p.bs_log2;
     for (int i = threadIdx.x; i < TABLE_SLOTS && table_first + i <= last; i += NT_TMA) s_table[i] = table[table_first + i];
     // a page that is skipped leaves its rows as they were: they must hold finite numbers (0 * V)
     uint4* z = reinterpret_cast<uint4*>(gbase);
@@ -503,7 +504,7 @@ attention_decode_tma_kernel(const __grid_constant__ CUtensorMap map_kv, const Pa
     bool waited = false, alive = true;
     for (int t = 0; t < n_tiles && alive; ++t) {
       const int s = t % STAGES;
-      const int j0 = (tile_begin + t) * BN;
+      const int j0 = tile_of(v0 + t, kept, tile_first) * BN;
       if (!waited && j0 + BN > pos) { pdl_wait(); waited = true; }        // the newest token's page
       bool ok = true;
       if (lane == 0) ok = mbar_wait(smem_u32(&empty_bar[s]), ((t / STAGES) & 1) ^ 1);
@@ -520,9 +521,9 @@ attention_decode_tma_kernel(const __grid_constant__ CUtensorMap map_kv, const Pa
         if (o < n_ops) {
           const int x = o / PER_BOX, r = o % PER_BOX, kv = r / NHF, h = r % NHF;
           const int key = j0 + x * br;
-          if (key < hi && key + br > lo) {
+          if (key < hi && (key + br > lo || key < p.keep)) {
             const int e = (key >> p.bs_log2) - table_first;
-            const int blk = e < TABLE_SLOTS ? s_table[e] : table[key >> p.bs_log2];
+            const int blk = e >= 0 && e < TABLE_SLOTS ? s_table[e] : table[key >> p.bs_log2];
             if (blk >= 0) {
               valid[u] = true;
               row[u] = ((blk * 2 + kv) * p.Hkv + hk) * p.block_size + (key & (p.block_size - 1));
@@ -571,7 +572,7 @@ attention_decode_tma_kernel(const __grid_constant__ CUtensorMap map_kv, const Pa
       if (!mbar_wait(smem_u32(&full_bar[s]), (t / STAGES) & 1)) { s_abort = 1; atomicExch(p.status, 22); ok = false; break; }
       const unsigned char* kt = gbase + s * 2 * KV_BYTES;
       const unsigned char* vt = kt + KV_BYTES;
-      const int jbase = (tile_begin + t) * BN + key_off;
+      const int jbase = tile_of(v0 + t, kept, tile_first) * BN + key_off;
       if (jbase < hi) {
         float st[NH8][4], st2[NH8][4];
 #pragma unroll
@@ -594,8 +595,8 @@ attention_decode_tma_kernel(const __grid_constant__ CUtensorMap map_kv, const Pa
         for (int nt = 0; nt < NH8; ++nt) {
           st[nt][0] += st2[nt][0]; st[nt][1] += st2[nt][1]; st[nt][2] += st2[nt][2]; st[nt][3] += st2[nt][3];
         }
-        const bool vis0 = jbase + g >= lo && jbase + g <= pos;
-        const bool vis1 = jbase + g + 8 >= lo && jbase + g + 8 <= pos;
+        const bool vis0 = (jbase + g >= lo || jbase + g < p.keep) && jbase + g <= pos;
+        const bool vis1 = (jbase + g + 8 >= lo || jbase + g + 8 < p.keep) && jbase + g + 8 <= pos;
         bool rescale = false;
         float alpha[NH8][2];
         unsigned pb[NH8][2];
@@ -603,6 +604,10 @@ attention_decode_tma_kernel(const __grid_constant__ CUtensorMap map_kv, const Pa
         for (int nt = 0; nt < NH8; ++nt) {
 #pragma unroll
           for (int c = 0; c < 2; ++c) {
+            if (CAP) {
+              st[nt][c] = softcap_log2(st[nt][c], p.cap_in, p.cap_out);
+              st[nt][c + 2] = softcap_log2(st[nt][c + 2], p.cap_in, p.cap_out);
+            }
             const float s0 = vis0 ? fmaf(st[nt][c], p.scale_log2, -sl[nt][c] * (float)(pos - jbase - g)) : -INFINITY;
             const float s1 = vis1 ? fmaf(st[nt][c + 2], p.scale_log2, -sl[nt][c] * (float)(pos - jbase - g - 8)) : -INFINITY;
             float mx = fmaxf(s0, s1);
@@ -747,9 +752,9 @@ EncodeTiledFn encode_fn() {
   return fn;
 }
 
-template <int D, int NH8>
+template <int D, int NH8, bool CAP>
 int launch_tma(const CUtensorMap& map, const Params& p, int B, cudaStream_t stream) {
-  auto k = attention_decode_tma_kernel<D, NH8>;
+  auto k = attention_decode_tma_kernel<D, NH8, CAP>;
   // tiles (the four warps' fold reuses them: it is smaller), then the cluster's receive buffer
   static_assert((size_t)(4 * NH8 * 8 * D + 2 * 4 * NH8 * 8) * sizeof(float) <= (size_t)2 * STAGES * (D / 64) * BN * 128,
                 "the fold of the four warps fits the tiles");
@@ -848,7 +853,7 @@ DINFER_API int dinfer_attention_decode(const void* q, int64_t ldq, void* out, in
   p.cu_seqlens = cu_seqlens; p.seq_lens = seq_lens; p.H = H; p.Hkv = Hkv; p.group = H / Hkv;
   p.block_size = block_size; p.bs_log2 = 0;
   while ((1 << p.bs_log2) < block_size) ++p.bs_log2;
-  p.window = window; p.chunked = 0; p.sink = 0; p.sinks = nullptr; p.scale_log2 = scale * 1.4426950408889634f; p.splits = splits;
+  p.window = window; p.chunked = 0; p.keep = 0; p.cap_in = p.cap_out = 0.f; p.sink = 0; p.sinks = nullptr; p.scale_log2 = scale * 1.4426950408889634f; p.splits = splits;
   p.slopes = nullptr;
   p.part_o = scratch_floats;
   p.part_ml = scratch_floats ? scratch_floats + (int64_t)B * H * splits * D : nullptr;
@@ -861,13 +866,14 @@ DINFER_API int dinfer_attention_decode(const void* q, int64_t ldq, void* out, in
 // The TMA variant (pages of at least 8 tokens): no scratch (the splits fold inside a cluster, at most
 // 16 of them), plus the number of pages of the cache tensor (for the tensor map) and the device status
 // word that a bounded wait sets when it runs out.
-// chunked: window is the size of the chunks (see first_key).
+// chunked: window is the size of the chunks (see first_key).  keep_first: with a window, the keys below it are seen too.
+// softcap > 0: a score is softcap * tanh(score / softcap), ahead of the bias.
 // sink != 0: the softmax has one more term that carries no value, of score sinks[h] (f32 [H]; null: 0).
 // slopes: f32 [H] or null; with them score_ij - slopes[h] * (i - j).
 DINFER_API int dinfer_attention_decode_tma_bias(const void* q, int64_t ldq, void* out, int64_t ldo, const void* cache,
                                                 int64_t num_blocks, const int* block_table, int max_blocks,
                                                 const int* cu_seqlens, const int* seq_lens, int B, int H, int Hkv, int D,
-                                                int block_size, float scale, int window, int chunked, int sink, const float* sinks, const float* slopes,
+                                                int block_size, float scale, int window, int chunked, int keep_first, float softcap, int sink, const float* sinks, const float* slopes,
                                                 int splits, int* status, cudaStream_t stream);
 
 DINFER_API int dinfer_attention_decode_tma_sink(const void* q, int64_t ldq, void* out, int64_t ldo, const void* cache,
@@ -876,16 +882,18 @@ DINFER_API int dinfer_attention_decode_tma_sink(const void* q, int64_t ldq, void
                                                 int block_size, float scale, int window, int sink, int splits,
                                                 int* status, cudaStream_t stream) {
   return dinfer_attention_decode_tma_bias(q, ldq, out, ldo, cache, num_blocks, block_table, max_blocks, cu_seqlens, seq_lens,
-                                          B, H, Hkv, D, block_size, scale, window, 0, sink, nullptr, nullptr, splits, status, stream);
+                                          B, H, Hkv, D, block_size, scale, window, 0, 0, 0.f, sink, nullptr, nullptr, splits, status, stream);
 }
 
 DINFER_API int dinfer_attention_decode_tma_bias(const void* q, int64_t ldq, void* out, int64_t ldo, const void* cache,
                                                 int64_t num_blocks, const int* block_table, int max_blocks,
                                                 const int* cu_seqlens, const int* seq_lens, int B, int H, int Hkv, int D,
-                                                int block_size, float scale, int window, int chunked, int sink, const float* sinks, const float* slopes,
+                                                int block_size, float scale, int window, int chunked, int keep_first, float softcap, int sink, const float* sinks, const float* slopes,
                                                 int splits, int* status, cudaStream_t stream) {
   if (B <= 0 || H <= 0 || Hkv <= 0 || H % Hkv || max_blocks <= 0 || num_blocks <= 0)
     return refuse(DINFER_BAD_ARGUMENT, "attention_decode_tma: bad sizes B=%d H=%d Hkv=%d", B, H, Hkv);
+  if (keep_first < 0 || (keep_first > 0 && chunked) || !(softcap >= 0.f))
+    return refuse(DINFER_BAD_ARGUMENT, "attention_decode_tma: keep_first %d, softcap %g (kept keys belong to a window)", keep_first, (double)softcap);
   if (!dinfer_attention_decode_supports(D, H / Hkv, block_size) || block_size < 8)
     return refuse(DINFER_BAD_ARGUMENT, "attention_decode_tma: head_dim %d, group %d, block_size %d not supported "
                   "(head_dim 64 or 128, group <= 16, power-of-two pages of at least 8)", D, H / Hkv, block_size);
@@ -918,11 +926,18 @@ DINFER_API int dinfer_attention_decode_tma_bias(const void* q, int64_t ldq, void
   p.block_size = block_size; p.bs_log2 = 0;
   while ((1 << p.bs_log2) < block_size) ++p.bs_log2;
   p.window = window; p.chunked = chunked; p.sink = sink; p.sinks = sinks; p.scale_log2 = scale * 1.4426950408889634f; p.splits = splits;
+  p.keep = window > 0 ? keep_first : 0;
+  p.cap_in = p.cap_out = 0.f;
+  if (softcap > 0.f) {                          // the capped scores come out in log2 units
+    p.cap_in = 2.f * p.scale_log2 / softcap; p.cap_out = softcap * 1.4426950408889634f; p.scale_log2 = 1.f;
+  }
   p.slopes = slopes;
   p.part_o = nullptr; p.part_ml = nullptr; p.counters = nullptr; p.status = status;
   const int nh8 = (p.group + 7) / 8;
-  if (D == 64) return nh8 == 1 ? launch_tma<64, 1>(map, p, B, stream) : launch_tma<64, 2>(map, p, B, stream);
-  return nh8 == 1 ? launch_tma<128, 1>(map, p, B, stream) : launch_tma<128, 2>(map, p, B, stream);
+#define GO(CAP) (D == 64 ? (nh8 == 1 ? launch_tma<64, 1, CAP>(map, p, B, stream) : launch_tma<64, 2, CAP>(map, p, B, stream)) \
+                         : (nh8 == 1 ? launch_tma<128, 1, CAP>(map, p, B, stream) : launch_tma<128, 2, CAP>(map, p, B, stream)))
+  return softcap > 0.f ? GO(true) : GO(false);
+#undef GO
 }
 
 DINFER_API int dinfer_attention_decode_tma(const void* q, int64_t ldq, void* out, int64_t ldo, const void* cache,

@@ -8,7 +8,8 @@
 // of its own request (`chunked`: those of its own chunk of `window` positions), read through the request's block table.  Values may be Dv wide where keys are D wide (the
 // cache's rows are then Dc = max(D, Dv) wide); with `sink` the softmax has one more term of score 0 and no value:
 // p_j = exp(s_j) / (1 + sum exp(s_j)); `sinks` gives that term a score of its own per query head.  With `slopes` (one number per query head) a distance bias is taken off every
-// score: s_ij - slopes[h] * (i - j).
+// score: s_ij - slopes[h] * (i - j).  `keep`: behind a window the keys below it are seen too.  `softcap` > 0: a score is
+// softcap * tanh(score / softcap), ahead of the bias.
 //
 // Counterpart in the reference: the any-D reference kernels crates/kernels/cuda/gqa.cu:956-1118.
 #include "common.cuh"
@@ -26,7 +27,8 @@ attention_generic_kernel(const T* __restrict__ q, int64_t ldq, T* __restrict__ o
                          const T* __restrict__ cache, const int* __restrict__ block_table, int max_blocks,
                          const int* __restrict__ cu_seqlens, const int* __restrict__ positions,
                          int num_reqs, int H, int Hkv, int D, int Dv, int Dc, int block_size, float scale, int window,
-                         int chunked, int sink, const float* __restrict__ sinks, const float* __restrict__ slopes) {
+                         int chunked, int keep, float softcap, int sink, const float* __restrict__ sinks,
+                         const float* __restrict__ slopes) {
   const int t = blockIdx.x;
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   const int h = blockIdx.y * WARPS + warp;
@@ -52,12 +54,14 @@ attention_generic_kernel(const T* __restrict__ q, int64_t ldq, T* __restrict__ o
   }
   float m = -INFINITY, l = 0.f;
   const int64_t plane = (int64_t)Hkv * block_size * Dc;      // one of k / v of one block
-  for (int j0 = first; j0 <= pos; j0 += KEYS) {
+  const int kept = min(keep, first);                           // the kept keys in front of the window, then the window
+  const int visits = kept + pos - first + 1;
+  for (int n0 = 0; n0 < visits; n0 += KEYS) {
     const T* kp[KEYS];
     float s[KEYS];
 #pragma unroll
     for (int u = 0; u < KEYS; ++u) {
-      const int j = j0 + u;
+      const int j = n0 + u < kept ? n0 + u : first + n0 + u - kept;
       kp[u] = nullptr;
       s[u] = 0.f;
       // a page the table does not hold (-1: a dummy row of a captured graph, a page a window has passed) is no key
@@ -72,7 +76,13 @@ attention_generic_kernel(const T* __restrict__ q, int64_t ldq, T* __restrict__ o
       }
     }
 #pragma unroll
-    for (int u = 0; u < KEYS; ++u) s[u] = kp[u] ? warp_sum(s[u]) - slope * (float)(pos - (j0 + u)) : -INFINITY;
+    for (int u = 0; u < KEYS; ++u) {
+      const int j = n0 + u < kept ? n0 + u : first + n0 + u - kept;
+      if (!kp[u]) { s[u] = -INFINITY; continue; }
+      s[u] = warp_sum(s[u]);
+      if (softcap > 0.f) s[u] = softcap * tanhf(s[u] / softcap);
+      s[u] -= slope * (float)(pos - j);
+    }
     float m_new = m;
 #pragma unroll
     for (int u = 0; u < KEYS; ++u) m_new = fmaxf(m_new, s[u]);
@@ -115,12 +125,12 @@ attention_generic_kernel(const T* __restrict__ q, int64_t ldq, T* __restrict__ o
 template <typename T, int C>
 int launch(const void* q, int64_t ldq, void* out, int64_t ldo, const void* cache, const int* block_table,
            int max_blocks, const int* cu_seqlens, const int* positions, int T_, int B, int H, int Hkv,
-           int D, int Dv, int Dc, int block_size, float scale, int window, int chunked, int sink, const float* sinks, const float* slopes,
-           cudaStream_t stream) {
+           int D, int Dv, int Dc, int block_size, float scale, int window, int chunked, int keep, float softcap, int sink,
+           const float* sinks, const float* slopes, cudaStream_t stream) {
   dim3 grid(T_, (H + WARPS - 1) / WARPS);
   attention_generic_kernel<T, C><<<grid, WARPS * 32, 0, stream>>>(
       (const T*)q, ldq, (T*)out, ldo, (const T*)cache, block_table, max_blocks, cu_seqlens, positions,
-      B, H, Hkv, D, Dv, Dc, block_size, scale, window, chunked, sink, sinks, slopes);
+      B, H, Hkv, D, Dv, Dc, block_size, scale, window, chunked, keep, softcap, sink, sinks, slopes);
   return cuda_status("attention_generic");
 }
 
@@ -131,8 +141,8 @@ DINFER_DEFINE_LAST_ERROR()
 DINFER_API int dinfer_attention_generic_bias(const void* q, int64_t ldq, void* out, int64_t ldo, const void* cache,
                                              const int* block_table, int max_blocks, const int* cu_seqlens,
                                              const int* positions, int T, int B, int H, int Hkv, int D, int Dv, int Dc,
-                                             int block_size, float scale, int window, int chunked, int sink, const float* sinks,
-                                             const float* slopes, int dtype, cudaStream_t stream);
+                                             int block_size, float scale, int window, int chunked, int keep_first, float softcap,
+                                             int sink, const float* sinks, const float* slopes, int dtype, cudaStream_t stream);
 
 // q: [T, ...] rows of stride ldq, head h at h*D; out likewise with stride ldo.
 // cache [num_blocks, 2, Hkv, block_size, D]; block_table [B, max_blocks] int32;
@@ -144,7 +154,7 @@ DINFER_API int dinfer_attention_generic(const void* q, int64_t ldq, void* out, i
                                         int block_size, float scale, int window, int dtype,
                                         cudaStream_t stream) {
   return dinfer_attention_generic_bias(q, ldq, out, ldo, cache, block_table, max_blocks, cu_seqlens, positions, T, B, H,
-                                       Hkv, D, D, D, block_size, scale, window, 0, 0, nullptr, nullptr, dtype, stream);
+                                       Hkv, D, D, D, block_size, scale, window, 0, 0, 0.f, 0, nullptr, nullptr, dtype, stream);
 }
 
 // The same with values Dv wide in a cache whose rows are Dc wide (out: head h at h*Dv), and an optional sink.
@@ -154,16 +164,20 @@ DINFER_API int dinfer_attention_generic_ex(const void* q, int64_t ldq, void* out
                                            int block_size, float scale, int window, int sink, int dtype,
                                            cudaStream_t stream) {
   return dinfer_attention_generic_bias(q, ldq, out, ldo, cache, block_table, max_blocks, cu_seqlens, positions, T, B, H,
-                                       Hkv, D, Dv, Dc, block_size, scale, window, 0, sink, nullptr, nullptr, dtype, stream);
+                                       Hkv, D, Dv, Dc, block_size, scale, window, 0, 0, 0.f, sink, nullptr, nullptr, dtype, stream);
 }
 
-// The same with a distance bias (slopes [H] f32 or null), keys by chunks (chunked, see first_key) and a score per head
+// The same with a distance bias (slopes [H] f32 or null), keys by chunks (chunked, see first_key), kept first keys
+// (keep_first > 0, with a window), a soft cap on the scores (softcap > 0) and a score per head
 // for the sink's term (sinks [H] f32 or null: 0).
 DINFER_API int dinfer_attention_generic_bias(const void* q, int64_t ldq, void* out, int64_t ldo, const void* cache,
                                              const int* block_table, int max_blocks, const int* cu_seqlens,
                                              const int* positions, int T, int B, int H, int Hkv, int D, int Dv, int Dc,
-                                             int block_size, float scale, int window, int chunked, int sink, const float* sinks,
-                                             const float* slopes, int dtype, cudaStream_t stream) {
+                                             int block_size, float scale, int window, int chunked, int keep_first, float softcap,
+                                             int sink, const float* sinks, const float* slopes, int dtype, cudaStream_t stream) {
+  if (keep_first < 0 || !(softcap >= 0.f) || (keep_first > 0 && chunked))
+    return refuse(DINFER_BAD_ARGUMENT, "attention_generic: keep_first %d, softcap %g (kept keys belong to a window)", keep_first, (double)softcap);
+  const int keep = window > 0 ? keep_first : 0;
   if (Dv <= 0 || Dc < D || Dc < Dv) return refuse(DINFER_BAD_ARGUMENT, "attention_generic: bad sizes D=%d Dv=%d Dc=%d", D, Dv, Dc);
   if (T < 0 || B <= 0 || H <= 0 || Hkv <= 0 || D <= 0 || block_size <= 0 || max_blocks <= 0)
     return refuse(DINFER_BAD_ARGUMENT, "attention_generic: bad sizes T=%d B=%d H=%d Hkv=%d D=%d block=%d",
@@ -174,7 +188,7 @@ DINFER_API int dinfer_attention_generic_bias(const void* q, int64_t ldq, void* o
   if (T == 0) return 0;
   const int c = ((D > Dv ? D : Dv) + 31) / 32;
 #define GO(C) return launch<T_, C>(q, ldq, out, ldo, cache, block_table, max_blocks, cu_seqlens, positions, \
-                                   T, B, H, Hkv, D, Dv, Dc, block_size, scale, window, chunked, sink, sinks, slopes, stream)
+                                   T, B, H, Hkv, D, Dv, Dc, block_size, scale, window, chunked, keep, softcap, sink, sinks, slopes, stream)
   DINFER_DISPATCH_DTYPE(dtype, T_, {
     if (c <= 1) GO(1);
     else if (c <= 2) GO(2);

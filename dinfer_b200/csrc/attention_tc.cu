@@ -40,6 +40,8 @@ struct Params {
   int H, Hkv, group, block_size, window, chunked;
   int sink;                    // one more softmax term without a value, of score sinks[head] (null: 0)
   const float* sinks;
+  int keep;                    // with a window: the keys below it are seen too
+  float cap_in, cap_out;       // a soft cap on the scores (CAP), see softcap_log2
   float scale_log2;            // scale * log2(e)
   const float* slopes;         // [H] or null: a distance bias, score - slopes[h] * (i - j)
   int splits;                  // decode shape only
@@ -95,11 +97,11 @@ __device__ __forceinline__ void load_kv_tile(const Params& p, const int* table, 
   for (int r0 = 0; r0 < BN; r0 += ROWS) {
     const int row = r0 + threadIdx.x / C;
     const int j = j0 + row;
-    bool ok = j >= lo && j < hi;
+    bool ok = (j >= lo || j < p.keep) && j < hi;
     int blk = 0;
     if (ok) {      // the CTA's slice of the page table sits in shared memory (no dependent global read per tile)
       const int e = j / p.block_size - table_first;
-      blk = e < TABLE_SLOTS ? s_table[e] : table[j / p.block_size];
+      blk = e >= 0 && e < TABLE_SLOTS ? s_table[e] : table[j / p.block_size];
       ok = blk >= 0;
     }
     const __nv_bfloat16* src = p.cache;
@@ -137,18 +139,18 @@ __global__ void __launch_bounds__(DECODE ? NT_DECODE : NT_PROMPT, 2) attention_t
   const int first_tok = row0 / p.group, last_tok = last_row / p.group;
   int hi = hist + last_tok + 1;
   int lo = first_key(hist + first_tok, p.window, p.chunked);
-  int tile_begin = lo / BN, tile_end = (hi + BN - 1) / BN;
+  // the visits: tiles with kept keys in front of the window, then the window's tiles (see tile_of)
+  const int tile_first = lo / BN, kept = kept_tiles(p.keep, BN, tile_first);
+  int v0 = 0, n_tiles = kept + (hi + BN - 1) / BN - tile_first;
   if (DECODE) {
-    const int n = tile_end - tile_begin;
-    const int per = (n + p.splits - 1) / p.splits;
-    tile_begin = tile_begin + blockIdx.x * per;
-    tile_end = min(tile_end, tile_begin + per);
+    const int per = (n_tiles + p.splits - 1) / p.splits;
+    v0 = blockIdx.x * per;
+    n_tiles = max(0, min(per, n_tiles - v0));
   }
-  const int n_tiles = max(0, tile_end - tile_begin);
   __shared__ int s_table[TABLE_SLOTS];
-  const int table_first = (tile_begin * BN) / p.block_size;
+  const int table_first = (tile_of(max(v0, kept), kept, tile_first) * BN) / p.block_size;   // (kept tiles' entries are read as they come)
   {
-    const int last = (min(tile_end * BN, hi) - 1) / p.block_size;
+    const int last = (min(tile_of(max(v0 + n_tiles, kept), kept, tile_first) * BN, hi) - 1) / p.block_size;
     for (int i = threadIdx.x; i < TABLE_SLOTS && table_first + i <= last; i += NT) s_table[i] = table[table_first + i];
     __syncthreads();
   }
@@ -167,7 +169,7 @@ __global__ void __launch_bounds__(DECODE ? NT_DECODE : NT_PROMPT, 2) attention_t
   }
 #pragma unroll
   for (int i = 0; i < STAGES - 1; ++i) {      // Q rides in the first group
-    if (i < n_tiles) load_kv_tile<D, NT>(p, table, s_table, table_first, hk, (tile_begin + i) * BN, lo, hi, sK + i * BN * D, sV + i * BN * D);
+    if (i < n_tiles) load_kv_tile<D, NT>(p, table, s_table, table_first, hk, tile_of(v0 + i, kept, tile_first) * BN, lo, hi, sK + i * BN * D, sV + i * BN * D);
     cp_async_commit();
   }
 
@@ -201,7 +203,7 @@ __global__ void __launch_bounds__(DECODE ? NT_DECODE : NT_PROMPT, 2) attention_t
   for (int t = 0; t < n_tiles; ++t) {
     const int buf = t % STAGES;
     if (t + STAGES - 1 < n_tiles)
-      load_kv_tile<D, NT>(p, table, s_table, table_first, hk, (tile_begin + t + STAGES - 1) * BN, lo, hi,
+      load_kv_tile<D, NT>(p, table, s_table, table_first, hk, tile_of(v0 + t + STAGES - 1, kept, tile_first) * BN, lo, hi,
                           sK + ((t + STAGES - 1) % STAGES) * BN * D, sV + ((t + STAGES - 1) % STAGES) * BN * D);
     cp_async_commit();
     cp_async_wait<STAGES - 1>();
@@ -235,18 +237,18 @@ __global__ void __launch_bounds__(DECODE ? NT_DECODE : NT_PROMPT, 2) attention_t
       }
     }
     // scale into the exp2 domain and mask by position
-    const int jbase = (tile_begin + t) * BN + key_off;
+    const int jbase = tile_of(v0 + t, kept, tile_first) * BN + key_off;
     const bool need_mask = (jbase + NK - 1 > hist + first_tok) || (p.window > 0) || (jbase < lo) || DECODE;
 #pragma unroll
     for (int i = 0; i < NK / 8; ++i) {
 #pragma unroll
       for (int e = 0; e < 4; ++e) {
-        float v = s[i][e] * p.scale_log2;
+        float v = p.cap_out > 0.f ? softcap_log2(s[i][e], p.cap_in, p.cap_out) : s[i][e] * p.scale_log2;
         if (p.slopes) v -= slope_r[e >> 1] * (float)(pos_r[e >> 1] - (jbase + i * 8 + tq * 2 + (e & 1)));
         if (need_mask) {
           const int j = jbase + i * 8 + tq * 2 + (e & 1);
           const int pr = pos_r[e >> 1];
-          const bool vis = j <= pr && j >= lo_r[e >> 1];
+          const bool vis = j <= pr && (j >= lo_r[e >> 1] || j < p.keep);
           if (!vis) v = -INFINITY;
         }
         s[i][e] = v;
@@ -433,14 +435,15 @@ DINFER_API int64_t dinfer_attention_tc_scratch_floats(int B, int H, int D, int s
 // block_table [B, max_blocks]; cu_seqlens [B+1]; seq_lens [B] (length after this step).
 // any_decode / any_prefill: whether the batch holds requests with q_len == 1 / q_len > 1.
 // scratch: dinfer_attention_tc_scratch_floats() floats, or null when splits == 1.
-// chunked: window is the size of the chunks (see first_key).
+// chunked: window is the size of the chunks (see first_key).  keep_first: with a window, the keys below it are seen too.
+// softcap > 0: a score is softcap * tanh(score / softcap), ahead of the bias.
 // sink != 0: the softmax has one more term that carries no value, of score sinks[h] (f32 [H]; null: 0, that is
 // p_j = exp(s_j) / (1 + sum exp(s_j))).
 // slopes: f32 [H] or null; with them score_ij - slopes[h] * (i - j).
 DINFER_API int dinfer_attention_tc_bias(const void* q, int64_t ldq, void* out, int64_t ldo, const void* cache,
                                         const int* block_table, int max_blocks, const int* cu_seqlens,
                                         const int* seq_lens, int B, int H, int Hkv, int D, int block_size,
-                                        float scale, int window, int chunked, int sink, const float* sinks,
+                                        float scale, int window, int chunked, int keep_first, float softcap, int sink, const float* sinks,
                                         const float* slopes, int max_q_len,
                                         int any_decode, int any_prefill, int splits, float* scratch, cudaStream_t stream) {
   if (B <= 0 || H <= 0 || Hkv <= 0 || H % Hkv || block_size <= 0 || max_blocks <= 0)
@@ -449,6 +452,8 @@ DINFER_API int dinfer_attention_tc_bias(const void* q, int64_t ldq, void* out, i
     return refuse(DINFER_BAD_ARGUMENT, "attention_tc: head_dim %d / group %d not supported (32, 64, 128; group <= 16)", D, H / Hkv);
   if ((ldq % 8) || (ldo % 2) || (reinterpret_cast<uintptr_t>(q) & 15) || (reinterpret_cast<uintptr_t>(cache) & 15))
     return refuse(DINFER_BAD_ARGUMENT, "attention_tc: q rows and the cache must be 16-byte aligned");
+  if (keep_first < 0 || (keep_first > 0 && chunked) || !(softcap >= 0.f))
+    return refuse(DINFER_BAD_ARGUMENT, "attention_tc: keep_first %d, softcap %g (kept keys belong to a window)", keep_first, (double)softcap);
   if (splits < 1 || (splits > 1 && !scratch)) return refuse(DINFER_BAD_ARGUMENT, "attention_tc: splits=%d needs scratch", splits);
   if (Hkv > 65535 || B > 65535) return refuse(DINFER_BAD_ARGUMENT, "attention_tc: too many heads or requests for the grid");
   Params p;
@@ -457,6 +462,11 @@ DINFER_API int dinfer_attention_tc_bias(const void* q, int64_t ldq, void* out, i
   p.cu_seqlens = cu_seqlens; p.seq_lens = seq_lens; p.H = H; p.Hkv = Hkv; p.group = H / Hkv;
   p.block_size = block_size; p.window = window; p.chunked = chunked; p.sink = sink; p.sinks = sinks; p.scale_log2 = scale * 1.4426950408889634f;
   p.slopes = slopes;
+  p.keep = window > 0 ? keep_first : 0;
+  p.cap_in = p.cap_out = 0.f;
+  if (softcap > 0.f) {                          // the capped scores come out in log2 units
+    p.cap_in = 2.f * p.scale_log2 / softcap; p.cap_out = softcap * 1.4426950408889634f; p.scale_log2 = 1.f;
+  }
   p.splits = splits; p.part_o = scratch;
   p.part_ml = scratch ? scratch + (int64_t)B * H * splits * D : nullptr;
   if (D == 32) return launch<32>(p, B, max_q_len, any_decode, any_prefill, stream);
@@ -470,7 +480,7 @@ DINFER_API int dinfer_attention_tc_sink(const void* q, int64_t ldq, void* out, i
                                         float scale, int window, int sink, int max_q_len, int any_decode,
                                         int any_prefill, int splits, float* scratch, cudaStream_t stream) {
   return dinfer_attention_tc_bias(q, ldq, out, ldo, cache, block_table, max_blocks, cu_seqlens, seq_lens, B, H, Hkv, D,
-                                  block_size, scale, window, 0, sink, nullptr, nullptr, max_q_len, any_decode, any_prefill, splits,
+                                  block_size, scale, window, 0, 0, 0.f, sink, nullptr, nullptr, max_q_len, any_decode, any_prefill, splits,
                                   scratch, stream);
 }
 

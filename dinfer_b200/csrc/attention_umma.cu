@@ -48,6 +48,8 @@ struct Params {
   int B, H, Hkv, group, block_size, bs_log2, window, chunked;
   int sink;                    // one more softmax term without a value, of score sinks[head] (null: 0)
   const float* sinks;
+  int keep;                    // with a window: the keys below it are seen too
+  float cap_in, cap_out;       // a soft cap on the scores (CAP), see softcap_log2
   int ksplit;                          // CTAs of a cluster that share a row-tile pair's keys (1, 2, 4 or 8)
   float scale_log2;
   const float* slopes;                 // [H] or null: a distance bias, score - slopes[h] * (i - j)
@@ -61,7 +63,7 @@ template <int D> constexpr size_t smem_bytes() {
 // Two row tiles (A, B) of 128 rows per CTA, each with eight softmax warps.  O accumulates in tensor memory
 // across tiles; a row's reference maximum is only raised when it grows by more than 2^8 (the accumulator and
 // the running sums are then rescaled in place), so P stays below 256 and the rescale is rare.
-template <int D>
+template <int D, bool CAP>
 __global__ void __maxnreg__(96)
 attention_umma_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_constant__ CUtensorMap map_kv, const Params p) {
   constexpr int NH = D / 64;                          // 64-wide halves of the head
@@ -131,15 +133,16 @@ attention_umma_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_co
   const int lo = first_key(hist + first_tok, p.window, p.chunked);
   // the key tiles of the pair, dealt out to the cluster's CTAs in runs of `per` (a CTA may get none)
   const int tile_first = lo / BN;
-  const int n_all = (hi + BN - 1) / BN - tile_first;   // tiles of B (or of A when B does not exist)
-  const int n_all_a = (hi_a + BN - 1) / BN - tile_first;
+  const int kept = kept_tiles(p.keep, BN, tile_first);    // tiles with kept keys in front of the window come first
+  const int n_all = kept + (hi + BN - 1) / BN - tile_first;   // tiles of B (or of A when B does not exist)
+  const int n_all_a = kept + (hi_a + BN - 1) / BN - tile_first;
   // The launch's split is an upper bound (a graph is captured for the longest request there may be): a pair is
   // shared by as many CTAs as leave each at least four tiles; the cluster's other CTAs have nothing to do with it.
   int ks = p.ksplit;
   while (ks > 1 && n_all < 4 * ks) ks >>= 1;
   if (rank >= ks) return;
   const int per = (n_all + ks - 1) / ks;
-  const int tile_begin = tile_first + rank * per;
+  const int v0 = rank * per;                           // this CTA's first visit (see tile_of)
   const int n_tiles = max(0, min(per, n_all - rank * per));
   const int n_tiles_a = max(0, min(per, n_all_a - rank * per));
 
@@ -148,9 +151,9 @@ attention_umma_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_co
 
   // page-table slice of this CTA's keys, and zeroed K/V stages (a page that is skipped leaves its slot as it
   // was: it must hold finite numbers, because a masked key still meets 0 * V)
-  const int table_first = (tile_begin * BN) >> p.bs_log2;
+  const int table_first = (tile_of(max(v0, kept), kept, tile_first) * BN) >> p.bs_log2;   // (kept tiles' entries are read as they come)
   {
-    const int last = (min((tile_begin + n_tiles) * BN, hi) - 1) >> p.bs_log2;
+    const int last = (min(tile_of(max(v0 + n_tiles, kept), kept, tile_first) * BN, hi) - 1) >> p.bs_log2;
     for (int i = threadIdx.x; i < TABLE_SLOTS && table_first + i <= last; i += NTHREADS) s_table[i] = table[table_first + i];
     uint4* z = reinterpret_cast<uint4*>(smem_dyn + (sK - smem_u32(smem_dyn)));
     for (int i = threadIdx.x; i < (int)(2 * STAGES * KV_BYTES / 16); i += NTHREADS) z[i] = make_uint4(0, 0, 0, 0);
@@ -199,16 +202,16 @@ attention_umma_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_co
     bool alive = true;
     for (int j = 0; j < n_tiles && alive; ++j) {
       const int s = j % STAGES;
-      const int j0 = (tile_begin + j) * BN;
+      const int j0 = tile_of(v0 + j, kept, tile_first) * BN;
       // this lane's copy: page x of the tile, 64-wide half h
       bool valid = false;
       int row_k = 0, col = 0; uint32_t off = 0;
       if (lane < n_ops) {
         const int x = lane / NH, h = lane % NH;
         const int key = j0 + x * br;
-        if (key < hi && key + br > lo) {
+        if (key < hi && (key + br > lo || key < p.keep)) {
           const int e = (key >> p.bs_log2) - table_first;
-          const int blk = e < TABLE_SLOTS ? s_table[e] : table[key >> p.bs_log2];
+          const int blk = e >= 0 && e < TABLE_SLOTS ? s_table[e] : table[key >> p.bs_log2];
           if (blk >= 0) {
             valid = true;
             row_k = (blk * 2 * p.Hkv + hk) * p.block_size + (key & (p.block_size - 1));
@@ -340,7 +343,7 @@ attention_umma_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_co
     for (int j = 0; j < n_w; ++j) {
       if (ok && !__all_sync(0xffffffffu, mbar_wait(smem_u32(&s_full[w]), j & 1))) { s_abort = 1; atomicExch(p.status, 15); ok = false; }
       tc_fence_after();
-      const int jbase = (tile_begin + j) * BN;
+      const int jbase = tile_of(v0 + j, kept, tile_first) * BN;
       const bool need_mask = (jbase + BN - 1 > hist + first_tok_w) || jbase < lo_all;
       // this thread's 64 scores; their maximum (raw: the scale is positive), as eight short chains
       float v0[32], v1[32];
@@ -349,6 +352,13 @@ attention_umma_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_co
         tmem_ld32(s_addr + h * 64, v0);
         tmem_ld32(s_addr + h * 64 + 32, v1);
         tmem_ld_wait();
+        if (CAP) {
+#pragma unroll
+          for (int i = 0; i < 32; ++i) {
+            v0[i] = softcap_log2(v0[i], p.cap_in, p.cap_out);
+            v1[i] = softcap_log2(v1[i], p.cap_in, p.cap_out);
+          }
+        }
         if (p.slopes) {
           const float d0 = (float)(jbase + h * 64 - pos);
 #pragma unroll
@@ -361,8 +371,8 @@ attention_umma_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_co
 #pragma unroll
           for (int i = 0; i < 32; ++i) {
             const int ja = jbase + h * 64 + i, jc = ja + 32;
-            if (!(ja <= pos && ja >= row_lo)) v0[i] = -INFINITY;
-            if (!(jc <= pos && jc >= row_lo)) v1[i] = -INFINITY;
+            if (!(ja <= pos && (ja >= row_lo || ja < p.keep))) v0[i] = -INFINITY;
+            if (!(jc <= pos && (jc >= row_lo || jc < p.keep))) v1[i] = -INFINITY;
           }
         }
         float mq[8];
@@ -572,10 +582,10 @@ EncodeTiledFn encode_fn() {
   return fn;
 }
 
-template <int D>
+template <int D, bool CAP>
 int launch(const CUtensorMap& mq, const CUtensorMap& mkv, const Params& p, dim3 grid, cudaStream_t stream) {
   static_assert((size_t)2 * STAGES * BN * D * 2 >= (size_t)7 * 32 * D * 4, "the K/V stages hold what seven senders bring");
-  auto k = attention_umma_kernel<D>;
+  auto k = attention_umma_kernel<D, CAP>;
   constexpr size_t sm = smem_bytes<D>();
   static bool opted = false;
   if (!opted) {
@@ -589,7 +599,7 @@ int launch(const CUtensorMap& mq, const CUtensorMap& mkv, const Params& p, dim3 
 
 template <int D>
 int max_clusters(int key_splits) {
-  auto k = attention_umma_kernel<D>;
+  auto k = attention_umma_kernel<D, false>;
   constexpr size_t sm = smem_bytes<D>();
   cudaError_t e = cudaFuncSetAttribute(k, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)sm);
   if (e != cudaSuccess) return -refuse((int)e, "attention_umma: shared memory opt-in failed: %s", cudaGetErrorString(e));
@@ -627,13 +637,14 @@ DINFER_API int dinfer_attention_umma_supports(int D, int group, int block_size) 
 // key_splits (1, 2, 4 or 8): that many CTAs of a cluster share the keys of a row-tile pair and fold their results
 // through distributed shared memory; for steps with fewer row tiles than the device has SMs.
 // q: [T, ...] rows of stride ldq with head h at h*D (all H heads); cache [num_blocks, 2, Hkv, block, D] bf16.
-// chunked: window is the size of the chunks (see first_key).
+// chunked: window is the size of the chunks (see first_key).  keep_first: with a window, the keys below it are seen too.
+// softcap > 0: a score is softcap * tanh(score / softcap), ahead of the bias.
 // sink != 0: the softmax has one more term that carries no value, of score sinks[h] (f32 [H]; null: 0).
 // slopes: f32 [H] or null; with them score_ij - slopes[h] * (i - j).
 DINFER_API int dinfer_attention_umma_bias(const void* q, int64_t ldq, void* out, int64_t ldo, const void* cache,
                                           int64_t num_blocks, const int* block_table, int max_blocks,
                                           const int* cu_seqlens, const int* seq_lens, int T, int B, int H, int Hkv, int D,
-                                          int block_size, float scale, int window, int chunked, int sink, const float* sinks, const float* slopes,
+                                          int block_size, float scale, int window, int chunked, int keep_first, float softcap, int sink, const float* sinks, const float* slopes,
                                           int max_q_len, int pair_bound, int key_splits, int* status, cudaStream_t stream);
 
 DINFER_API int dinfer_attention_umma_sink(const void* q, int64_t ldq, void* out, int64_t ldo, const void* cache,
@@ -642,18 +653,20 @@ DINFER_API int dinfer_attention_umma_sink(const void* q, int64_t ldq, void* out,
                                           int block_size, float scale, int window, int sink, int max_q_len,
                                           int pair_bound, int key_splits, int* status, cudaStream_t stream) {
   return dinfer_attention_umma_bias(q, ldq, out, ldo, cache, num_blocks, block_table, max_blocks, cu_seqlens, seq_lens, T, B,
-                                    H, Hkv, D, block_size, scale, window, 0, sink, nullptr, nullptr, max_q_len, pair_bound, key_splits,
+                                    H, Hkv, D, block_size, scale, window, 0, 0, 0.f, sink, nullptr, nullptr, max_q_len, pair_bound, key_splits,
                                     status, stream);
 }
 
 DINFER_API int dinfer_attention_umma_bias(const void* q, int64_t ldq, void* out, int64_t ldo, const void* cache,
                                           int64_t num_blocks, const int* block_table, int max_blocks,
                                           const int* cu_seqlens, const int* seq_lens, int T, int B, int H, int Hkv, int D,
-                                          int block_size, float scale, int window, int chunked, int sink, const float* sinks, const float* slopes,
+                                          int block_size, float scale, int window, int chunked, int keep_first, float softcap, int sink, const float* sinks, const float* slopes,
                                           int max_q_len, int pair_bound, int key_splits, int* status, cudaStream_t stream) {
   if (T <= 0 || B <= 0 || H <= 0 || Hkv <= 0 || H % Hkv || max_blocks <= 0 || num_blocks <= 0)
     return refuse(DINFER_BAD_ARGUMENT, "attention_umma: bad sizes T=%d B=%d H=%d Hkv=%d", T, B, H, Hkv);
   const int group = H / Hkv;
+  if (keep_first < 0 || (keep_first > 0 && chunked) || !(softcap >= 0.f))
+    return refuse(DINFER_BAD_ARGUMENT, "attention_umma: keep_first %d, softcap %g (kept keys belong to a window)", keep_first, (double)softcap);
   if (!(scale > 0.f)) return refuse(DINFER_BAD_ARGUMENT, "attention_umma: the score scale must be positive, got %g", (double)scale);
   if (!dinfer_attention_umma_supports(D, group, block_size))
     return refuse(DINFER_BAD_ARGUMENT, "attention_umma: head_dim %d, group %d, block_size %d not supported "
@@ -698,12 +711,18 @@ DINFER_API int dinfer_attention_umma_bias(const void* q, int64_t ldq, void* out,
   while ((1 << p.bs_log2) < block_size) ++p.bs_log2;
   p.window = window; p.chunked = chunked; p.sink = sink; p.sinks = sinks; p.scale_log2 = scale * 1.4426950408889634f; p.status = status;
   p.slopes = slopes;
+  p.keep = window > 0 ? keep_first : 0;
+  p.cap_in = p.cap_out = 0.f;
+  if (softcap > 0.f) {                          // the capped scores come out in log2 units
+    p.cap_in = 2.f * p.scale_log2 / softcap; p.cap_out = softcap * 1.4426950408889634f; p.scale_log2 = 1.f;
+  }
   p.ksplit = key_splits; p.B = B;
   // pairs of 128-row tiles in the batch: the caller's bound, or every request taken for the longest
   int64_t pairs = pair_bound > 0 ? pair_bound : (int64_t)B * (((int64_t)max_q_len * group + 2 * BM - 1) / (2 * BM));
   if (pairs > 65535) return refuse(DINFER_BAD_ARGUMENT, "attention_umma: %lld row-tile pairs are too many for the grid", (long long)pairs);
   dim3 grid(Hkv * key_splits, (unsigned)pairs, 1);
-  return D == 64 ? launch<64>(mq, mkv, p, grid, stream) : launch<128>(mq, mkv, p, grid, stream);
+  if (softcap > 0.f) return D == 64 ? launch<64, true>(mq, mkv, p, grid, stream) : launch<128, true>(mq, mkv, p, grid, stream);
+  return D == 64 ? launch<64, false>(mq, mkv, p, grid, stream) : launch<128, false>(mq, mkv, p, grid, stream);
 }
 
 DINFER_API int dinfer_attention_umma(const void* q, int64_t ldq, void* out, int64_t ldo, const void* cache,

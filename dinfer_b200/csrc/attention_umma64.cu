@@ -46,6 +46,8 @@ struct Params {
   int B, H, Hkv, group, block_size, bs_log2, window, chunked;
   int sink;                    // one more softmax term without a value, of score sinks[head] (null: 0)
   const float* sinks;
+  int keep;                    // with a window: the keys below it are seen too
+  float cap_in, cap_out;       // a soft cap on the scores (CAP), see softcap_log2
   float scale_log2;
   const float* slopes;         // [H] or null: a distance bias, score - slopes[h] * (i - j)
   int* status;
@@ -60,7 +62,7 @@ template <int D> constexpr size_t smem_bytes() {
 // O accumulates in tensor memory across tiles; a row's reference maximum is only raised when it grows
 // by more than 2^8 (the accumulator and the running sum are then rescaled in place), so P stays below
 // 256 and the rescale is rare.
-template <int D>
+template <int D, bool CAP>
 __global__ void __launch_bounds__(NTHREADS, 1)
 attention_umma64_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_constant__ CUtensorMap map_kv, const Params p) {
   constexpr int NH = D / 64;                          // 64-wide halves of the head
@@ -124,16 +126,17 @@ attention_umma64_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_
   const int hi = hist + last_tok + 1;
   const int hi_a = hist + last_tok_a + 1;
   const int lo = first_key(hist + first_tok, p.window, p.chunked);
-  const int tile_begin = lo / BN, tile_end = (hi + BN - 1) / BN;
-  const int n_tiles = tile_end - tile_begin;           // tiles of B (or of A when B does not exist)
-  const int n_tiles_a = (hi_a + BN - 1) / BN - tile_begin;
+  const int tile_first = lo / BN, tile_end = (hi + BN - 1) / BN;
+  const int kept = kept_tiles(p.keep, BN, tile_first); // tiles with kept keys in front of the window come first
+  const int n_tiles = kept + tile_end - tile_first;    // tiles of B (or of A when B does not exist)
+  const int n_tiles_a = kept + (hi_a + BN - 1) / BN - tile_first;
 
   const uint32_t base = (smem_u32(smem_dyn) + 1023u) & ~1023u;
   const uint32_t sQ = base, sK = sQ + 2 * Q_BYTES, sV = sK + STAGES * KV_BYTES, sP = sV + STAGES * KV_BYTES;
 
   // page-table slice of this CTA's keys, and zeroed K/V stages (a page that is skipped leaves its slot as it
   // was: it must hold finite numbers, because a masked key still meets 0 * V)
-  const int table_first = (tile_begin * BN) >> p.bs_log2;
+  const int table_first = (tile_first * BN) >> p.bs_log2;  // (kept tiles' entries are read as they come)
   {
     const int last = (min(tile_end * BN, hi) - 1) >> p.bs_log2;
     for (int i = threadIdx.x; i < TABLE_SLOTS && table_first + i <= last; i += NTHREADS) s_table[i] = table[table_first + i];
@@ -184,16 +187,16 @@ attention_umma64_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_
     bool alive = true;
     for (int j = 0; j < n_tiles && alive; ++j) {
       const int s = j % STAGES;
-      const int j0 = (tile_begin + j) * BN;
+      const int j0 = tile_of(j, kept, tile_first) * BN;
       // this lane's copy: page x of the tile, 64-wide half h (the same for K and for V)
       bool valid = false;
       int row_k = 0, col = 0; uint32_t off = 0;
       if (lane < n_ops) {
         const int x = lane / NH, h = lane % NH;
         const int key = j0 + x * br;
-        if (key < hi && key + br > lo) {
+        if (key < hi && (key + br > lo || key < p.keep)) {
           const int e = (key >> p.bs_log2) - table_first;
-          const int blk = e < TABLE_SLOTS ? s_table[e] : table[key >> p.bs_log2];
+          const int blk = e >= 0 && e < TABLE_SLOTS ? s_table[e] : table[key >> p.bs_log2];
           if (blk >= 0) {
             valid = true;
             row_k = (blk * 2 * p.Hkv + hk) * p.block_size + (key & (p.block_size - 1));
@@ -316,7 +319,14 @@ attention_umma64_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_
       tmem_ld32(s_addr + (j & 1) * BN, s0);
       tmem_ld32(s_addr + (j & 1) * BN + 32, s1);
       tmem_ld_wait();
-      const int jbase = (tile_begin + j) * BN;
+      const int jbase = tile_of(j, kept, tile_first) * BN;
+      if (CAP) {
+#pragma unroll
+        for (int i = 0; i < 32; ++i) {
+          s0[i] = softcap_log2(s0[i], p.cap_in, p.cap_out);
+          s1[i] = softcap_log2(s1[i], p.cap_in, p.cap_out);
+        }
+      }
       if (p.slopes) {
         const float d0 = (float)(jbase - pos);
 #pragma unroll
@@ -330,8 +340,8 @@ attention_umma64_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_
 #pragma unroll
         for (int i = 0; i < 32; ++i) {
           const int ja = jbase + i, jc = jbase + 32 + i;
-          if (!(ja <= pos && ja >= row_lo)) s0[i] = -INFINITY;
-          if (!(jc <= pos && jc >= row_lo)) s1[i] = -INFINITY;
+          if (!(ja <= pos && (ja >= row_lo || ja < p.keep))) s0[i] = -INFINITY;
+          if (!(jc <= pos && (jc >= row_lo || jc < p.keep))) s1[i] = -INFINITY;
         }
       }
       // maximum of the raw scores (the scale is positive), as eight short chains instead of one long one
@@ -445,9 +455,9 @@ EncodeTiledFn encode_fn() {
   return fn;
 }
 
-template <int D>
+template <int D, bool CAP>
 int launch(const CUtensorMap& mq, const CUtensorMap& mkv, const Params& p, dim3 grid, cudaStream_t stream) {
-  auto k = attention_umma64_kernel<D>;
+  auto k = attention_umma64_kernel<D, CAP>;
   constexpr size_t sm = smem_bytes<D>();
   static bool opted = false;
   if (!opted) {
@@ -470,13 +480,14 @@ DINFER_API int dinfer_attention_umma64_supports(int D, int group, int block_size
 
 // Prompt portions (q_len > 1) only; requests that bring one token are skipped.
 // q: [T, ...] rows of stride ldq with head h at h*D (all H heads); cache [num_blocks, 2, Hkv, block, D] bf16.
-// chunked: window is the size of the chunks (see first_key).
+// chunked: window is the size of the chunks (see first_key).  keep_first: with a window, the keys below it are seen too.
+// softcap > 0: a score is softcap * tanh(score / softcap), ahead of the bias.
 // sink != 0: the softmax has one more term that carries no value, of score sinks[h] (f32 [H]; null: 0).
 // slopes: f32 [H] or null; with them score_ij - slopes[h] * (i - j).
 DINFER_API int dinfer_attention_umma64_bias(const void* q, int64_t ldq, void* out, int64_t ldo, const void* cache,
                                      int64_t num_blocks, const int* block_table, int max_blocks,
                                      const int* cu_seqlens, const int* seq_lens, int T, int B, int H, int Hkv, int D,
-                                     int block_size, float scale, int window, int chunked, int sink, const float* sinks, const float* slopes, int max_q_len,
+                                     int block_size, float scale, int window, int chunked, int keep_first, float softcap, int sink, const float* sinks, const float* slopes, int max_q_len,
                                      int pair_bound, int* status, cudaStream_t stream);
 
 DINFER_API int dinfer_attention_umma64_sink(const void* q, int64_t ldq, void* out, int64_t ldo, const void* cache,
@@ -485,17 +496,19 @@ DINFER_API int dinfer_attention_umma64_sink(const void* q, int64_t ldq, void* ou
                                      int block_size, float scale, int window, int sink, int max_q_len, int pair_bound,
                                      int* status, cudaStream_t stream) {
   return dinfer_attention_umma64_bias(q, ldq, out, ldo, cache, num_blocks, block_table, max_blocks, cu_seqlens, seq_lens, T, B,
-                                      H, Hkv, D, block_size, scale, window, 0, sink, nullptr, nullptr, max_q_len, pair_bound, status, stream);
+                                      H, Hkv, D, block_size, scale, window, 0, 0, 0.f, sink, nullptr, nullptr, max_q_len, pair_bound, status, stream);
 }
 
 DINFER_API int dinfer_attention_umma64_bias(const void* q, int64_t ldq, void* out, int64_t ldo, const void* cache,
                                      int64_t num_blocks, const int* block_table, int max_blocks,
                                      const int* cu_seqlens, const int* seq_lens, int T, int B, int H, int Hkv, int D,
-                                     int block_size, float scale, int window, int chunked, int sink, const float* sinks, const float* slopes, int max_q_len,
+                                     int block_size, float scale, int window, int chunked, int keep_first, float softcap, int sink, const float* sinks, const float* slopes, int max_q_len,
                                      int pair_bound, int* status, cudaStream_t stream) {
   if (T <= 0 || B <= 0 || H <= 0 || Hkv <= 0 || H % Hkv || max_blocks <= 0 || num_blocks <= 0)
     return refuse(DINFER_BAD_ARGUMENT, "attention_umma64: bad sizes T=%d B=%d H=%d Hkv=%d", T, B, H, Hkv);
   const int group = H / Hkv;
+  if (keep_first < 0 || (keep_first > 0 && chunked) || !(softcap >= 0.f))
+    return refuse(DINFER_BAD_ARGUMENT, "attention_umma64: keep_first %d, softcap %g (kept keys belong to a window)", keep_first, (double)softcap);
   if (!(scale > 0.f)) return refuse(DINFER_BAD_ARGUMENT, "attention_umma64: the score scale must be positive, got %g", (double)scale);
   if (!dinfer_attention_umma64_supports(D, group, block_size))
     return refuse(DINFER_BAD_ARGUMENT, "attention_umma64: head_dim %d, group %d, block_size %d not supported "
@@ -538,11 +551,17 @@ DINFER_API int dinfer_attention_umma64_bias(const void* q, int64_t ldq, void* ou
   while ((1 << p.bs_log2) < block_size) ++p.bs_log2;
   p.window = window; p.chunked = chunked; p.sink = sink; p.sinks = sinks; p.scale_log2 = scale * 1.4426950408889634f; p.status = status; p.B = B;
   p.slopes = slopes;
+  p.keep = window > 0 ? keep_first : 0;
+  p.cap_in = p.cap_out = 0.f;
+  if (softcap > 0.f) {                          // the capped scores come out in log2 units
+    p.cap_in = 2.f * p.scale_log2 / softcap; p.cap_out = softcap * 1.4426950408889634f; p.scale_log2 = 1.f;
+  }
   // pairs of 128-row tiles in the batch: the caller's bound, or every request taken for the longest
   int64_t pairs = pair_bound > 0 ? pair_bound : (int64_t)B * (((int64_t)max_q_len * group + 2 * BM - 1) / (2 * BM));
   if (pairs > 65535) return refuse(DINFER_BAD_ARGUMENT, "attention_umma64: %lld row-tile pairs are too many for the grid", (long long)pairs);
   dim3 grid(Hkv, (unsigned)pairs, 1);
-  return D == 64 ? launch<64>(mq, mkv, p, grid, stream) : launch<128>(mq, mkv, p, grid, stream);
+  if (softcap > 0.f) return D == 64 ? launch<64, true>(mq, mkv, p, grid, stream) : launch<128, true>(mq, mkv, p, grid, stream);
+  return D == 64 ? launch<64, false>(mq, mkv, p, grid, stream) : launch<128, false>(mq, mkv, p, grid, stream);
 }
 
 DINFER_API int dinfer_attention_umma64(const void* q, int64_t ldq, void* out, int64_t ldo, const void* cache,

@@ -49,6 +49,7 @@ LIBRARIES: Dict[str, tuple] = {
     "sandwich": ("sandwich.cu", []),
     "linear_state": ("linear_state.cu", []),
     "token_side": ("token_side.cu", []),
+    "state_space": ("state_space.cu", []),
     # host-side bookkeeping (page pools, cache manager, decode plans): plain C++, no CUDA
     "host_core": ("host_core.cpp", []),
 }

@@ -81,6 +81,17 @@ __device__ __forceinline__ float xielu_fast(float z, float a_pos, float a_neg) {
   return fmaf(0.5f, z, fmaf(a_pos * p, p, a_neg * e));
 }
 
+// A gate with a bias on the up side and both sides clamped: g = min(gate, limit), u = clamp(up, -limit, limit),
+// g * sigmoid(alpha g) * (u + 1).  `fast`: for results that are rounded to bfloat16.
+__device__ __forceinline__ float clamped_swish(float gate, float up, float limit, float alpha) {
+  const float g = fminf(gate, limit), u = fminf(fmaxf(up, -limit), limit);
+  return g / (1.f + expf(-alpha * g)) * (u + 1.f);
+}
+__device__ __forceinline__ float clamped_swish_fast(float gate, float up, float limit, float alpha) {
+  const float g = fminf(gate, limit), u = fminf(fmaxf(up, -limit), limit);
+  return __fdividef(g, 1.f + __expf(-alpha * g)) * (u + 1.f);      // 0 where 1 + e^.. passes 2^126, as is its limit
+}
+
 // ---- which keys a query sees
 // The first key that a query at position pos (>= 0) sees: all of its request's (window <= 0), the last `window` ones
 // (itself included), or with `chunked` those of its own chunk (chunks of `window` positions, counted from the
@@ -88,6 +99,22 @@ __device__ __forceinline__ float xielu_fast(float z, float a_pos, float a_neg) {
 __device__ __forceinline__ int first_key(int pos, int window, int chunked) {
   if (window <= 0) return 0;
   return chunked ? pos / window * window : max(0, pos - window + 1);
+}
+// Kept first keys: with keep > 0 a query sees the keys below `keep` too, however far back they lie.  A kernel that walks
+// key tiles of BN visits the tiles that hold kept keys and lie before the first tile of its own range [tile_first, ..),
+// then its range: `kept_tiles` of them, and visit i is tile `tile_of(i, ...)`.
+__device__ __forceinline__ int kept_tiles(int keep, int bn, int tile_first) {
+  return min((keep + bn - 1) / bn, tile_first);
+}
+__device__ __forceinline__ int tile_of(int i, int kept, int tile_first) { return i < kept ? i : tile_first + i - kept; }
+// A soft cap on a score, in log2 units: log2(e) * cap * tanh(s / cap) with cap_in = 2 log2(e) / cap (times the score's
+// scale) and cap_out = log2(e) * cap.  tanh x = 1 - 2 / (1 + e^2x) through the fast exponential and reciprocal: its error
+// is a few 1e-7 of the cap, absolute, which is what a score's error counts by.
+__device__ __forceinline__ float softcap_log2(float s, float cap_in, float cap_out) {
+  float e, r;
+  asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(e) : "f"(s * cap_in));
+  asm("rcp.approx.ftz.f32 %0, %1;" : "=f"(r) : "f"(1.f + e));       // e = inf gives 0
+  return fmaf(-2.f * cap_out, r, cap_out);
 }
 // The softmax's extra term of a head (it has no key and no value): its score times log2(e); the score is sinks[head],
 // or 0 where no sinks are given.

@@ -130,7 +130,8 @@ __device__ __forceinline__ float gate_activation(float z, int act) {
   }
 }
 template <typename T>
-__global__ void gated_act_kernel(const T* __restrict__ x, T* __restrict__ out, int inter, int64_t ldx, int pairs, int act) {
+__global__ void gated_act_kernel(const T* __restrict__ x, T* __restrict__ out, int inter, int64_t ldx, int pairs, int act,
+                                 float ga, float gb) {
   pdl_enter();
   const int t = blockIdx.x;
   const T* row = x + (int64_t)t * ldx;
@@ -138,7 +139,33 @@ __global__ void gated_act_kernel(const T* __restrict__ x, T* __restrict__ out, i
   for (int i = blockIdx.y * blockDim.x + threadIdx.x; i < inter; i += gridDim.y * blockDim.x) {
     const float a = to_f32<T>(pairs ? row[2 * i] : row[i]);
     const float b = to_f32<T>(pairs ? row[2 * i + 1] : row[inter + i]);
-    o[i] = from_f32<T>(gate_activation(a, act) * b);
+    o[i] = from_f32<T>(act == 4 ? clamped_swish(a, b, ga, gb) : gate_activation(a, act) * b);
+  }
+}
+
+// bfloat16 in pairs, the clamped gate: 16 inputs (two 16-byte loads) -> 8 outputs (one 16-byte store) per thread
+__global__ void clamped_swish_pairs_bf16_kernel(const __nv_bfloat16* __restrict__ x, __nv_bfloat16* __restrict__ out,
+                                                int inter8, int64_t ldx, int inter, float limit, float alpha) {
+  pdl_enter();
+  const int t = blockIdx.x;
+  const uint4* src = reinterpret_cast<const uint4*>(x + (int64_t)t * ldx);
+  uint4* o = reinterpret_cast<uint4*>(out + (int64_t)t * inter);
+  for (int i = blockIdx.y * blockDim.x + threadIdx.x; i < inter8; i += gridDim.y * blockDim.x) {
+    const uint4 a = src[2 * i], b = src[2 * i + 1];
+    const __nv_bfloat162* pa = reinterpret_cast<const __nv_bfloat162*>(&a);
+    const __nv_bfloat162* pb = reinterpret_cast<const __nv_bfloat162*>(&b);
+    float r[8];
+#pragma unroll
+    for (int j = 0; j < 4; ++j) {
+      const float2 g0 = __bfloat1622float2(pa[j]), g1 = __bfloat1622float2(pb[j]);
+      r[j] = clamped_swish_fast(g0.x, g0.y, limit, alpha);
+      r[4 + j] = clamped_swish_fast(g1.x, g1.y, limit, alpha);
+    }
+    uint4 w;
+    __nv_bfloat162* pw = reinterpret_cast<__nv_bfloat162*>(&w);
+#pragma unroll
+    for (int j = 0; j < 4; ++j) pw[j] = __floats2bfloat162_rn(r[2 * j], r[2 * j + 1]);
+    o[i] = w;
   }
 }
 
@@ -420,18 +447,31 @@ DINFER_API int dinfer_add_bias(void* out, int64_t ld, const void* bias, int T, i
   return 0;
 }
 
-// x [T, 2*inter] with row stride ldx; out [T, inter]; act 0 silu, 1 tanh-gelu, 2 relu, 3 relu squared.
-DINFER_API int dinfer_gated_act(const void* x, void* out, int T, int inter, int64_t ldx, int dtype, int pairs, int act,
-                                cudaStream_t stream) {
+// x [T, 2*inter] with row stride ldx; out [T, inter]; act 0 silu, 1 tanh-gelu, 2 relu, 3 relu squared, 4 the clamped gate
+// with its limit ga > 0 and its factor gb (see clamped_swish).
+DINFER_API int dinfer_gated_act_ex(const void* x, void* out, int T, int inter, int64_t ldx, int dtype, int pairs, int act,
+                                   float ga, float gb, cudaStream_t stream) {
   if (act == 0) return dinfer_silu_mul(x, out, T, inter, ldx, dtype, pairs, stream);
-  if (T < 0 || inter <= 0 || ldx < 2 * (int64_t)inter || act < 0 || act > 3)
+  if (T < 0 || inter <= 0 || ldx < 2 * (int64_t)inter || act < 0 || act > 4 || (act == 4 && !(ga > 0.f)))
     return refuse(DINFER_BAD_ARGUMENT, "gated_act: bad arguments T=%d inter=%d ldx=%lld act=%d", T, inter, (long long)ldx, act);
   if (T == 0) return 0;
+  if (act == 4 && pairs && dtype == DINFER_BF16 && inter % 8 == 0 && ldx % 8 == 0 && !(reinterpret_cast<uintptr_t>(x) & 15) &&
+      !(reinterpret_cast<uintptr_t>(out) & 15)) {
+    const int bv = (inter / 8 + 127) / 128;
+    launch_pdl(clamped_swish_pairs_bf16_kernel, dim3(T, bv > 64 ? 64 : bv), dim3(128), 0, stream, (const __nv_bfloat16*)x,
+               (__nv_bfloat16*)out, inter / 8, ldx, inter, ga, gb);
+    return cuda_status("gated_act");
+  }
   int by = (inter + 255) / 256;
   if (by > 64) by = 64;
   DINFER_DISPATCH_DTYPE(dtype, T_, {
-    launch_pdl(gated_act_kernel<T_>, dim3(T, by), dim3(256), 0, stream, (const T_*)x, (T_*)out, inter, ldx, pairs, act);
+    launch_pdl(gated_act_kernel<T_>, dim3(T, by), dim3(256), 0, stream, (const T_*)x, (T_*)out, inter, ldx, pairs, act, ga, gb);
     return cuda_status("gated_act");
   });
   return 0;
+}
+
+DINFER_API int dinfer_gated_act(const void* x, void* out, int T, int inter, int64_t ldx, int dtype, int pairs, int act,
+                                cudaStream_t stream) {
+  return dinfer_gated_act_ex(x, out, T, inter, ldx, dtype, pairs, act, 0.f, 0.f, stream);
 }

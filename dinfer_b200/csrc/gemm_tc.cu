@@ -48,7 +48,7 @@ struct GemmParams {
   int tokens, N, K;
   int k_blocks_per_split, splits;
   int act;                       // > 0: weight rows come in (gate, up) pairs and out[t, j] = g(gate_j) * up_j, N / 2 wide;
-                                 // g = silu (1) or the tanh form of gelu (2)
+                                 // g = silu (1) or the tanh form of gelu (2); 3: the clamped gate (clamped_swish with a_pos, a_neg)
   // residual mode (decode orientation): the product is added into resid [tokens, ldr] (f32) and out gets the new
   // residual times norm_w, rounded; the sums of squares of the rows this CTA owns go to ss_out[part][token]
   float* resid; int64_t ldr;
@@ -167,7 +167,10 @@ __device__ __forceinline__ float silu_mul_fast(float g, float u) { return __fdiv
 __device__ __forceinline__ float gelu_tanh_mul(float g, float u) {
   return 0.5f * g * (1.f + tanhf(0.7978845608028654f * (g + 0.044715f * g * g * g))) * u;
 }
-__device__ __forceinline__ float gate_mul(float g, float u, int act) { return act == 2 ? gelu_tanh_mul(g, u) : silu_mul(g, u); }
+__device__ __forceinline__ float gate_mul(float g, float u, const GemmParams& p) {
+  if (p.act == 3) return clamped_swish(g, u, p.a_pos, p.a_neg);
+  return p.act == 2 ? gelu_tanh_mul(g, u) : silu_mul(g, u);
+}
 __device__ __forceinline__ float grouped_act(float z, const GemmParams& p) {
   switch (p.grp_act) {
     case 5: return xielu_fast(z, p.a_pos, p.a_neg);
@@ -353,7 +356,7 @@ gemm_tc_kernel(const __grid_constant__ CUtensorMap map_a, const __grid_constant_
               const float g = __uint_as_float(v[j]);
               const float u = __shfl_down_sync(0xffffffffu, g, 1);
               if (!(lane & 1) && n + 1 < p.N && b0 + c0 + j < p.tokens)
-                out[(int64_t)(b0 + c0 + j) * p.ldc + (n >> 1)] = out_cast<OutT>(gate_mul(g, u, p.act));
+                out[(int64_t)(b0 + c0 + j) * p.ldc + (n >> 1)] = out_cast<OutT>(gate_mul(g, u, p));
             }
           } else if (!clustered) {
             if (n < p.N) {
@@ -443,7 +446,7 @@ gemm_tc_kernel(const __grid_constant__ CUtensorMap map_a, const __grid_constant_
           }
           if (p.ss_in) { g *= s_rstd[c]; u *= s_rstd[c]; }
           const int n = a0 + rank * rows_per + 2 * pr;
-          if (n + 1 < p.N) out[(int64_t)(b0 + c) * p.ldc + (n >> 1)] = out_cast<OutT>(gate_mul(g, u, p.act));
+          if (n + 1 < p.N) out[(int64_t)(b0 + c) * p.ldc + (n >> 1)] = out_cast<OutT>(gate_mul(g, u, p));
         }
       } else {
         for (int i = threadIdx.x; i < cols * rows_mine; i += NTHREADS) {
@@ -667,8 +670,9 @@ gemm_tc_pair_kernel(const __grid_constant__ CUtensorMap map_a, const __grid_cons
             float y[8];
 #pragma unroll
             for (int j = 0; j < 8; ++j)
-              y[j] = p.act == 2 ? gelu_tanh_mul(__uint_as_float(v[h][2 * j]), __uint_as_float(v[h][2 * j + 1]))
-                                : silu_mul_fast(__uint_as_float(v[h][2 * j]), __uint_as_float(v[h][2 * j + 1]));
+              y[j] = p.act == 3 ? clamped_swish_fast(__uint_as_float(v[h][2 * j]), __uint_as_float(v[h][2 * j + 1]), p.a_pos, p.a_neg)
+                     : p.act == 2 ? gelu_tanh_mul(__uint_as_float(v[h][2 * j]), __uint_as_float(v[h][2 * j + 1]))
+                                  : silu_mul_fast(__uint_as_float(v[h][2 * j]), __uint_as_float(v[h][2 * j + 1]));
             if (vec && o0 + 8 <= n_out) {
               uint4 w0;
               __nv_bfloat162* h0 = reinterpret_cast<__nv_bfloat162*>(&w0);
@@ -845,7 +849,8 @@ DINFER_DEFINE_LAST_ERROR()
 // bf16 (out_f32 = 0) or f32.  tokens <= 64: decode orientation with `splits` K splits (at most 8: the
 // CTAs of a tile form a cluster).  More tokens: prompt orientation (two SMs on a tile), splits ignored.
 // act > 0 (N even): the rows of w are (gate, up) pairs and out is [tokens, N / 2],
-// out[t, j] = g(x w_{2j}) * (x w_{2j+1}) with g = silu (act 1) or the tanh form of gelu (act 2).
+// out[t, j] = g(x w_{2j}) * (x w_{2j+1}) with g = silu (act 1) or the tanh form of gelu (act 2), or the clamped gate
+// (act 3: clamped_swish with the limit a_pos and the factor a_neg).
 // status: a device int that a kernel sets non-zero when one of its bounded waits ran out.
 //
 // The two halves of an RMSNorm between two decode products (tokens <= 64, see the kernel's header):
@@ -878,7 +883,8 @@ DINFER_API int dinfer_gemm_tc_all(const void* x, int64_t ldx, const void* w, int
     return refuse(DINFER_BAD_ARGUMENT, "gemm_tc: activation %d (0 to 5) without a gate and a residual", unary);
   GemmParams p = {};
   p.grp_act = unary; p.a_pos = a_pos; p.a_neg = a_neg;
-  if (act < 0 || act > 2) return refuse(DINFER_BAD_ARGUMENT, "gemm_tc: unknown gate %d (0 none, 1 silu, 2 tanh-gelu)", act);
+  if (act < 0 || act > 3 || (act == 3 && !(a_pos > 0.f)))
+    return refuse(DINFER_BAD_ARGUMENT, "gemm_tc: unknown gate %d (0 none, 1 silu, 2 tanh-gelu, 3 clamped with a positive limit)", act);
   p.act = act;
   p.resid = resid; p.ldr = ldr; p.norm_w = norm_w; p.norm_w_f32 = norm_w_f32; p.ss_out = ss_out;
   p.ss_in = ss_in; p.ss_parts = ss_parts; p.ss_stride = ss_stride; p.inv_size = inv_size; p.eps = eps;
@@ -933,13 +939,14 @@ DINFER_API int dinfer_gemm_tc_fused(const void* x, int64_t ldx, const void* w, i
 // by expert, every expert's run padded to a multiple of 256 (cap a multiple of 256), tile_expert [cap / 256] names the
 // expert of each 256-row tile (-1: none); w [E * N, K] holds the experts' matrices one behind the other.
 // epi 0: out [cap, N] = act(x w_e^T) row for row (act: 0 none, 1 relu squared, 2 silu, 3 tanh-gelu, 4 relu), or with gate
-// (1 silu, 2 tanh-gelu; N even, act 0) the expert's rows are (gate, up) pairs and out [cap, N / 2] = g(gate) * up;
+// (1 silu, 2 tanh-gelu, 3 clamped with gate_a, gate_b; N even, act 0) the expert's rows are (gate, up) pairs and out [cap, N / 2] = g(gate) * up;
 // epi 1: out [pairs, N]: row t of the product, times row_w[sorted[t]], goes to row sorted[t] (sorted[t] >= pairs: padding).
 DINFER_API int dinfer_gemm_tc_grouped(const void* x, int64_t ldx, const void* w, void* out, int64_t ldc,
                                       const int* tile_expert, const int* sorted, const float* row_w, int cap, int pairs,
-                                      int E, int N, int K, int epi, int act, int gate, int* status, cudaStream_t stream) {
+                                      int E, int N, int K, int epi, int act, int gate, float gate_a, float gate_b, int* status,
+                                      cudaStream_t stream) {
   if (cap <= 0 || cap % 256 || pairs < 0 || E <= 0 || N <= 0 || K <= 0 || !tile_expert || (epi != 0 && epi != 1) ||
-      (epi == 1 && (!sorted || !row_w)) || act < 0 || act > 4 || gate < 0 || gate > 2 || (gate && (epi || act || (N & 1))) ||
+      (epi == 1 && (!sorted || !row_w)) || act < 0 || act > 4 || gate < 0 || gate > 3 || (gate == 3 && !(gate_a > 0.f)) || (gate && (epi || act || (N & 1))) ||
       (epi == 1 && act))
     return refuse(DINFER_BAD_ARGUMENT, "gemm_tc_grouped: bad arguments cap=%d pairs=%d E=%d N=%d K=%d epi=%d", cap, pairs, E, N, K, epi);
   if ((K % 8) || (ldx % 8) || (reinterpret_cast<uintptr_t>(x) & 15) || (reinterpret_cast<uintptr_t>(w) & 15))
@@ -949,7 +956,7 @@ DINFER_API int dinfer_gemm_tc_grouped(const void* x, int64_t ldx, const void* w,
   p.out = out; p.ldc = ldc; p.tokens = cap; p.N = N; p.K = K; p.status = status;
   p.k_blocks_per_split = (K + BLOCK_K - 1) / BLOCK_K; p.splits = 1;
   p.tile_expert = tile_expert; p.sorted = sorted; p.row_w = epi == 1 ? row_w : nullptr; p.pairs = pairs; p.grp_epi = epi; p.grp_act = act;
-  p.act = gate;
+  p.act = gate; p.a_pos = gate_a; p.a_neg = gate_b;
   CUtensorMap ma, mb;
   int rc;
   if ((rc = make_map(&ma, x, cap, K, ldx, TILE_M))) return rc;

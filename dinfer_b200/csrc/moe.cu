@@ -96,7 +96,7 @@ moe_route_kernel(const float* __restrict__ logits, int64_t ldz, int* __restrict_
 // ---------------------------------------------------------------- router that chooses by corrected scores
 // The scores as above over all E experts; an expert is chosen by score + correction[e], its weight is the score alone
 // (divided by the chosen ones' sum with renorm).  The experts form `groups` equal runs of neighbours; a run's rank is its
-// largest choice score, and only experts of the `keep` best runs can be chosen.  Equal choice scores go to the lower index.
+// largest choice score, or the sum of its two largest (rank_two), and only experts of the `keep` best runs can be chosen.  Equal choice scores go to the lower index.
 __device__ __forceinline__ void warp_best(float& best, int& arg) {
 #pragma unroll
   for (int o = 16; o > 0; o >>= 1) {
@@ -109,7 +109,7 @@ __device__ __forceinline__ void warp_best(float& best, int& arg) {
 __global__ void __launch_bounds__(RW * 32)
 moe_route_choice_kernel(const float* __restrict__ logits, int64_t ldz, const float* __restrict__ correction,
                         int* __restrict__ ids, float* __restrict__ weights, int T, int E, int top, int sigmoid_scores,
-                        int renorm, int groups, int keep) {
+                        int renorm, int groups, int keep, int rank_two) {
   extern __shared__ float sm[];                          // per warp: E scores, E choice scores, `groups` ranks
   pdl_enter();
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
@@ -130,14 +130,21 @@ moe_route_choice_kernel(const float* __restrict__ logits, int64_t ldz, const flo
     sum = warp_sum(sum);
     for (int e = lane; e < E; e += 32) z[e] = z[e] / sum;
   }
-  for (int e = lane; e < E; e += 32) c[e] = z[e] + (correction ? correction[e] : 0.f);
+  // without a correction a sigmoid's choice is made on the logits: scores that round to the same number (large logits all
+  // give 1) then still rank as the exact scores do
+  const bool by_logit = sigmoid_scores && !correction;
+  for (int e = lane; e < E; e += 32) c[e] = by_logit ? row[e] : z[e] + (correction ? correction[e] : 0.f);
   __syncwarp();
   if (keep < groups) {
     const int size = E / groups;
     for (int g = lane; g < groups; g += 32) {
-      float m = -INFINITY;
-      for (int i = 0; i < size; ++i) m = fmaxf(m, c[g * size + i]);
-      rank[g] = m;
+      float m = -INFINITY, m2 = -INFINITY;
+      for (int i = 0; i < size; ++i) {
+        const float v = by_logit && rank_two ? z[g * size + i] : c[g * size + i];
+        m2 = fmaxf(m2, fminf(m, v));
+        m = fmaxf(m, v);
+      }
+      rank[g] = rank_two && size > 1 ? m + m2 : m;
     }
     __syncwarp();
     for (int k = 0; k < keep; ++k) {
@@ -173,7 +180,7 @@ moe_route_choice_kernel(const float* __restrict__ logits, int64_t ldz, const flo
     __syncwarp();
   }
   if (renorm && lane == 0) {
-    const float inv = 1.f / chosen_sum;
+    const float inv = 1.f / (chosen_sum + 1e-20f);        // scores may all round to 0
     for (int k = 0; k < top; ++k) weights[(int64_t)t * top + k] *= inv;
   }
 }
@@ -543,18 +550,19 @@ DINFER_API int dinfer_moe_route(const float* logits, int64_t ldz, int* ids, floa
 }
 
 // logits [T, >= E] f32 rows of stride ldz; correction [E] f32 or null; groups divides E, keep <= groups, and the keep
-// best groups hold at least `top` experts; ids, weights [T, top].
+// best groups hold at least `top` experts; group_rank 1 or 2: a group ranks by its largest choice score or the sum of its
+// two largest (a sigmoid's scores then, also where the choice is made on the logits); ids, weights [T, top].
 DINFER_API int dinfer_moe_route_choice(const float* logits, int64_t ldz, const float* correction, int* ids, float* weights,
                                        int T, int E, int top, int sigmoid_scores, int renorm, int groups, int keep,
-                                       cudaStream_t stream) {
+                                       int group_rank, cudaStream_t stream) {
   if (T < 0 || E <= 0 || top <= 0 || groups <= 0 || E % groups || keep <= 0 || keep > groups ||
-      (int64_t)top > (int64_t)keep * (E / groups) || ldz < E)
+      (int64_t)top > (int64_t)keep * (E / groups) || ldz < E || (group_rank != 1 && group_rank != 2))
     return refuse(DINFER_BAD_ARGUMENT, "moe_route_choice: bad sizes T=%d E=%d top=%d groups=%d keep=%d", T, E, top, groups, keep);
   const size_t smem = (size_t)RW * (2 * E + groups) * sizeof(float);
   if (smem > 48 * 1024) return refuse(DINFER_BAD_ARGUMENT, "moe_route_choice: %d experts in %d groups are too many", E, groups);
   if (T == 0) return 0;
   launch_pdl(moe_route_choice_kernel, dim3((T + RW - 1) / RW), dim3(RW * 32), smem, stream, logits, ldz, correction, ids, weights,
-             T, E, top, sigmoid_scores, renorm, groups, keep);
+             T, E, top, sigmoid_scores, renorm, groups, keep, group_rank == 2);
   return cuda_status("moe_route_choice");
 }
 

@@ -704,3 +704,162 @@ DINFER_API int dinfer_qkv_post_general(void* qkv, int64_t ld, const int* positio
                                cache, slots, block_size, T, H, Hkv, D, Dv, Dc, bias, 0.f, 1, nullptr, 0, 0.f, act_dtype,
                                w_dtype, stream);
 }
+
+// One norm over all of q and one over all of k.  Per token: x = the projection's row [q: H * D | k: Hkv * D | v: Hkv * Dv]
+// (32-bit or the activations' type), q and k each divided by the root mean square over all their heads at once and
+// multiplied by a weight per row of the projection, then rotated by the position's angles; v times v_scale.  q goes to rows
+// of its own [T, H * D] in the activations' type, k and v to the token's slot of a cache [blocks, 2, Hkv, block_size, Dc].
+// The projection's row is only read, so it may be the 32-bit result of a product that feeds other parts too.
+namespace {
+
+constexpr int WHOLE_THREADS = 512;
+
+// V = 4: four neighbouring elements at a time (widths, strides and bases allow it), V = 1: one
+template <int V> struct Run { float x[V]; };
+template <typename T, int V> __device__ __forceinline__ Run<V> load_run(const T* p) {
+  Run<V> r;
+  if constexpr (V == 4 && sizeof(T) == 4) {
+    const float4 a = *reinterpret_cast<const float4*>(p);
+    r.x[0] = a.x; r.x[1] = a.y; r.x[2] = a.z; r.x[3] = a.w;
+  } else if constexpr (V == 4) {
+    const uint2 a = *reinterpret_cast<const uint2*>(p);
+    const __nv_bfloat162* h = reinterpret_cast<const __nv_bfloat162*>(&a);
+    const float2 f0 = __bfloat1622float2(h[0]), f1 = __bfloat1622float2(h[1]);
+    r.x[0] = f0.x; r.x[1] = f0.y; r.x[2] = f1.x; r.x[3] = f1.y;
+  } else {
+#pragma unroll
+    for (int i = 0; i < V; ++i) r.x[i] = to_f32<T>(p[i]);
+  }
+  return r;
+}
+template <typename T, int V> __device__ __forceinline__ void store_run(T* p, const Run<V>& r) {
+  if constexpr (V == 4 && sizeof(T) == 4) {
+    *reinterpret_cast<float4*>(p) = make_float4(r.x[0], r.x[1], r.x[2], r.x[3]);
+  } else if constexpr (V == 4) {
+    uint2 a;
+    __nv_bfloat162* h = reinterpret_cast<__nv_bfloat162*>(&a);
+    h[0] = __floats2bfloat162_rn(r.x[0], r.x[1]);
+    h[1] = __floats2bfloat162_rn(r.x[2], r.x[3]);
+    *reinterpret_cast<uint2*>(p) = a;
+  } else {
+#pragma unroll
+    for (int i = 0; i < V; ++i) p[i] = from_f32<T>(r.x[i]);
+  }
+}
+
+template <typename TI, typename TA, int V>
+__global__ void __launch_bounds__(WHOLE_THREADS)
+qkv_post_whole_kernel(const TI* __restrict__ qkv, int64_t ld, const int* __restrict__ positions,
+                      const float* __restrict__ q_weight, const float* __restrict__ k_weight, float eps,
+                      const float* __restrict__ cos_sin, int rot, int interleaved, float v_scale, TA* __restrict__ q_out,
+                      TA* __restrict__ cache, const int* __restrict__ slots, int block_size, int H, int Hkv, int D, int Dv,
+                      int Dc) {
+  __shared__ float red[2][WHOLE_THREADS / 32];
+  __shared__ float inv[2];
+  pdl_launch_dependents();
+  const int t = blockIdx.x, tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
+  const int64_t pos = positions[t];
+  const int slot = (cache && slots) ? slots[t] : -1;
+  pdl_wait();
+  const TI* row = qkv + (int64_t)t * ld;
+  const int nq = H * D, nk = Hkv * D, nv = Hkv * Dv;
+  if (q_weight) {
+    float sq = 0.f, sk = 0.f;
+    for (int i = tid * V; i < nq + nk; i += WHOLE_THREADS * V) {     // (a run lies in q or in k: both are whole runs)
+      const Run<V> a = load_run<TI, V>(row + i);
+      float s = 0.f;
+#pragma unroll
+      for (int j = 0; j < V; ++j) s = fmaf(a.x[j], a.x[j], s);
+      if (i < nq) sq += s; else sk += s;
+    }
+    sq = warp_sum(sq);
+    sk = warp_sum(sk);
+    if (lane == 0) { red[0][warp] = sq; red[1][warp] = sk; }
+    __syncthreads();
+    if (warp < 2) {
+      const float v = warp_sum(lane < WHOLE_THREADS / 32 ? red[warp][lane] : 0.f);
+      if (lane == 0) inv[warp] = 1.f / sqrtf(v / (float)(warp == 0 ? nq : nk) + eps);
+    }
+    __syncthreads();
+  }
+  const int half = cos_sin ? rot >> 1 : 0;
+  const float* cs = cos_sin + pos * rot;
+  const int64_t blk = slot >= 0 ? slot / block_size : 0, off = slot >= 0 ? slot % block_size : 0;
+  // a head's work: its pairs of runs (e, e + half), then the runs that pass unturned
+  const int pairs = half / V, units = pairs + (D - 2 * half) / V;
+  auto normed = [&](int i) {
+    Run<V> a = load_run<TI, V>(row + i);
+    if (q_weight) {
+      const bool is_q = i < nq;
+      const Run<V> w = load_run<float, V>(is_q ? q_weight + i : k_weight + (i - nq));
+      const float r = inv[is_q ? 0 : 1];
+#pragma unroll
+      for (int j = 0; j < V; ++j) a.x[j] = a.x[j] * r * w.x[j];
+    }
+    return a;
+  };
+  for (int w = tid; w < (H + Hkv) * units; w += WHOLE_THREADS) {
+    const int head = w / units, u = w - head * units;
+    TA* dst = nullptr;
+    if (head < H) dst = q_out + (int64_t)t * nq + (int64_t)head * D;
+    else if (slot >= 0) dst = cache + ((blk * 2 * Hkv + (head - H)) * block_size + off) * Dc;
+    if (!dst) continue;
+    if (u < pairs) {
+      // in halves: elements e.. and e + half..; interleaved (V = 1 only): elements 2 u and 2 u + 1
+      const int e0 = interleaved ? 2 * u : u * V, e1 = interleaved ? 2 * u + 1 : u * V + half;
+      const Run<V> a = normed(head * D + e0), b = normed(head * D + e1);
+      const Run<V> c = load_run<float, V>(cs + u * V), s = load_run<float, V>(cs + half + u * V);
+      Run<V> x, y;
+#pragma unroll
+      for (int j = 0; j < V; ++j) {
+        x.x[j] = a.x[j] * c.x[j] - b.x[j] * s.x[j];
+        y.x[j] = b.x[j] * c.x[j] + a.x[j] * s.x[j];
+      }
+      store_run<TA, V>(dst + e0, x);
+      store_run<TA, V>(dst + e1, y);
+    } else {
+      const int e = 2 * half + (u - pairs) * V;
+      store_run<TA, V>(dst + e, normed(head * D + e));
+    }
+  }
+  if (slot >= 0)
+    for (int i = tid * V; i < nv; i += WHOLE_THREADS * V) {
+      Run<V> a = load_run<TI, V>(row + nq + nk + i);
+#pragma unroll
+      for (int j = 0; j < V; ++j) a.x[j] *= v_scale;
+      const int hk = i / Dv;
+      store_run<TA, V>(cache + (((blk * 2 + 1) * Hkv + hk) * block_size + off) * Dc + (i - hk * Dv), a);
+    }
+}
+
+}  // namespace
+
+// qkv [T, >= (H + Hkv) D + Hkv Dv] rows of stride ld in in_dtype; q_weight [H * D] / k_weight [Hkv * D] f32 (both null: no
+// norm); cos_sin [positions, rot] f32 or null; q_out [T, H * D] contiguous; cache rows Dc = max(D, Dv) wide.
+DINFER_API int dinfer_qkv_post_whole(const void* qkv, int64_t ld, const int* positions, const float* q_weight,
+                                     const float* k_weight, float eps, const float* cos_sin, int rot, int interleaved,
+                                     float v_scale, void* q_out, void* cache, const int* slots, int block_size, int T, int H,
+                                     int Hkv, int D, int Dv, int Dc, int in_dtype, int act_dtype, cudaStream_t stream) {
+  if (T < 0 || H <= 0 || Hkv <= 0 || D <= 0 || Dv <= 0 || Dc < D || Dc < Dv || !q_out)
+    return refuse(DINFER_BAD_ARGUMENT, "qkv_post_whole: bad sizes T=%d H=%d Hkv=%d D=%d Dv=%d Dc=%d", T, H, Hkv, D, Dv, Dc);
+  if (cos_sin && (rot <= 0 || rot > D || (rot & 1)))
+    return refuse(DINFER_BAD_ARGUMENT, "qkv_post_whole: rotary dim %d must be even and at most head_dim %d", rot, D);
+  if (ld < (int64_t)(H + Hkv) * D + (int64_t)Hkv * Dv) return refuse(DINFER_BAD_ARGUMENT, "qkv_post_whole: row stride below the row's width");
+  if (cache && (block_size <= 0 || !slots)) return refuse(DINFER_BAD_ARGUMENT, "qkv_post_whole: a cache needs slots and block_size, got %d", block_size);
+  if ((q_weight == nullptr) != (k_weight == nullptr)) return refuse(DINFER_BAD_ARGUMENT, "qkv_post_whole: q and k norm weights come together");
+  if (T == 0) return 0;
+  const auto al16 = [](const void* q) { return (reinterpret_cast<uintptr_t>(q) & 15) == 0; };
+  const bool vec = D % 8 == 0 && Dv % 4 == 0 && Dc % 4 == 0 && ld % 4 == 0 && (!cos_sin || (rot % 8 == 0 && !interleaved)) &&
+                   al16(qkv) && al16(q_out) && al16(cache) && al16(q_weight) && al16(k_weight) && al16(cos_sin);
+#define GO(TI, TA, V)                                                                                                      \
+  launch_pdl(qkv_post_whole_kernel<TI, TA, V>, dim3(T), dim3(WHOLE_THREADS), 0, stream, (const TI*)qkv, ld, positions,     \
+             q_weight, k_weight, eps, cos_sin, rot, interleaved, v_scale, (TA*)q_out, (TA*)cache, slots, block_size, H, Hkv, \
+             D, Dv, Dc)
+  DINFER_DISPATCH_DTYPE(in_dtype, TI,
+    DINFER_DISPATCH_DTYPE(act_dtype, TA, {
+      if (vec) GO(TI, TA, 4); else GO(TI, TA, 1);
+      return cuda_status("qkv_post_whole");
+    }));
+#undef GO
+  return 0;
+}

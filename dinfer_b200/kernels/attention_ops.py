@@ -62,12 +62,13 @@ def attention_decode(q: torch.Tensor, out: torch.Tensor, cache: torch.Tensor, bl
                      cu_seqlens: torch.Tensor, seq_lens: torch.Tensor, num_heads: int, num_kv_heads: int,
                      head_dim: int, scale: float, window: int, splits: int, sink: bool = False,
                      slopes: Optional[torch.Tensor] = None, chunked: bool = False,
-                     sinks: Optional[torch.Tensor] = None) -> torch.Tensor:
+                     sinks: Optional[torch.Tensor] = None, keep_first: int = 0, softcap: float = 0.0) -> torch.Tensor:
     """Attention of the requests that bring exactly one token (the others are skipped), keys split
     ``splits`` ways; the splits are folded inside the kernel.  ``sink``: one more softmax term of score 0 without a
     value, of score ``sinks[h]`` where that is given (f32 [H]); ``slopes`` (f32 [H]): a distance bias ``score_ij -
-    slopes[h] * (i - j)``; ``chunked``: a token sees the keys of its own chunk of ``window`` positions (all of them:
-    pages of at least 8 tokens only)."""
+    slopes[h] * (i - j)``; ``chunked``: a token sees the keys of its own chunk of ``window`` positions;
+    ``keep_first``: with a window, the first so many keys of a request are seen from everywhere; ``softcap`` > 0: a score
+    is ``softcap * tanh(score / softcap)``, ahead of the bias (all of them: pages of at least 8 tokens only)."""
     require_cuda(q, out, cache, block_table, cu_seqlens, seq_lens, slopes, sinks)
     sink = _check_heads(num_heads, slopes, sinks) or sink
     if q.dtype != torch.bfloat16 or out.dtype != torch.bfloat16 or cache.dtype != torch.bfloat16:
@@ -87,15 +88,15 @@ def attention_decode(q: torch.Tensor, out: torch.Tensor, cache: torch.Tensor, bl
         status = gemm_ops._state(q.device)["status"]
         lib, f = _fn("attention_decode", "dinfer_attention_decode_tma_bias",
                      [c_void_p, c_int64, c_void_p, c_int64, c_void_p, c_int64, c_void_p, c_int, c_void_p, c_void_p,
-                      c_int, c_int, c_int, c_int, c_int, c_float, c_int, c_int, c_int, c_void_p, c_void_p, c_int, c_void_p,
-                      c_void_p])
+                      c_int, c_int, c_int, c_int, c_int, c_float, c_int, c_int, c_int, c_float, c_int, c_void_p, c_void_p,
+                      c_int, c_void_p, c_void_p])
         check(lib, f(ptr(q), q.stride(0), ptr(out), out.stride(0), ptr(cache), cache.shape[0], ptr(block_table),
                      block_table.shape[1], ptr(cu_seqlens), ptr(seq_lens), B, num_heads, num_kv_heads, head_dim,
-                     cache.shape[3], float(scale), int(window), int(bool(chunked)), int(bool(sink)), ptr(sinks), ptr(slopes), min(int(splits), MAX_CLUSTER_SPLITS),
+                     cache.shape[3], float(scale), int(window), int(bool(chunked)), int(keep_first or 0), float(softcap or 0.0), int(bool(sink)), ptr(sinks), ptr(slopes), min(int(splits), MAX_CLUSTER_SPLITS),
                      ptr(status), stream_handle()), "attention_decode_tma")
         return out
-    if sink or slopes is not None or chunked:
-        raise KernelError("attention_decode: the sink, the distance bias and chunks need pages of at least 8 tokens")
+    if sink or slopes is not None or chunked or keep_first or softcap:
+        raise KernelError("attention_decode: the sink, the distance bias, chunks, kept keys and the soft cap need pages of at least 8 tokens")
     floats = counters = None
     if splits > 1:
         floats, counters = _decode_scratch(q.device, B * num_heads * splits * (head_dim + 2), B * num_kv_heads)
@@ -179,14 +180,14 @@ def attention_umma(q: torch.Tensor, out: torch.Tensor, cache: torch.Tensor, bloc
                    cu_seqlens: torch.Tensor, seq_lens: torch.Tensor, num_heads: int, num_kv_heads: int,
                    head_dim: int, scale: float, window: int, max_q_len: int, key_splits: int = 1,
                    pair_bound: int = 0, sink: bool = False, slopes: Optional[torch.Tensor] = None, chunked: bool = False,
-                   sinks: Optional[torch.Tensor] = None) -> torch.Tensor:
+                   sinks: Optional[torch.Tensor] = None, keep_first: int = 0, softcap: float = 0.0) -> torch.Tensor:
     """Attention of the prompt portions of the batch (requests with more than one token; the others
     are skipped) on tcgen05 / TMEM / TMA.  ``q``: the [T, H*D] columns of the step's rows (a view with a
     row stride is fine).  ``key_splits``: see ``umma_key_splits``; ``pair_bound``: see ``umma_pair_bound``
     (0: every request is taken for the longest portion); ``slopes`` (f32 [H]): a distance bias
-    ``score_ij - slopes[h] * (i - j)``; ``chunked``, ``sinks``: see ``attention_decode``."""
+    ``score_ij - slopes[h] * (i - j)``; ``chunked``, ``sinks``, ``keep_first``, ``softcap``: see ``attention_decode``."""
     _umma_launch(False, q, out, cache, block_table, cu_seqlens, seq_lens, num_heads, num_kv_heads, head_dim, scale,
-                 window, max_q_len, key_splits, pair_bound, sink, slopes, chunked, sinks)
+                 window, max_q_len, key_splits, pair_bound, sink, slopes, chunked, sinks, keep_first, softcap)
     return out
 
 
@@ -194,15 +195,16 @@ def attention_umma64(q: torch.Tensor, out: torch.Tensor, cache: torch.Tensor, bl
                      cu_seqlens: torch.Tensor, seq_lens: torch.Tensor, num_heads: int, num_kv_heads: int,
                      head_dim: int, scale: float, window: int, max_q_len: int, pair_bound: int = 0,
                      sink: bool = False, slopes: Optional[torch.Tensor] = None, chunked: bool = False,
-                     sinks: Optional[torch.Tensor] = None) -> torch.Tensor:
+                     sinks: Optional[torch.Tensor] = None, keep_first: int = 0, softcap: float = 0.0) -> torch.Tensor:
     """The same attention through the kernel with 64-key tiles (``UMMA_SHORT_CONTEXT``); no key split."""
     _umma_launch(True, q, out, cache, block_table, cu_seqlens, seq_lens, num_heads, num_kv_heads, head_dim, scale,
-                 window, max_q_len, 1, pair_bound, sink, slopes, chunked, sinks)
+                 window, max_q_len, 1, pair_bound, sink, slopes, chunked, sinks, keep_first, softcap)
     return out
 
 
 def _umma_launch(short, q, out, cache, block_table, cu_seqlens, seq_lens, num_heads, num_kv_heads, head_dim, scale,
-                 window, max_q_len, key_splits, pair_bound, sink=False, slopes=None, chunked=False, sinks=None) -> None:
+                 window, max_q_len, key_splits, pair_bound, sink=False, slopes=None, chunked=False, sinks=None,
+                 keep_first=0, softcap=0.0) -> None:
     from . import gemm_ops
     require_cuda(q, out, cache, block_table, cu_seqlens, seq_lens, slopes, sinks)
     sink = _check_heads(num_heads, slopes, sinks) or sink
@@ -219,10 +221,11 @@ def _umma_launch(short, q, out, cache, block_table, cu_seqlens, seq_lens, num_he
     status = gemm_ops._state(q.device)["status"]
     head = (ptr(q), q.stride(0), ptr(out), out.stride(0), ptr(cache), cache.shape[0], ptr(block_table),
             block_table.shape[1], ptr(cu_seqlens), ptr(seq_lens), q.shape[0], B, num_heads, num_kv_heads,
-            head_dim, cache.shape[3], float(scale), int(window), int(bool(chunked)), int(bool(sink)), ptr(sinks), ptr(slopes),
+            head_dim, cache.shape[3], float(scale), int(window), int(bool(chunked)), int(keep_first or 0), float(softcap or 0.0), int(bool(sink)), ptr(sinks), ptr(slopes),
             int(max_q_len), int(pair_bound))
     types = [c_void_p, c_int64, c_void_p, c_int64, c_void_p, c_int64, c_void_p, c_int, c_void_p, c_void_p,
-             c_int, c_int, c_int, c_int, c_int, c_int, c_float, c_int, c_int, c_int, c_void_p, c_void_p, c_int, c_int]
+             c_int, c_int, c_int, c_int, c_int, c_int, c_float, c_int, c_int, c_int, c_float, c_int, c_void_p, c_void_p,
+             c_int, c_int]
     if short:
         lib, f = _fn("attention_umma64", "dinfer_attention_umma64_bias", types + [c_void_p, c_void_p])
         check(lib, f(*head, ptr(status), stream_handle()), "attention_umma64")
@@ -236,11 +239,11 @@ def attention_tc(q: torch.Tensor, out: torch.Tensor, cache: torch.Tensor, block_
                  head_dim: int, scale: float, window: int, max_q_len: int, any_decode: bool,
                  any_prefill: bool, splits: int, scratch: Optional[torch.Tensor] = None,
                  sink: bool = False, slopes: Optional[torch.Tensor] = None, chunked: bool = False,
-                 sinks: Optional[torch.Tensor] = None) -> torch.Tensor:
+                 sinks: Optional[torch.Tensor] = None, keep_first: int = 0, softcap: float = 0.0) -> torch.Tensor:
     """Paged causal attention on the tensor cores.  ``q`` / ``out``: rows with a contiguous last axis,
     head h at columns [h*D, (h+1)*D).  ``splits`` > 1 needs ``scratch`` (f32) of
     ``B * H * splits * (D + 2)`` elements; it is allocated here when not given.  ``slopes`` (f32 [H]): a distance
-    bias, ``score_ij - slopes[h] * (i - j)``; ``chunked``, ``sinks``: see ``attention_decode``."""
+    bias, ``score_ij - slopes[h] * (i - j)``; ``chunked``, ``sinks``, ``keep_first``, ``softcap``: see ``attention_decode``."""
     require_cuda(q, out, cache, block_table, cu_seqlens, seq_lens, slopes, sinks)
     sink = _check_heads(num_heads, slopes, sinks) or sink
     if q.dtype != torch.bfloat16 or out.dtype != torch.bfloat16 or cache.dtype != torch.bfloat16:
@@ -261,11 +264,11 @@ def attention_tc(q: torch.Tensor, out: torch.Tensor, cache: torch.Tensor, block_
         raise KernelError("attention_tc: scratch too small")
     lib, f = _fn("attention_tc", "dinfer_attention_tc_bias",
                  [c_void_p, c_int64, c_void_p, c_int64, c_void_p, c_void_p, c_int, c_void_p, c_void_p,
-                  c_int, c_int, c_int, c_int, c_int, c_float, c_int, c_int, c_int, c_void_p, c_void_p, c_int, c_int, c_int,
-                  c_int, c_void_p, c_void_p])
+                  c_int, c_int, c_int, c_int, c_int, c_float, c_int, c_int, c_int, c_float, c_int, c_void_p, c_void_p,
+                  c_int, c_int, c_int, c_int, c_void_p, c_void_p])
     check(lib, f(ptr(q), q.stride(0), ptr(out), out.stride(0), ptr(cache), ptr(block_table), block_table.shape[1],
                  ptr(cu_seqlens), ptr(seq_lens), B, num_heads, num_kv_heads, head_dim, cache.shape[3],
-                 float(scale), int(window), int(bool(chunked)), int(bool(sink)), ptr(sinks), ptr(slopes), int(max_q_len),
+                 float(scale), int(window), int(bool(chunked)), int(keep_first or 0), float(softcap or 0.0), int(bool(sink)), ptr(sinks), ptr(slopes), int(max_q_len),
                  int(any_decode), int(any_prefill), int(splits),
                  ptr(scratch if splits > 1 else None), stream_handle()), "attention_tc")
     return out

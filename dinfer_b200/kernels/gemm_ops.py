@@ -7,7 +7,7 @@ from typing import Optional
 import torch
 
 from .lib import KernelError, check, num_sms, ptr, require_cuda, stream_handle
-from .ops import _fn
+from .ops import _fn, gate_constants
 
 DECODE_MAX_TOKENS = 64          # up to here the operands are swapped (weight rows fill the tile)
 MAX_SPLITS = 8                  # the portable cluster size
@@ -110,8 +110,8 @@ def decode_splits(tokens: int, N: int, K: int) -> int:
     return max(1, min(slots // tiles, k_blocks // 8, MAX_SPLITS))
 
 
-# the gates the product's epilogue knows
-GATES = {False: 0, None: 0, True: 1, "silu": 1, "gelu_tanh": 2}
+# the gates the product's epilogue knows; the clamped gate comes with its constants (see ops.gate_constants)
+GATES = {False: 0, None: 0, True: 1, "silu": 1, "gelu_tanh": 2, "clamped_swish": 3}
 # the activations it knows without a gate; an xIELU comes as ("xielu", a_pos, a_neg)
 UNARY = {None: 0, "relu2": 1, "silu": 2, "gelu_tanh": 3, "relu": 4, "xielu": 5}
 
@@ -121,7 +121,7 @@ def gemm_tc(x: torch.Tensor, w: torch.Tensor, out: torch.Tensor, splits: Optiona
             sums: Optional[torch.Tensor] = None, row_scale=None, activation=None) -> torch.Tensor:
     """out[tokens, N] = x[tokens, K] @ w[N, K]^T.  out: bfloat16 or float32, last axis contiguous.
 
-    ``gated`` (any number of rows; True or "silu", or "gelu_tanh"): the rows of w are (gate, up) pairs, out is
+    ``gated`` (any number of rows; True or "silu", "gelu_tanh", or a clamped gate with its constants): the rows of w are (gate, up) pairs, out is
     [tokens, N / 2], out[t, j] = g(x w_2j) * (x w_2j+1) with that g.
     ``activation`` (any number of rows; no gate, no residual): a key of ``UNARY`` or ("xielu", a_pos, a_neg), applied to
     the result.
@@ -136,11 +136,12 @@ def gemm_tc(x: torch.Tensor, w: torch.Tensor, out: torch.Tensor, splits: Optiona
         raise KernelError("gemm_tc: bfloat16 operands with K and row strides multiples of 8 and 16-byte aligned bases")
     tokens, K = x.shape
     N = w.shape[0]
+    gated, gate_a, gate_b = gate_constants(gated)
     if gated not in GATES:
         raise KernelError(f"gemm_tc: unknown gate {gated!r}")
     if (residual is not None or row_scale is not None) and tokens > DECODE_MAX_TOKENS:
         raise KernelError("gemm_tc: the norm epilogues take at most 64 rows")
-    unary, a_pos, a_neg = activation if isinstance(activation, (tuple, list)) else (activation, 0.0, 0.0)
+    unary, a_pos, a_neg = activation if isinstance(activation, (tuple, list)) else (activation, gate_a, gate_b)
     if unary not in UNARY or (unary == "xielu") != isinstance(activation, (tuple, list)) or (unary and (gated or residual is not None)):
         raise KernelError(f"gemm_tc: activation {activation!r}: one of {', '.join(str(k) for k in UNARY)}, without a gate or a residual")
     if gated and (N % 2 or residual is not None):

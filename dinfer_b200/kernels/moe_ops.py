@@ -36,10 +36,10 @@ def route(logits: torch.Tensor, num_experts: int, top_k: int, scoring: str = "so
 
 def route_choice(logits: torch.Tensor, num_experts: int, top_k: int, correction: Optional[torch.Tensor] = None,
                  scoring: str = "softmax", renormalize: bool = False, groups: int = 1,
-                 keep: int = 1) -> Tuple[torch.Tensor, torch.Tensor]:
+                 keep: int = 1, group_rank: int = 1) -> Tuple[torch.Tensor, torch.Tensor]:
     """(expert ids int32 [T, top_k], weights f32 [T, top_k]) of a router that chooses by ``score + correction[e]`` (f32
     [num_experts]) and weighs by the score alone: the experts form ``groups`` equal runs of neighbours, a run ranks by
-    its largest choice score, and only the ``keep`` best runs' experts can be chosen."""
+    the sum of its ``group_rank`` (1 or 2) largest choice scores, and only the ``keep`` best runs' experts can be chosen."""
     require_cuda(logits, correction)
     _rows_contiguous(logits, "moe route_choice")
     T = logits.shape[0]
@@ -52,9 +52,9 @@ def route_choice(logits: torch.Tensor, num_experts: int, top_k: int, correction:
     ids = torch.empty((T, top_k), dtype=torch.int32, device=logits.device)
     weights = torch.empty((T, top_k), dtype=torch.float32, device=logits.device)
     lib, f = _fn("moe", "dinfer_moe_route_choice",
-                 [c_void_p, c_int64, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_void_p])
+                 [c_void_p, c_int64, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_void_p])
     check(lib, f(ptr(logits), logits.stride(0), ptr(correction), ptr(ids), ptr(weights), T, num_experts, top_k,
-                 int(scoring == "sigmoid"), int(bool(renormalize)), int(groups), int(keep), stream_handle()), "moe_route_choice")
+                 int(scoring == "sigmoid"), int(bool(renormalize)), int(groups), int(keep), int(group_rank), stream_handle()), "moe_route_choice")
     return ids, weights
 
 
@@ -124,10 +124,12 @@ def grouped_gemm_tc(a: torch.Tensor, w: torch.Tensor, out: torch.Tensor, sorted_
                     gate: Optional[str] = None) -> torch.Tensor:
     """The grouped product on the two-SM tcgen05 kernel (bfloat16; the layout padded to ``TC_ROW_TILE`` rows per
     expert run).  a [cap, K] by position.  mode 0: ``out[pos] = act(a[pos] @ w[e]^T)`` (out [cap, N]); mode 1:
-    ``out[pair] = (a[pos] @ w[e]^T) * weights[pair]`` (out [pairs, N]).  ``gate`` (mode 0; "silu" or "gelu_tanh"): the rows
+    ``out[pair] = (a[pos] @ w[e]^T) * weights[pair]`` (out [pairs, N]).  ``gate`` (mode 0; "silu", "gelu_tanh" or a clamped gate with its constants): the rows
     of w[e] are (gate, up) pairs and out is [cap, N / 2], act(gate) * up."""
     from . import gemm_ops
+    from .ops import gate_constants
     require_cuda(a, w, out, sorted_, tile_expert, weights)
+    gate, gate_a, gate_b = gate_constants(gate)
     E, N, K = w.shape
     cap = sorted_.numel()
     if gate is not None and (gate not in gemm_ops.GATES or mode != 0 or activation != "none" or N % 2):
@@ -142,9 +144,9 @@ def grouped_gemm_tc(a: torch.Tensor, w: torch.Tensor, out: torch.Tensor, sorted_
     st = gemm_ops._state(a.device)
     lib, f = _fn("gemm_tc", "dinfer_gemm_tc_grouped",
                  [c_void_p, c_int64, c_void_p, c_void_p, c_int64, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int,
-                  c_int, c_int, c_int, c_int, c_void_p, c_void_p])
+                  c_int, c_int, c_int, c_int, c_float, c_float, c_void_p, c_void_p])
     check(lib, f(ptr(a), a.stride(0), ptr(w), ptr(out), out.stride(0), ptr(tile_expert), ptr(sorted_), ptr(weights), cap,
-                 pairs, E, N, K, int(mode), ACTIVATIONS[activation], gemm_ops.GATES[gate], ptr(st["status"]), stream_handle()), "gemm_tc_grouped")
+                 pairs, E, N, K, int(mode), ACTIVATIONS[activation], gemm_ops.GATES[gate], gate_a, gate_b, ptr(st["status"]), stream_handle()), "gemm_tc_grouped")
     return out
 
 

@@ -263,13 +263,15 @@ def attention_generic(q: torch.Tensor, out: torch.Tensor, cache: torch.Tensor, b
                       cu_seqlens: torch.Tensor, positions: torch.Tensor, num_heads: int, num_kv_heads: int,
                       head_dim: int, scale: float, window: int = 0, v_dim: Optional[int] = None,
                       sink: bool = False, slopes: Optional[torch.Tensor] = None, chunked: bool = False,
-                      sinks: Optional[torch.Tensor] = None) -> torch.Tensor:
+                      sinks: Optional[torch.Tensor] = None, keep_first: int = 0, softcap: float = 0.0) -> torch.Tensor:
     """Paged causal attention, plain arithmetic, any head size.  ``q`` may be a strided view (for
     instance the q columns of the qkv rows).  ``v_dim``: the values' width where it differs from the keys' (the
     cache's rows are then ``max(head_dim, v_dim)`` wide, ``out`` holds head h at ``h * v_dim``); ``sink``: one more
     term without a value in the softmax's denominator, of score 0 or, where ``sinks`` (f32 [H]) is given, ``sinks[h]``;
     ``slopes`` (f32 [H]): a distance bias, ``score_ij - slopes[h] * (i - j)``; ``chunked``: a token sees the keys of its
-    own chunk of ``window`` positions, counted from the sequence's first."""
+    own chunk of ``window`` positions, counted from the sequence's first; ``keep_first``: with a window, the first so many
+    keys of a request are seen from everywhere; ``softcap`` > 0: a score is ``softcap * tanh(score / softcap)``, ahead of
+    the bias."""
     require_cuda(q, out, cache, block_table, cu_seqlens, positions, slopes, sinks)
     for t, n in ((slopes, "slopes"), (sinks, "sinks")):
         if t is not None and (t.dtype != torch.float32 or t.numel() != num_heads or not t.is_contiguous()):
@@ -293,12 +295,12 @@ def attention_generic(q: torch.Tensor, out: torch.Tensor, cache: torch.Tensor, b
         raise KernelError(f"attention: cache shape {tuple(cache.shape)} is not [blocks, 2, Hkv, block, {row}]")
     lib, f = _fn("attention_generic", "dinfer_attention_generic_bias",
                  [c_void_p, c_int64, c_void_p, c_int64, c_void_p, c_void_p, c_int, c_void_p, c_void_p,
-                  c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_float, c_int, c_int, c_int, c_void_p, c_void_p,
-                  c_int, c_void_p])
+                  c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_float, c_int, c_int, c_int, c_float, c_int, c_void_p,
+                  c_void_p, c_int, c_void_p])
     check(lib, f(ptr(q), q.stride(0), ptr(out), out.stride(0), ptr(cache), ptr(block_table),
                  block_table.shape[1], ptr(cu_seqlens), ptr(positions), T, B, num_heads, num_kv_heads,
-                 head_dim, v_dim, row, cache.shape[3], float(scale), int(window), int(bool(chunked)), int(bool(sink)),
-                 ptr(sinks), ptr(slopes), dtype_code(q.dtype), stream_handle()), "attention_generic")
+                 head_dim, v_dim, row, cache.shape[3], float(scale), int(window), int(bool(chunked)), int(keep_first or 0),
+                 float(softcap or 0.0), int(bool(sink)), ptr(sinks), ptr(slopes), dtype_code(q.dtype), stream_handle()), "attention_generic")
     return out
 
 
@@ -356,6 +358,46 @@ def qkv_post_general(qkv: torch.Tensor, positions: torch.Tensor, num_heads: int,
                  block_size, T, num_heads, num_kv_heads, head_dim, v_dim, row, ptr(bias), coef, every, ptr(v_first),
                  v_first.stride(0) if v_first is not None else 0, float(v_lambda), dtype_code(qkv.dtype), dtype_code(w_dt),
                  stream_handle()), "qkv_post_general")
+
+
+def qkv_post_whole(qkv: torch.Tensor, positions: torch.Tensor, num_heads: int, num_kv_heads: int, head_dim: int,
+                   v_dim: int, eps: float, q_weight: Optional[torch.Tensor], k_weight: Optional[torch.Tensor],
+                   cos_sin: Optional[torch.Tensor], q_out: torch.Tensor, cache: Optional[torch.Tensor],
+                   slots: Optional[torch.Tensor], block_size: int, interleaved: bool = False, v_scale: float = 1.0) -> torch.Tensor:
+    """q/k/v post-processing with one RMS norm over all of q and one over all of k (``q_weight`` f32 [H * D], ``k_weight``
+    f32 [Hkv * D]; None: no norm), a rotation by ``cos_sin``, ``v_scale`` times v.  ``qkv`` (rows with a stride are fine;
+    float32 or the activations' dtype) is only read; q goes to ``q_out`` [T, H * D], k and v into the cache."""
+    require_cuda(qkv, positions, q_weight, k_weight, cos_sin, q_out, cache, slots)
+    _rows_contiguous(qkv, "qkv_post_whole")
+    T = qkv.shape[0]
+    row = max(head_dim, v_dim)
+    if positions.dtype != torch.int32 or positions.numel() != T:
+        raise KernelError("qkv_post_whole: positions int32 [T]")
+    if qkv.shape[1] < (num_heads + num_kv_heads) * head_dim + num_kv_heads * v_dim or qkv.dtype not in (torch.float32, q_out.dtype):
+        raise KernelError("qkv_post_whole: qkv [T, (H + Hkv) D + Hkv Dv], float32 or the activations' dtype")
+    if tuple(q_out.shape) != (T, num_heads * head_dim) or not q_out.is_contiguous():
+        raise KernelError("qkv_post_whole: q_out [T, H * D] contiguous")
+    for w, n in ((q_weight, num_heads * head_dim), (k_weight, num_kv_heads * head_dim)):
+        if w is not None and (w.dtype != torch.float32 or w.numel() != n or not w.is_contiguous()):
+            raise KernelError("qkv_post_whole: norm weights contiguous float32, one number per row of q / k")
+    rot = 0
+    if cos_sin is not None:
+        if cos_sin.dtype != torch.float32 or not cos_sin.is_contiguous() or cos_sin.dim() != 2:
+            raise KernelError("qkv_post_whole: angle table must be contiguous float32 [max_pos, rot]")
+        rot = cos_sin.shape[1]
+    if cache is not None:
+        if cache.dtype != q_out.dtype or not cache.is_contiguous() or slots is None or slots.dtype != torch.int32 \
+                or slots.numel() != T or tuple(cache.shape[1:]) != (2, num_kv_heads, block_size, row):
+            raise KernelError(f"qkv_post_whole: cache [blocks, 2, {num_kv_heads}, {block_size}, {row}] of the "
+                              f"activations' dtype, contiguous; slots int32 [T]")
+    lib, f = _fn("qk_post", "dinfer_qkv_post_whole",
+                 [c_void_p, c_int64, c_void_p, c_void_p, c_void_p, c_float, c_void_p, c_int, c_int, c_float, c_void_p, c_void_p,
+                  c_void_p, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_void_p])
+    check(lib, f(ptr(qkv), qkv.stride(0), ptr(positions), ptr(q_weight), ptr(k_weight), float(eps), ptr(cos_sin), rot,
+                 int(bool(interleaved)), float(v_scale), ptr(q_out), ptr(cache), ptr(slots), block_size, T, num_heads,
+                 num_kv_heads, head_dim, v_dim, row, dtype_code(qkv.dtype), dtype_code(q_out.dtype), stream_handle()),
+          "qkv_post_whole")
+    return q_out
 
 
 def heads_out(x: torch.Tensor, positions: torch.Tensor, num_heads: int, v_dim: int, cos_sin: Optional[torch.Tensor] = None,
@@ -480,13 +522,28 @@ def scaled_add(residual: torch.Tensor, deltas) -> torch.Tensor:
     return residual
 
 
-GATE_ACTIVATIONS = {"silu": 0, "gelu_tanh": 1, "relu": 2, "relu2": 3}
+GATE_ACTIVATIONS = {"silu": 0, "gelu_tanh": 1, "relu": 2, "relu2": 3, "clamped_swish": 4}
+
+
+def gate_constants(activation):
+    """(name, a, b) of a gate: a plain name, or a tuple of a name and its constants: ("clamped_swish", limit, alpha) is
+    ``g sigmoid(alpha g) (u + 1)`` with ``g = min(gate, limit)``, ``u = clamp(up, -limit, limit)``."""
+    if isinstance(activation, (tuple, list)):
+        name, a, b = activation
+        if name != "clamped_swish" or not a > 0:
+            raise KernelError(f"gate {activation!r}: only clamped_swish takes constants, and its limit is positive")
+        return name, float(a), float(b)
+    if activation == "clamped_swish":
+        raise KernelError("gate: clamped_swish comes as (name, limit, alpha)")
+    return activation, 0.0, 0.0
 
 
 def gated_act(x: torch.Tensor, out: torch.Tensor, activation: str = "silu", pairs: bool = False) -> torch.Tensor:
-    """out[t, i] = act(gate_i) * up_i; the layouts of ``silu_mul``; ``activation`` a key of ``GATE_ACTIVATIONS``."""
+    """out[t, i] = act(gate_i) * up_i; the layouts of ``silu_mul``; ``activation`` a key of ``GATE_ACTIVATIONS``
+    (with its constants as ``gate_constants`` says)."""
     if activation == "silu":
         return silu_mul(x, out, pairs)
+    activation, ga, gb = gate_constants(activation)
     require_cuda(x, out)
     _rows_contiguous(x, "gated_act")
     T, two_i = x.shape
@@ -495,9 +552,9 @@ def gated_act(x: torch.Tensor, out: torch.Tensor, activation: str = "silu", pair
         raise KernelError(f"gated_act: unknown activation {activation!r}")
     if two_i % 2 or out.shape != (T, inter) or not out.is_contiguous() or out.dtype != x.dtype:
         raise KernelError("gated_act: x [T, 2I], out [T, I] contiguous, same dtype")
-    lib, f = _fn("elementwise", "dinfer_gated_act", [c_void_p, c_void_p, c_int, c_int, c_int64, c_int, c_int, c_int, c_void_p])
+    lib, f = _fn("elementwise", "dinfer_gated_act_ex", [c_void_p, c_void_p, c_int, c_int, c_int64, c_int, c_int, c_int, c_float, c_float, c_void_p])
     check(lib, f(ptr(x), ptr(out), T, inter, x.stride(0), dtype_code(x.dtype), int(bool(pairs)),
-                 GATE_ACTIVATIONS[activation], stream_handle()), "gated_act")
+                 GATE_ACTIVATIONS[activation], ga, gb, stream_handle()), "gated_act")
     return out
 
 
@@ -509,7 +566,7 @@ def gated_act_scaled(x: torch.Tensor, out: torch.Tensor, scale: torch.Tensor, in
     _rows_contiguous(x, "gated_act_scaled")
     T, two_i = x.shape
     inter = two_i // 2
-    if activation not in GATE_ACTIVATIONS:
+    if activation not in GATE_ACTIVATIONS or activation == "clamped_swish":
         raise KernelError(f"gated_act_scaled: unknown activation {activation!r}")
     if two_i % 2 or out.shape != (T, inter) or not out.is_contiguous() or out.dtype != x.dtype:
         raise KernelError("gated_act_scaled: x [T, 2I], out [T, I] contiguous, same dtype")

@@ -1,5 +1,6 @@
 """Wrappers of the kernels for linear-attention mixers with a decay per key channel (``csrc/linear_state.cu``): the
-general delta rule and the gate-write form share one recurrence."""
+general delta rule and the gate-write form share one recurrence; and of those of the state-space mixer
+(``csrc/state_space.cu``)."""
 from __future__ import annotations
 
 from ctypes import c_float, c_int, c_int64, c_void_p
@@ -7,7 +8,7 @@ from typing import Optional, Tuple
 
 import torch
 
-from .lib import KernelError, check, ptr, require_cuda, stream_handle
+from .lib import KernelError, add_launches, check, dtype_code, ptr, require_cuda, stream_handle
 from .ops import _fn
 
 
@@ -109,4 +110,78 @@ def recurrence(r: torch.Tensor, w: torch.Tensor, v: torch.Tensor, state: torch.T
     check(lib, f(ptr(r), st(r), ptr(k), st(k), ptr(w), st(w), ptr(u), st(u), ptr(p), st(p), ptr(v), st(v), ptr(state),
                  state.stride(0), ptr(cu_seqlens), ptr(slots), ptr(fresh), ptr(out), B, H, dk, dv,
                  int(remove), int(widen), int(T > B), stream_handle()), "linear_state")
+    return out
+
+
+def _state_space_sizes(P, conv_w, state, cu_seqlens, slots, fresh, H, G, N, dv, taps):
+    """Checks shared by the two calls; returns (channels of the convolution, offset of its inputs in a state row)."""
+    _ints(cu_seqlens, slots, fresh)
+    inner = H * dv
+    channels = inner + 2 * G * N
+    hist = H * N * dv
+    if P.dtype != torch.float32 or P.dim() != 2 or P.stride(1) != 1 or P.shape[1] < inner + channels + H:
+        raise KernelError("state space: the projected rows are float32 [T, >= 2 H P + 2 G N + H]")
+    if conv_w is not None and (conv_w.dtype != torch.float32 or tuple(conv_w.shape) != (channels, taps) or not conv_w.is_contiguous()):
+        raise KernelError("state space: conv_w contiguous float32 [channels, taps]")
+    if state.dtype != torch.float32 or state.dim() != 2 or state.stride(1) != 1 or state.shape[1] < hist + (taps - 1) * channels:
+        raise KernelError("state space: state f32 [slots, >= H N P + (taps - 1) * channels]")
+    return channels, hist
+
+
+def state_space(P: torch.Tensor, conv_w: torch.Tensor, conv_b: torch.Tensor, dt_bias: torch.Tensor, A_log: torch.Tensor,
+                D: torch.Tensor, state: torch.Tensor, cu_seqlens: torch.Tensor, slots: torch.Tensor, fresh: torch.Tensor,
+                num_heads: int, groups: int, state_dim: int, value_dim: int, taps: int, any_single: bool = True,
+                any_portion: bool = True, max_q_len: int = 0) -> torch.Tensor:
+    """``P`` float32 rows [z | x | B | C | dt] (a view with a row stride is fine): convolution with bias and silu of x, B, C,
+    ``dt = softplus(dt + dt_bias)``, ``S <- exp(-exp(A_log) dt) S + dt B x^T``, ``y = S^T C + D x`` per request and head, S
+    [N, P] carried in the first ``H N P`` floats of row ``slots[b]`` of ``state`` (zero for a fresh request); the
+    convolution's earlier inputs are read from behind them and moved on by ``state_space_post``.  Requests that bring one
+    token go through one kernel, the others' chunks of 64 tokens side by side through four; ``any_single`` /
+    ``any_portion`` say which there are, ``max_q_len`` (0: not known) bounds the longest portion.  Returns y f32 [T, H * P]."""
+    require_cuda(P, conv_w, conv_b, dt_bias, A_log, D, state, cu_seqlens, slots, fresh)
+    H, G, N, dv = num_heads, groups, state_dim, value_dim
+    channels, hist = _state_space_sizes(P, conv_w, state, cu_seqlens, slots, fresh, H, G, N, dv, taps)
+    for t, n, what in ((conv_b, channels, "conv_b [channels]"), (dt_bias, H, "dt_bias [H]"), (A_log, H, "A_log [H]"), (D, H, "D [H]")):
+        _vec(t, n, "state space " + what)
+    T, B = P.shape[0], cu_seqlens.numel() - 1
+    y = torch.empty((T, H * dv), dtype=torch.float32, device=P.device)
+    if T == 0:
+        return y
+    lib, f = _fn("state_space", "dinfer_state_space",
+                 [c_void_p, c_int64, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_int64, c_int, c_void_p,
+                  c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_int,
+                  c_int, c_void_p])
+    work = None
+    if any_portion:
+        size = lib.dinfer_state_space_work_floats
+        size.restype, size.argtypes = c_int64, [c_int64, c_int, c_int, c_int, c_int, c_int]
+        work = torch.empty(size(T, B, H, G, N, dv), dtype=torch.float32, device=P.device)
+    check(lib, f(ptr(P), P.stride(0), ptr(conv_w), ptr(conv_b), ptr(dt_bias), ptr(A_log), ptr(D), ptr(state),
+                 state.stride(0), hist, ptr(cu_seqlens), ptr(slots), ptr(fresh), ptr(y), ptr(work), T, B, H, G, N, dv, taps,
+                 int(bool(any_single)), int(bool(any_portion)), int(max_q_len) if max_q_len > 0 else T, stream_handle()),
+          "state_space")
+    add_launches((1 if any_single else 0) + (4 if any_portion else 0) - 1)
+    return y
+
+
+def state_space_post(y: torch.Tensor, P: torch.Tensor, weight: torch.Tensor, eps: float, parts: int, out: torch.Tensor,
+                     state: torch.Tensor, cu_seqlens: torch.Tensor, slots: torch.Tensor, fresh: torch.Tensor, num_heads: int,
+                     groups: int, state_dim: int, value_dim: int, taps: int) -> torch.Tensor:
+    """``out[t] = y[t] * silu(z[t])`` with each of ``parts`` equal parts of the row divided by its own root mean square, times
+    ``weight`` f32 [H * P]; ``out`` (rows with a stride are fine) may be wider than H * P, the rest gets zeros.  Then the
+    requests' last ``taps - 1`` convolution inputs move into ``state``."""
+    require_cuda(y, P, weight, out, state, cu_seqlens, slots, fresh)
+    H, G, N, dv = num_heads, groups, state_dim, value_dim
+    _, hist = _state_space_sizes(P, None, state, cu_seqlens, slots, fresh, H, G, N, dv, taps)
+    inner, T, B = H * dv, P.shape[0], cu_seqlens.numel() - 1
+    _vec(weight, inner, "state space norm weight [H * P]")
+    if y.dtype != torch.float32 or tuple(y.shape) != (T, inner) or not y.is_contiguous() or out.stride(1) != 1 \
+            or out.shape[0] != T or out.shape[1] < inner or parts <= 0 or inner % parts:
+        raise KernelError("state space post: y f32 [T, H * P], out [T, >= H * P], parts divides H * P")
+    lib, f = _fn("state_space", "dinfer_state_space_post",
+                 [c_void_p, c_void_p, c_int64, c_void_p, c_float, c_int, c_void_p, c_int64, c_int, c_void_p, c_int64, c_int,
+                  c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_void_p])
+    check(lib, f(ptr(y), ptr(P), P.stride(0), ptr(weight), float(eps), int(parts), ptr(out), out.stride(0), out.shape[1],
+                 ptr(state), state.stride(0), hist, ptr(cu_seqlens), ptr(slots), ptr(fresh), T, B, H, G, N, dv, taps,
+                 dtype_code(out.dtype), stream_handle()), "state_space_post")
     return out

@@ -12,7 +12,7 @@ import torch
 
 from ..kernels import ops
 from ..parts import (attention, block, delta_rule, differential_attention, embedding, latent_attention,  # noqa: F401
-                     linear_state, mlp, moe, norm, parallel_mixers, retention, rope, short_conv, token_side)   # (register the built-in parts)
+                     linear_state, mlp, moe, norm, parallel_mixers, retention, rope, short_conv, state_space, token_side)   # (register the built-in parts)
 from ..parts.base import (BLOCKS, EMBEDDINGS, FEED_FORWARDS, MIXERS, NORMS, BuildEnv, CacheBinding, ResidualStream,
                           StepContext, build_part)
 from ..parts.linear import Linear

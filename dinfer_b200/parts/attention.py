@@ -43,7 +43,10 @@ class GQAttention(Mixer):
     ``chunked``: ``window`` is the size of chunks of positions, counted from the sequence's first, and a token sees the
     tokens of its own chunk.  ``value_turn`` (a rotation's base): the value of position j is cached turned by j over its
     whole width, pair m by ``j * base^(-2m / v_dim)`` in the position encoding's layout of pairs, and every head's output at
-    position i is turned back by i, ahead of the gate."""
+    position i is turned back by i, ahead of the gate.
+    ``qk_norm_over``: "head" (the default) or "all": one norm over all of q and one over all of k, their weights as wide as
+    the projections.  ``keep_first``: with a window, the first so many tokens of a request stay visible behind it (their
+    pages are kept).  ``softcap`` > 0: a score is ``softcap * tanh(score / softcap)``."""
 
     def __init__(self, params, env: BuildEnv, prefix=""):
         super().__init__(params, env, prefix)
@@ -93,6 +96,17 @@ class GQAttention(Mixer):
         self.value_mix = dict(p["value_mix"]) if p.get("value_mix") else None
         self.gate_name = prefix + p["gate_proj"] if p.get("gate_proj") else None
         # the q/k kernel with lane paths takes the usual order and equal widths; anything else takes the general one
+        self.keep_first = int(p.get("keep_first") or 0) if self.window else 0
+        self.softcap = float(p.get("softcap") or 0.0)
+        self.norm_all = p.get("qk_norm_over", "head") == "all"
+        if p.get("qk_norm_over", "head") not in ("head", "all") or self.softcap < 0 or self.keep_first < 0 \
+                or (self.keep_first and self.chunked):
+            raise ValueError("attention: qk_norm_over is head or all; softcap and keep_first are not negative, and kept tokens "
+                             "belong to a window")
+        if self.norm_all and not self._plain_ends():
+            raise ValueError("attention: one norm over all heads comes ahead of the rotation, with weights, without biases, "
+                             "gates, a query temperature, mixed or turned values")
+        self.v_scale = 1.0
         self.general = (self.Dv != self.D or (self.qk_norm and (self.norm_after or not self.norm_weight))
                         or self.q_temperature is not None or self.value_mix is not None or self.value_turn is not None)
         pos: PartSpec = p.get("position") or PartSpec("none")
@@ -111,12 +125,18 @@ class GQAttention(Mixer):
         self.o: Optional[Linear] = None
         self.q_norm_w = self.k_norm_w = None
 
+    def _plain_ends(self) -> bool:
+        """Whether nothing but q, k, v stands in the projection and nothing but the heads in the result."""
+        return not (self.bias or self.gate_name or self.value_mix or self.value_turn or self.q_temperature or self.norm_after
+                    or (self.qk_norm and not self.norm_weight))
+
     def declare(self) -> List[TensorDecl]:
         H, Hkv, D, Dv, h = self.H, self.Hkv, self.D, self.Dv, self.hidden
         d = [TensorDecl(self.names["q"], (H * D, h)), TensorDecl(self.names["k"], (Hkv * D, h)),
              TensorDecl(self.names["v"], (Hkv * Dv, h)), TensorDecl(self.names["o"], (h, H * Dv))]
         if self.qk_norm and self.norm_weight:
-            d += [TensorDecl(self.names["qn"], (D,), init="ones"), TensorDecl(self.names["kn"], (D,), init="ones")]
+            nq, nk = (H * D, Hkv * D) if self.norm_all else (D, D)
+            d += [TensorDecl(self.names["qn"], (nq,), init="ones"), TensorDecl(self.names["kn"], (nk,), init="ones")]
         if self.bias:
             d += [TensorDecl(self._bias_name(x), (n,)) for x, n in (("q", H * D), ("k", Hkv * D), ("v", Hkv * Dv), ("o", h))]
         if self.value_mix:
@@ -164,13 +184,18 @@ class GQAttention(Mixer):
         if self.value_mix:
             self.v_lambda = float(tensors[self.names["vmix"]].float().item())
         self.o = Linear(tensors[self.names["o"]], o_bias)
-        if self.qk_norm and self.norm_weight:
+        self._bind_norms(tensors)
+
+    def _bind_norms(self, tensors) -> None:
+        if self.qk_norm and self.norm_weight and self.norm_all:
+            self.q_norm_w, self.k_norm_w = (tensors[self.names[x]].to(torch.float32).contiguous() for x in ("qn", "kn"))
+        elif self.qk_norm and self.norm_weight:
             self.q_norm_w = tensors[self.names["qn"]].contiguous()
             self.k_norm_w = tensors[self.names["kn"]].to(self.q_norm_w.dtype).contiguous()
 
     def cache_need(self):
         return KvCacheNeed(self.Hkv, max(self.D, self.Dv), self.window, int(self.page_size) if self.page_size else None,
-                           chunked=self.chunked)
+                           keep_first=self.keep_first, chunked=self.chunked)
 
     def _fast(self, dtype) -> bool:
         """Whether the tensor-core kernels take this attention: keys and values of one width."""
@@ -183,7 +208,34 @@ class GQAttention(Mixer):
             att = ["attention_tc"]
             if self.D in (64, 128):
                 att += ["attention_decode", "attention_umma", "attention_umma64"]
-        return ["qk_post"] + att + self.qkv.kernel_libraries() + self.o.kernel_libraries()
+        ends = [l for l in (self.qkv, self.o) if l is not None]     # (none where another part owns the two products)
+        return ["qk_post"] + att + [n for l in ends for n in l.kernel_libraries()]
+
+    # ---- between two products of another part (see Mixer.open_ends)
+    def open_ends(self):
+        if not self._plain_ends() or (self.qk_norm and not self.norm_all):
+            return None
+        return (self.H + self.Hkv) * self.D + self.Hkv * self.Dv, self.H * self.Dv
+
+    def input_rows(self, tensors) -> torch.Tensor:
+        rows = [tensors[self.names[x]] for x in ("q", "k", "v")]
+        dt = torch.float32 if any(t.dtype == torch.float32 for t in rows) else rows[0].dtype
+        return torch.cat([t.to(dt) for t in rows], dim=0)
+
+    def output_columns(self, tensors) -> torch.Tensor:
+        return tensors[self.names["o"]]
+
+    def bind_inner(self, tensors, scale: float = 1.0) -> None:
+        self._bind_norms(tensors)
+        self.v_scale = float(scale)                          # the heads are linear in the values: cached times the scale
+
+    def mix(self, P, out, ctx: StepContext, cache: CacheBinding) -> None:
+        g = ctx.groups[cache.group]
+        q = torch.empty((P.shape[0], self.H * self.D), dtype=self.env.act_dtype, device=P.device)
+        ops.qkv_post_whole(P, ctx.positions, self.H, self.Hkv, self.D, self.Dv, self.eps, self.q_norm_w, self.k_norm_w,
+                           self.position.fused_table(), q, cache.kv if cache.write else None, g.slot_mapping, g.block_size,
+                           interleaved=getattr(self.position, "interleaved", False), v_scale=self.v_scale)
+        self.attend(q, out, cache.kv, g, ctx)
 
     def takes_half_normed(self, rows: int) -> bool:
         return self.qkv.fuses_norm(rows, self.env.act_dtype)
@@ -192,6 +244,12 @@ class GQAttention(Mixer):
         return self.o.fuses_norm(rows, self.env.act_dtype)
 
     def forward(self, x, ctx: StepContext, cache: CacheBinding, sink=None):
+        if self.norm_all:
+            out = torch.empty((x.shape[0], self.H * self.Dv), dtype=self.env.act_dtype, device=x.device)
+            self.mix(self.qkv(x, out_dtype=torch.float32), out, ctx, cache)
+            if sink is not None:
+                return self.o.into_residual(out, sink[0], sink[1])
+            return self.o(out, out_dtype=torch.float32 if self.out_float32 else None)
         H, Hkv, D = self.H, self.Hkv, self.D
         g = ctx.groups[cache.group]
         qkv = self.qkv(x)
@@ -247,15 +305,16 @@ class GQAttention(Mixer):
         """Tensor-core kernels where they take the head size (bfloat16; 32, 64, 128), else the
         plain-arithmetic kernel, which takes every size."""
         window = int(self.window or 0)
-        seen = dict(sink=self.sink, slopes=self.slopes, chunked=self.chunked, sinks=self.sinks)
+        seen = dict(sink=self.sink, slopes=self.slopes, chunked=self.chunked, sinks=self.sinks, keep_first=self.keep_first,
+                    softcap=self.softcap)
         if self._fast(q.dtype):
             splits = ctx.decode_splits or attention_ops.decode_splits(ctx.num_reqs, self.Hkv, ctx.max_seq_len)
-            if self.chunked:                                # a decoded token sees its chunk at most: no more splits than that fills
+            if self.chunked or self.keep_first:             # a decoded token sees its chunk, or the window and the kept tokens, at most
                 longest = int(self.env.max_positions) if ctx.decode_splits else ctx.max_seq_len    # (a captured graph's bound)
-                splits = min(splits, attention_ops.decode_splits(ctx.num_reqs, self.Hkv, min(window, longest)))
+                splits = min(splits, attention_ops.decode_splits(ctx.num_reqs, self.Hkv, min(window + self.keep_first, longest)))
             tc_decode = ctx.any_decode
             if ctx.any_decode and attention_ops.decode_supported(q.dtype, self.D, self.H // self.Hkv, g.block_size) \
-                    and (g.block_size >= 8 or not (self.sink or self.slopes is not None or self.chunked)):
+                    and (g.block_size >= 8 or not (self.sink or self.slopes is not None or self.chunked or self.keep_first or self.softcap)):
                 # decoded tokens: the kernel made for them (keys on the tile's rows, in-kernel fold)
                 attention_ops.attention_decode(q, out, kv, g.block_table, ctx.cu_seqlens, ctx.seq_lens, self.H,
                                                self.Hkv, self.D, self.scale, window, splits, **seen)

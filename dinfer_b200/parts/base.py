@@ -155,6 +155,14 @@ class Mixer(Part):
     norm))`` adds the part's output into the residual itself and returns the ``HalfNormed`` input of the
     next part instead of the output.  A part without them always gets and gives plain tensors."""
 
+    # A mixer with open ends can be run between two products that are not its own (a pair of mixers then shares one
+    # product in front and one behind): ``open_ends()`` is then (columns of the projected rows, columns of the result
+    # rows), ``input_rows(tensors)`` / ``output_columns(tensors)`` give the two matrices, ``bind_inner(tensors, scale)`` binds
+    # the rest (``scale`` multiplies the result, folded in where it costs nothing), and ``mix(P, out, ctx, cache)`` turns
+    # the projected rows P (32-bit) into the rows ``out`` (a view of the activations' type) ahead of the output product.
+    def open_ends(self):
+        return None
+
     # A mixer with per-request state says here whether its forward can be captured in a CUDA graph: it must read the
     # step's state slots and fresh flags from the device tensors of the context (``ctx.state_slots``,
     # ``ctx.state_fresh``, ``ctx.cu_seqlens``), never from their host copies, and take rows without a request (the

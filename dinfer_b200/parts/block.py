@@ -20,7 +20,7 @@ def norm_comes_apart(producer, norm, consumer, rows: int) -> bool:
 
 @BLOCKS.register("prenorm_residual")
 class PreNormResidual(Block):
-    """``x += mixer(norm1(x)); x += ffn(norm2(x))``.
+    """``x += mixer(norm1(x)); x += ffn(norm2(x))`` (a layer may have no feed-forward, kind "none").
 
     Each add is done inside the norm that follows it, and the feed-forward's output stays pending
     until the next layer's (or the model's final) norm picks it up, as the reference defers its MLP
@@ -44,6 +44,9 @@ class PreNormResidual(Block):
             h = self.mixer_norm.forward(stream.x, delta=stream.pending)
             stream.pending = None
         split = bool(getattr(ctx, "split_norms", False))
+        if getattr(self.feed_forward, "absent", False):     # a layer that is a mixer alone
+            stream.pending = self.mixer.forward(h, ctx, cache)
+            return
         if split and norm_comes_apart(self.mixer, self.feed_forward_norm, self.feed_forward, rows):
             h = self.mixer.forward(h, ctx, cache, sink=(stream.x, self.feed_forward_norm))
         else:

@@ -23,6 +23,7 @@ from typing import Dict, List, Optional
 import torch
 
 from ..kernels import gemm_ops, moe_ops
+from ..kernels.ops import gate_constants
 from .base import FEED_FORWARDS, FeedForward
 from .linear import Linear
 from .spec import TensorDecl
@@ -42,7 +43,9 @@ class MoE(FeedForward):
     ``num_experts`` that have tensors: the router scores and chooses them too, their output is their input, times the
     weight), ``correction`` (tensor name of one number per expert, identity experts included, added to the scores for the
     choice only), ``groups`` = (count, keep): the experts in ``count`` equal runs of neighbours, of which only the ``keep``
-    with the largest choice scores in them take part."""
+    with the largest choice scores in them take part; ``group_rank`` 2: a run ranks by the sum of its two largest.  The
+    ``activation`` of gated experts may be a tuple with constants: ("clamped_swish", limit, alpha), see
+    ``ops.gate_constants``."""
 
     def __init__(self, params, env, prefix=""):
         super().__init__(params, env, prefix)
@@ -51,7 +54,10 @@ class MoE(FeedForward):
         self.E, self.top = int(p["num_experts"]), int(p["top_k"])
         self.ff = int(p["expert_size"])
         self.shared_ff = int(p.get("shared_size", 0) or 0)
-        self.activation = str(p.get("activation", "relu2"))
+        act = p.get("activation", "relu2")
+        # a gate with constants stays a tuple (name, constants)
+        self.activation = (str(act[0]), float(act[1]), float(act[2])) if isinstance(act, (tuple, list)) else str(act)
+        self.act_name = self.activation[0] if isinstance(self.activation, tuple) else self.activation
         self.scoring = str(p.get("scoring", "softmax"))
         self.renormalize = bool(p.get("renormalize", False))
         self.shared_gate = p.get("shared_gate")
@@ -66,6 +72,7 @@ class MoE(FeedForward):
         self.E_all = self.E + self.identity                 # what the router scores
         self.correction_name = prefix + p["correction"] if p.get("correction") else None
         self.groups = tuple(int(v) for v in p["groups"]) if p.get("groups") else (1, 1)
+        self.group_rank = int(p.get("group_rank", 1))
         self.by_choice = bool(self.identity or self.correction_name or p.get("groups"))
         self.correction = None
         if self.by_choice:
@@ -73,13 +80,19 @@ class MoE(FeedForward):
             if self.routing != "router" or self.shared_gate or self.weight_on_input:
                 raise ValueError("moe: identity experts, a correction and groups need a router, the weight on the output and "
                                  "no gate on the shared expert")
+            if self.group_rank not in (1, 2):
+                raise ValueError("moe: group_rank is 1 or 2")
             if count <= 0 or self.E_all % count or not (0 < keep <= count) or self.top > keep * (self.E_all // count):
                 raise ValueError(f"moe: groups {self.groups} do not divide {self.E_all} experts, or keep fewer than top_k {self.top}")
         if self.routing not in ("router", "table") or (self.routing == "table" and (self.vocab <= 0 or self.shared_gate)):
             raise ValueError("moe: routing is router or table; a table needs vocab_size and takes no gate on the shared expert")
         if not (0 < self.top <= self.E_all):
             raise ValueError(f"moe: top_k {self.top} must be between 1 and the {self.E_all} experts")
-        if self.activation not in moe_ops.ACTIVATIONS or self.activation == "none":
+        if isinstance(self.activation, tuple):
+            gate_constants(self.activation)
+            if not self.gated or self.weight_on_input:
+                raise ValueError("moe: a gate with constants needs gated experts with the weight on the output")
+        elif self.activation not in moe_ops.ACTIVATIONS or self.activation == "none":
             raise ValueError(f"moe: unknown activation {self.activation!r}")
         if self.scoring not in ("softmax", "sigmoid") or self.shared_gate not in (None, "sigmoid"):
             raise ValueError("moe: scoring is softmax or sigmoid, shared_gate sigmoid or None")
@@ -169,7 +182,7 @@ class MoE(FeedForward):
             if self.by_choice:
                 gate = None
                 ids, weights = moe_ops.route_choice(z, self.E_all, self.top, self.correction, self.scoring, self.renormalize,
-                                                    *self.groups)
+                                                    *self.groups, group_rank=self.group_rank)
             else:
                 ids, weights, gate = moe_ops.route(z, self.E, self.top, self.scoring, self.renormalize,
                                                    bool(self.shared_ff and self.shared_gate))
@@ -182,7 +195,7 @@ class MoE(FeedForward):
             # prompt-sized steps: rows laid out expert by expert in whole 256-row tiles, both products on tcgen05
             order, tile_expert = moe_ops.align(ids, self.E, moe_ops.TC_ROW_TILE)
             a = moe_ops.gather_rows(x, order, pairs, self.top)
-            if self.gated and not self.weight_on_input and self.activation in gemm_ops.GATES:
+            if self.gated and not self.weight_on_input and self.act_name in gemm_ops.GATES:
                 u = torch.empty((order.numel(), self.ff), dtype=x.dtype, device=x.device)      # the gate in the epilogue
                 moe_ops.grouped_gemm_tc(a, self.w_up, u, order, tile_expert, pairs, 0, gate=self.activation)
             else:
