@@ -455,9 +455,34 @@ DATOZEN_SIZES = {
     "medium": (_datozen_cfg(2048, 16, 4, 128, 64, 16, 8, 4, 6, 1408, 2816, 11520, 128), _qwen3_cfg(2048, 16, 4, 128, 7680)),
     "large": (_datozen_cfg(4096, 32, 8, 128, 64, 16, 8, 4, 6, 2048, 4096, 18432, 256), _qwen3_cfg(4096, 32, 8, 128, 12288)),
 }
-DESIGNS = {"datozen": DATOZEN_SIZES, "dobedra": DESIGN_SIZES, "zasipel": ZASIPEL_SIZES, "sobivik": SOBIVIK_SIZES, "porovik": POROVIK_SIZES}
+
+
+# ---------------------------------------------------------------- Rorutar beside Zasipel at equal layer sizes
+def _rorutar_cfg(width, heads, kv_heads, dim, window, state_heads, vdim, state, groups, experts, expert_groups, keep, top, ff,
+                 vocab=32768):
+    left = {"heads": heads, "kv_heads": kv_heads, "dim": dim, "vdim": dim, "scale": dim ** -0.5, "softcap": 30.0,
+            "mask": {"size": window, "keep_first": 4}, "rot": {"base": 10000.0, "dims": dim, "scaling": {"factor": 4.0}}}
+    right = {"heads": state_heads, "vdim": vdim, "state": state, "groups": groups, "conv": 4, "norm_groups": groups}
+    moe = {"kind": "moe", "expert": {"ff": ff, "limit": 7.0},
+           "router": {"experts": experts, "top": top, "groups": {"count": expert_groups, "keep": keep}}}
+    layer = {"type": "parallel", "mixer": {"left": left, "right": right, "left_scale": 0.5, "right_scale": 0.7}, "mlp": moe}
+    return {"architecture": "Rorutar", "vocab": vocab, "width": width, "norm": {"eps": 1e-6}, "embedding": {"scale": 1.0},
+            "layers": [layer] * 4}
+
+
+# four layers (attention over a window of 1024 and four kept tokens, heads of 64 or 128, beside a state-space mixer whose
+# state is as large as the delta rule's of the Zasipel layers at that size, 16 or 64 experts of which a token uses 4 or 8: the
+# weights of Zasipel's chosen experts and its shared one); no loop, so that four layers run; beside each the Zasipel
+# layers of the same width, heads and experts (the closest design: two mixers side by side, attention over a window with a
+# sink and a recurrence with a short convolution, routed gated experts)
+RORUTAR_SIZES = {
+    "small": (_rorutar_cfg(1024, 16, 4, 64, 1024, 16, 64, 64, 2, 16, 4, 2, 4, 512), ZASIPEL_SIZES["small"][0]),
+    "medium": (_rorutar_cfg(2048, 16, 4, 128, 1024, 32, 64, 128, 4, 64, 8, 4, 8, 1408), ZASIPEL_SIZES["medium"][0]),
+    "large": (_rorutar_cfg(4096, 32, 8, 128, 1024, 64, 64, 128, 8, 64, 8, 4, 8, 2048), ZASIPEL_SIZES["large"][0]),
+}
+DESIGNS = {"rorutar": RORUTAR_SIZES, "datozen": DATOZEN_SIZES, "dobedra": DESIGN_SIZES, "zasipel": ZASIPEL_SIZES, "sobivik": SOBIVIK_SIZES, "porovik": POROVIK_SIZES}
 # the model a design stands beside (the closest one this package has)
-BESIDE = {"porovik": "zasipel"}
+BESIDE = {"porovik": "zasipel", "rorutar": "zasipel"}
 
 
 def _time_model(cfg, batch, context, prefill_tokens, steps, seed=5, profile=None):
@@ -519,7 +544,7 @@ def _time_model(cfg, batch, context, prefill_tokens, steps, seed=5, profile=None
 
 
 def design_run(a) -> int:
-    """``--design dobedra|zasipel|sobivik|porovik|datozen``: prefill and decode throughput of four layers of the design beside four
+    """``--design dobedra|zasipel|sobivik|porovik|datozen|rorutar``: prefill and decode throughput of four layers of the design beside four
     layers of the model it is compared with (Qwen3, or ``BESIDE``) at the same width and head count, at the sizes of
     ``DESIGNS``; one JSON line."""
     rows = {}
@@ -564,11 +589,11 @@ def main() -> int:
     ap.add_argument("--closed-loop", default=None, metavar="C,P,O",
                     help="the reference's serving measurement at engine level instead: C clients, each sending its "
                          "next request when the last has ended, prompts of P tokens, O generated tokens (--shape applies)")
-    ap.add_argument("--design", choices=["dobedra", "zasipel", "sobivik", "porovik", "datozen"], default=None,
+    ap.add_argument("--design", choices=["dobedra", "zasipel", "sobivik", "porovik", "datozen", "rorutar"], default=None,
                     help="instead of the benchmark: four layers of this design beside four Qwen3 layers of equal width, "
                          "prefill and decode, at a few layer sizes")
     ap.add_argument("--design-size", choices=["small", "medium", "large"], default=None, help="only this size")
-    ap.add_argument("--design-model", choices=["dobedra", "zasipel", "sobivik", "porovik", "datozen", "qwen3"], default=None, help="with --profile: which of the two")
+    ap.add_argument("--design-model", choices=["dobedra", "zasipel", "sobivik", "porovik", "datozen", "rorutar", "qwen3"], default=None, help="with --profile: which of the two")
     a = ap.parse_args()
     if a.impl == "reference":
         print(json.dumps({"impl": "reference", "unavailable":

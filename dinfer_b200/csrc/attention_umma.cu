@@ -354,9 +354,9 @@ attention_umma_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_co
         tmem_ld_wait();
         if (CAP) {
 #pragma unroll
-          for (int i = 0; i < 32; ++i) {
-            v0[i] = softcap_log2(v0[i], p.cap_in, p.cap_out);
-            v1[i] = softcap_log2(v1[i], p.cap_in, p.cap_out);
+          for (int i = 0; i < 32; i += 4) {
+            softcap4_log2(v0[i], v0[i + 1], v0[i + 2], v0[i + 3], p.cap_in, p.cap_out);
+            softcap4_log2(v1[i], v1[i + 1], v1[i + 2], v1[i + 3], p.cap_in, p.cap_out);
           }
         }
         if (p.slopes) {

@@ -322,9 +322,9 @@ attention_umma64_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_
       const int jbase = tile_of(j, kept, tile_first) * BN;
       if (CAP) {
 #pragma unroll
-        for (int i = 0; i < 32; ++i) {
-          s0[i] = softcap_log2(s0[i], p.cap_in, p.cap_out);
-          s1[i] = softcap_log2(s1[i], p.cap_in, p.cap_out);
+        for (int i = 0; i < 32; i += 4) {
+          softcap4_log2(s0[i], s0[i + 1], s0[i + 2], s0[i + 3], p.cap_in, p.cap_out);
+          softcap4_log2(s1[i], s1[i + 1], s1[i + 2], s1[i + 3], p.cap_in, p.cap_out);
         }
       }
       if (p.slopes) {

@@ -116,6 +116,24 @@ __device__ __forceinline__ float softcap_log2(float s, float cap_in, float cap_o
   asm("rcp.approx.ftz.f32 %0, %1;" : "=f"(r) : "f"(1.f + e));       // e = inf gives 0
   return fmaf(-2.f * cap_out, r, cap_out);
 }
+// The same for four scores with one reciprocal, of the product of the four denominators (the special function unit is what
+// such a kernel waits for).  The exponent stops at 30, where tanh has long rounded to 1, so that the product stays finite.
+__device__ __forceinline__ void softcap4_log2(float& a, float& b, float& c, float& d, float cap_in, float cap_out) {
+  auto denominator = [&](float s) {
+    float e;
+    asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(e) : "f"(fminf(s * cap_in, 30.f)));
+    return 1.f + e;
+  };
+  const float da = denominator(a), db = denominator(b), dc = denominator(c), dd = denominator(d);
+  const float ab = da * db, cd = dc * dd;
+  float r;
+  asm("rcp.approx.ftz.f32 %0, %1;" : "=f"(r) : "f"(ab * cd));
+  const float k = -2.f * cap_out * r, rab = k * cd, rcd = k * ab;
+  a = fmaf(rab, db, cap_out);
+  b = fmaf(rab, da, cap_out);
+  c = fmaf(rcd, dd, cap_out);
+  d = fmaf(rcd, dc, cap_out);
+}
 // The softmax's extra term of a head (it has no key and no value): its score times log2(e); the score is sinks[head],
 // or 0 where no sinks are given.
 __device__ __forceinline__ float sink_log2(const float* sinks, int head) {

@@ -97,10 +97,11 @@ moe_route_kernel(const float* __restrict__ logits, int64_t ldz, int* __restrict_
 // The scores as above over all E experts; an expert is chosen by score + correction[e], its weight is the score alone
 // (divided by the chosen ones' sum with renorm).  The experts form `groups` equal runs of neighbours; a run's rank is its
 // largest choice score, or the sum of its two largest (rank_two), and only experts of the `keep` best runs can be chosen.  Equal choice scores go to the lower index.
-__device__ __forceinline__ void warp_best(float& best, int& arg) {
+template <typename T>
+__device__ __forceinline__ void warp_best(T& best, int& arg) {
 #pragma unroll
   for (int o = 16; o > 0; o >>= 1) {
-    const float ob = __shfl_xor_sync(0xffffffffu, best, o);
+    const T ob = __shfl_xor_sync(0xffffffffu, best, o);
     const int oa = __shfl_xor_sync(0xffffffffu, arg, o);
     if (ob > best || (ob == best && oa < arg)) { best = ob; arg = oa; }
   }
@@ -110,14 +111,14 @@ __global__ void __launch_bounds__(RW * 32)
 moe_route_choice_kernel(const float* __restrict__ logits, int64_t ldz, const float* __restrict__ correction,
                         int* __restrict__ ids, float* __restrict__ weights, int T, int E, int top, int sigmoid_scores,
                         int renorm, int groups, int keep, int rank_two) {
-  extern __shared__ float sm[];                          // per warp: E scores, E choice scores, `groups` ranks
+  extern __shared__ double smd[];                        // per warp: `groups` ranks, then E scores, E choice scores
   pdl_enter();
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   const int t = blockIdx.x * RW + warp;
   if (t >= T) return;
-  float* z = sm + (size_t)warp * (2 * E + groups);
+  double* rank = smd + (size_t)warp * groups;
+  float* z = reinterpret_cast<float*>(smd + (size_t)RW * groups) + (size_t)warp * 2 * E;
   float* c = z + E;
-  float* rank = c + E;
   const float* row = logits + (int64_t)t * ldz;
   float mx = -INFINITY;
   for (int e = lane; e < E; e += 32) { z[e] = row[e]; mx = fmaxf(mx, z[e]); }
@@ -140,15 +141,18 @@ moe_route_choice_kernel(const float* __restrict__ logits, int64_t ldz, const flo
     for (int g = lane; g < groups; g += 32) {
       float m = -INFINITY, m2 = -INFINITY;
       for (int i = 0; i < size; ++i) {
-        const float v = by_logit && rank_two ? z[g * size + i] : c[g * size + i];
+        const float v = c[g * size + i];
         m2 = fmaxf(m2, fminf(m, v));
         m = fmaxf(m, v);
       }
-      rank[g] = rank_two && size > 1 ? m + m2 : m;
+      // (the two scores of large logits in 64-bit, so that sums close to 2 keep their order)
+      const bool two = rank_two && size > 1;
+      if (by_logit && two) rank[g] = 1.0 / (1.0 + exp(-(double)m)) + 1.0 / (1.0 + exp(-(double)m2));
+      else rank[g] = two ? (double)m + (double)m2 : (double)m;
     }
     __syncwarp();
     for (int k = 0; k < keep; ++k) {
-      float best = -INFINITY;
+      double best = -INFINITY;
       int arg = groups;
       for (int g = lane; g < groups; g += 32)
         if (rank[g] > best) { best = rank[g]; arg = g; }
@@ -558,7 +562,7 @@ DINFER_API int dinfer_moe_route_choice(const float* logits, int64_t ldz, const f
   if (T < 0 || E <= 0 || top <= 0 || groups <= 0 || E % groups || keep <= 0 || keep > groups ||
       (int64_t)top > (int64_t)keep * (E / groups) || ldz < E || (group_rank != 1 && group_rank != 2))
     return refuse(DINFER_BAD_ARGUMENT, "moe_route_choice: bad sizes T=%d E=%d top=%d groups=%d keep=%d", T, E, top, groups, keep);
-  const size_t smem = (size_t)RW * (2 * E + groups) * sizeof(float);
+  const size_t smem = (size_t)RW * (2 * E * sizeof(float) + groups * sizeof(double));
   if (smem > 48 * 1024) return refuse(DINFER_BAD_ARGUMENT, "moe_route_choice: %d experts in %d groups are too many", E, groups);
   if (T == 0) return 0;
   launch_pdl(moe_route_choice_kernel, dim3((T + RW - 1) / RW), dim3(RW * 32), smem, stream, logits, ldz, correction, ids, weights,

@@ -62,7 +62,7 @@ template <int V> __device__ __forceinline__ void stv(float* p, const Vec<V>& v) 
 // L lanes share a row of S, V neighbouring columns each; 256 / L rows at a time.  RPT > 0: a thread's rows (at most RPT)
 // stay in registers from the loads ahead of the wait on; RPT = 0: rows as they come.
 template <int V, int L, int RPT>
-__global__ void __launch_bounds__(THREADS) ssm_step_kernel(const Params p) {
+__global__ void __launch_bounds__(THREADS, RPT == 16 ? 2 : (RPT == 8 ? 3 : 4)) ssm_step_kernel(const Params p) {
   constexpr int PT = V * L, R = THREADS / L, WARPS = THREADS / 32;
   extern __shared__ float sm[];                    // B [N], C [N], x [PT], partial sums [WARPS][PT]
   float* sB = sm;
@@ -486,60 +486,77 @@ __global__ void __launch_bounds__(THREADS) ssm_outputs_kernel(const Params p) {
 
 // ---------------------------------------------------------------- gate, norm, the convolution's inputs
 constexpr int POST_THREADS = 128;
+constexpr int HOLD = 4;                             // runs a thread holds in registers (longer parts read theirs again)
 
-// grid T * parts + B: a (token, part of the row) each, then a request's convolution inputs each.  out: rows of stride ldo,
-// columns [inner, pad_to) are filled with zeros.
-template <typename TO, int V>
+// The last CTAs of the launch: run `job` of the channels of a request (V channels a thread).  Four rows at a time are read
+// before they are written; rows rise, so a row is read before it is overwritten.
+template <int V>
+__device__ __forceinline__ void move_inputs(const Params& p, int job, int jobs_per_request) {
+  const int b = job / jobs_per_request;
+  const int start = p.cu[b], n = p.cu[b + 1] - start, rows = p.taps - 1, ch = p.channels();
+  const int c = ((job % jobs_per_request) * POST_THREADS + threadIdx.x) * V;
+  if (n <= 0 || c >= ch) return;
+  float* hist = p.state + (int64_t)p.slots[b] * p.ld_state + p.hist + c;
+  const float* x = p.P + (int64_t)start * p.ldp + p.inner() + c;
+  const bool have = !p.fresh[b];
+  for (int r0 = 0; r0 < rows; r0 += 4) {
+    Vec<V> v[4];
+#pragma unroll
+    for (int u = 0; u < 4; ++u) {
+      const int i = n - rows + r0 + u;              // index inside the portion; negative: from the inputs before it
+#pragma unroll
+      for (int e = 0; e < V; ++e) v[u].x[e] = 0.f;
+      if (r0 + u >= rows) continue;
+      if (i >= 0) v[u] = ldv<V>(x + (int64_t)i * p.ldp);
+      else if (have) v[u] = ldv<V>(hist + (int64_t)(rows + i) * ch);
+    }
+#pragma unroll
+    for (int u = 0; u < 4; ++u)
+      if (r0 + u < rows) stv<V>(hist + (int64_t)(r0 + u) * ch, v[u]);
+  }
+}
+
+// W threads (a warp, or the whole CTA) share a part of a token's row: rows_ctas CTAs of POST_THREADS / W parts each, then
+// the CTAs that move the convolution's inputs.  out: rows of stride ldo, columns [inner, pad_to) are filled with zeros.
+template <typename TO, int V, int W>
 __global__ void __launch_bounds__(POST_THREADS)
 ssm_post_kernel(const Params p, const float* __restrict__ weight, float eps, int parts, TO* __restrict__ out, int64_t ldo,
-                int pad_to) {
-  constexpr int HOLD = 4;                          // runs a thread holds in registers (longer parts read theirs again)
+                int pad_to, int rows_ctas, int jobs_per_request) {
   __shared__ float red[33];
   pdl_enter();
-  const int inner = p.inner(), ch = p.channels(), tid = threadIdx.x;
-  if ((int64_t)blockIdx.x >= (int64_t)p.T * parts) {
-    const int b = (int)(blockIdx.x - (int64_t)p.T * parts);
-    const int start = p.cu[b], n = p.cu[b + 1] - start, rows = p.taps - 1;
-    if (n <= 0) return;
-    float* hist = p.state + (int64_t)p.slots[b] * p.ld_state + p.hist;
-    const bool have = !p.fresh[b];
-    for (int c = tid; c < ch; c += POST_THREADS)
-      for (int r = 0; r < rows; ++r) {             // rising r: a row is read before it is overwritten
-        const int i = n - rows + r;                // index inside the portion; negative: from the inputs before it
-        float x = 0.f;
-        if (i >= 0) x = p.P[(int64_t)(start + i) * p.ldp + inner + c];
-        else if (have) x = hist[(int64_t)(rows + i) * ch + c];
-        hist[(int64_t)r * ch + c] = x;
-      }
-    return;
-  }
-  const int t = blockIdx.x / parts, part = blockIdx.x % parts, len = inner / parts;
+  if ((int)blockIdx.x >= rows_ctas) return move_inputs<V>(p, blockIdx.x - rows_ctas, jobs_per_request);
+  const int inner = p.inner(), len = inner / parts, tid = threadIdx.x % W;
+  const int64_t job = (int64_t)blockIdx.x * (POST_THREADS / W) + threadIdx.x / W;
+  if (job >= (int64_t)p.T * parts) return;           // (a whole warp of them, or the CTA: W divides it)
+  const int t = (int)(job / parts), part = (int)(job % parts);
   const float* y = p.y + (int64_t)t * inner + (int64_t)part * len;
   const float* z = p.P + (int64_t)t * p.ldp + (int64_t)part * len;
-  auto gated = [&](int i) {
-    const Vec<V> a = ldv<V>(y + i), g = ldv<V>(z + i);
+  auto gated = [&](const Vec<V>& a, const Vec<V>& g) {
     Vec<V> v;
 #pragma unroll
     for (int e = 0; e < V; ++e) v.x[e] = a.x[e] * silu_f(g.x[e]);
     return v;
   };
-  Vec<V> hold[HOLD];
+  Vec<V> hold[HOLD], gate[HOLD];
+#pragma unroll
+  for (int k = 0; k < HOLD; ++k) {
+    const int i = (k * W + tid) * V;
+    if (i < len) { hold[k] = ldv<V>(y + i); gate[k] = ldv<V>(z + i); }
+  }
   float ss = 0.f;
 #pragma unroll
   for (int k = 0; k < HOLD; ++k) {
-    const int i = (k * POST_THREADS + tid) * V;
-    if (i < len) {
-      hold[k] = gated(i);
+    if ((k * W + tid) * V >= len) continue;
+    hold[k] = gated(hold[k], gate[k]);
 #pragma unroll
-      for (int e = 0; e < V; ++e) ss = fmaf(hold[k].x[e], hold[k].x[e], ss);
-    }
+    for (int e = 0; e < V; ++e) ss = fmaf(hold[k].x[e], hold[k].x[e], ss);
   }
-  for (int i = (HOLD * POST_THREADS + tid) * V; i < len; i += POST_THREADS * V) {
-    const Vec<V> v = gated(i);
+  for (int i = (HOLD * W + tid) * V; i < len; i += W * V) {
+    const Vec<V> v = gated(ldv<V>(y + i), ldv<V>(z + i));
 #pragma unroll
     for (int e = 0; e < V; ++e) ss = fmaf(v.x[e], v.x[e], ss);
   }
-  ss = block_sum(ss, red);
+  ss = W == 32 ? warp_sum(ss) : block_sum(ss, red);
   const float inv = 1.f / sqrtf(ss / (float)len + eps);
   TO* o = out + (int64_t)t * ldo + (int64_t)part * len;
   const float* w = weight + (int64_t)part * len;
@@ -558,12 +575,12 @@ ssm_post_kernel(const Params p, const float* __restrict__ weight, float eps, int
   };
 #pragma unroll
   for (int k = 0; k < HOLD; ++k) {
-    const int i = (k * POST_THREADS + tid) * V;
+    const int i = (k * W + tid) * V;
     if (i < len) put(i, hold[k]);
   }
-  for (int i = (HOLD * POST_THREADS + tid) * V; i < len; i += POST_THREADS * V) put(i, gated(i));
+  for (int i = (HOLD * W + tid) * V; i < len; i += W * V) put(i, gated(ldv<V>(y + i), ldv<V>(z + i)));
   if (part == parts - 1)
-    for (int i = inner + tid; i < pad_to; i += POST_THREADS) out[(int64_t)t * ldo + i] = from_f32<TO>(0.f);
+    for (int i = inner + tid; i < pad_to; i += W) out[(int64_t)t * ldo + i] = from_f32<TO>(0.f);
 }
 
 template <int V, int L>
@@ -671,14 +688,23 @@ DINFER_API int dinfer_state_space_post(const float* y, const float* proj, int64_
   const int inner = p.inner(), len = inner / parts;
   if (ldp < (int64_t)inner + p.channels() || ldo < (pad_to > inner ? pad_to : inner) || ld_state < hist + (int64_t)(taps - 1) * p.channels())
     return refuse(DINFER_BAD_ARGUMENT, "state_space_post: a row stride is shorter than its row");
-  if ((int64_t)T * parts + B > 0x7fffffffLL) return refuse(DINFER_BAD_ARGUMENT, "state_space_post: too many rows for the grid");
+  if ((int64_t)T * parts + (int64_t)B * p.channels() > 0x7fffffffLL) return refuse(DINFER_BAD_ARGUMENT, "state_space_post: too many rows for the grid");
   if (T == 0) return 0;
-  const bool vec = len % 4 == 0 && ldp % 4 == 0 && ldo % 4 == 0 && al16(y) && al16(proj) && al16(weight) && al16(out);
-  const dim3 grid((unsigned)(T * parts + B));
+  const bool vec = len % 4 == 0 && p.channels() % 4 == 0 && hist % 4 == 0 && ld_state % 4 == 0 && ldp % 4 == 0 && ldo % 4 == 0 &&
+                   al16(state) && al16(y) && al16(proj) && al16(weight) && al16(out);
+  // parts that a warp can hold go a warp each (unless there are too few of them to fill the device)
+  const bool warps = len <= 32 * HOLD * (vec ? 4 : 1) && (int64_t)T * parts >= 592;
+  const int per = warps ? POST_THREADS / 32 : 1;
+  const int rows_ctas = (int)(((int64_t)T * parts + per - 1) / per);
+  const int run = POST_THREADS * (vec ? 4 : 1), jobs = taps > 1 ? (p.channels() + run - 1) / run : 0;
+  const dim3 grid((unsigned)(rows_ctas + (int64_t)B * jobs));
+#define GO(V, W) launch_pdl(ssm_post_kernel<TO, V, W>, grid, dim3(POST_THREADS), 0, stream, p, weight, eps, parts, (TO*)out, \
+                            ldo, pad_to, rows_ctas, jobs)
   DINFER_DISPATCH_DTYPE(out_dtype, TO, {
-    if (vec) launch_pdl(ssm_post_kernel<TO, 4>, grid, dim3(POST_THREADS), 0, stream, p, weight, eps, parts, (TO*)out, ldo, pad_to);
-    else launch_pdl(ssm_post_kernel<TO, 1>, grid, dim3(POST_THREADS), 0, stream, p, weight, eps, parts, (TO*)out, ldo, pad_to);
+    if (vec) { if (warps) GO(4, 32); else GO(4, POST_THREADS); }
+    else { if (warps) GO(1, 32); else GO(1, POST_THREADS); }
     return cuda_status("state_space_post");
   });
+#undef GO
   return 0;
 }
