@@ -268,10 +268,38 @@ __device__ __forceinline__ void chunk_log_decay(const float* la, int64_t ld, int
   cum[2 * lane + 1] = s;
 }
 
+// four neighbouring elements of which `left` are there (the others read as zeros); VEC: all four or none, 16-byte aligned
+template <bool VEC>
+__device__ __forceinline__ float4 load4(const float* p, int left) {
+  float4 v = make_float4(0.f, 0.f, 0.f, 0.f);
+  if (VEC) {
+    if (left > 0) v = *reinterpret_cast<const float4*>(p);
+  } else {
+    if (left > 0) v.x = p[0];
+    if (left > 1) v.y = p[1];
+    if (left > 2) v.z = p[2];
+    if (left > 3) v.w = p[3];
+  }
+  return v;
+}
+template <bool VEC>
+__device__ __forceinline__ void store4(float* p, int left, const float (&v)[4]) {
+  if (VEC) {
+    if (left > 0) *reinterpret_cast<float4*>(p) = make_float4(v[0], v[1], v[2], v[3]);
+  } else {
+#pragma unroll
+    for (int u = 0; u < 4; ++u)
+      if (left > u) p[u] = v[u];
+  }
+}
+__device__ __forceinline__ float4 get4(const float* p) { return *reinterpret_cast<const float4*>(p); }
+__device__ __forceinline__ void put4(float* p, const float4& v) { *reinterpret_cast<float4*>(p) = v; }
+
 // grid (chunks, H * tiles + G, B): a 64 x 64 tile of U for one (chunk, head), or the scores C_t . B_s of one (chunk, group)
+template <bool VEC>
 __global__ void __launch_bounds__(THREADS) ssm_sums_kernel(const Params p) {
-  __shared__ __align__(16) float a_s[CP][LDT];     // [token][state channel], or [channel][token s]
-  __shared__ __align__(16) float b_s[CP][LDT];     // [token][value column], scaled; or [channel][token t]
+  __shared__ __align__(16) float a_s[CP][LDT];     // [token][state channel] of B
+  __shared__ __align__(16) float b_s[CP][LDT];     // [token][value column], scaled; or [token][state channel] of C
   __shared__ double cum[CP];
   __shared__ float wgt[CP];
   pdl_enter();
@@ -283,58 +311,73 @@ __global__ void __launch_bounds__(THREADS) ssm_sums_kernel(const Params p) {
   const int n = min(CP, t_end - t0), ch = p.channels(), inner = p.inner();
   const int64_t slot = chunk_slot(t_begin, b, c);
   const int ty = tid >> 4, tx = tid & 15;
+  const int ls = tid >> 4, le = (tid & 15) * 4;    // this thread's place in a tile it loads: rows ls + 16 k, columns le ..
   float acc[4][4] = {};
   const int job = (int)blockIdx.y - p.H * tiles_n * tiles_v;
   if (job >= 0) {
-    // ---- scores of group `job`
+    // ---- scores of group `job`: rows t = 4 ty + i, columns s = tx + 16 j (neighbouring lanes read neighbouring rows)
     const float* Bp = p.xbc + (int64_t)t0 * ch + inner + job * p.N;
     const float* Cp = Bp + p.G * p.N;
     for (int e0 = 0; e0 < p.N; e0 += CP) {
-      const int ne = min(CP, p.N - e0);
       __syncthreads();
-      for (int i = tid; i < CP * CP; i += THREADS) {
-        const int s = i / CP, e = i % CP;
-        const bool live = s < n && e < ne;
-        a_s[e][s] = live ? Bp[(int64_t)s * ch + e0 + e] : 0.f;
-        b_s[e][s] = live ? Cp[(int64_t)s * ch + e0 + e] : 0.f;
+#pragma unroll
+      for (int k = 0; k < CP / 16; ++k) {
+        const int s = ls + 16 * k, left = s < n ? p.N - e0 - le : 0;
+        put4(&a_s[s][le], load4<VEC>(Bp + (int64_t)s * ch + e0 + le, left));
+        put4(&b_s[s][le], load4<VEC>(Cp + (int64_t)s * ch + e0 + le, left));
       }
       __syncthreads();
-#pragma unroll 8
-      for (int e = 0; e < ne; ++e) {
-        const float4 a = *reinterpret_cast<const float4*>(&b_s[e][ty * 4]);
-        const float4 w = *reinterpret_cast<const float4*>(&a_s[e][tx * 4]);
-        const float av[4] = {a.x, a.y, a.z, a.w}, wv[4] = {w.x, w.y, w.z, w.w};
+      const int ne = min(CP, p.N - e0);
+      for (int e = 0; e < ne; e += 4) {
+        float4 q[4], k4[4];
+#pragma unroll
+        for (int i = 0; i < 4; ++i) { q[i] = get4(&b_s[ty * 4 + i][e]); k4[i] = get4(&a_s[tx + 16 * i][e]); }
 #pragma unroll
         for (int i = 0; i < 4; ++i)
 #pragma unroll
-          for (int j = 0; j < 4; ++j) acc[i][j] = fmaf(av[i], wv[j], acc[i][j]);
+          for (int j = 0; j < 4; ++j) {
+            acc[i][j] = fmaf(q[i].x, k4[j].x, acc[i][j]);
+            acc[i][j] = fmaf(q[i].y, k4[j].y, acc[i][j]);
+            acc[i][j] = fmaf(q[i].z, k4[j].z, acc[i][j]);
+            acc[i][j] = fmaf(q[i].w, k4[j].w, acc[i][j]);
+          }
       }
     }
     float* out = p.cb + (slot * p.G + job) * (int64_t)CP * CP;      // [t][s]
 #pragma unroll
     for (int i = 0; i < 4; ++i)
-      *reinterpret_cast<float4*>(out + (ty * 4 + i) * CP + tx * 4) = make_float4(acc[i][0], acc[i][1], acc[i][2], acc[i][3]);
+#pragma unroll
+      for (int j = 0; j < 4; ++j) out[(ty * 4 + i) * CP + tx + 16 * j] = acc[i][j];
     return;
   }
   const int h = blockIdx.y / (tiles_n * tiles_v), tile = blockIdx.y % (tiles_n * tiles_v);
   const int e0 = (tile / tiles_v) * TP, c0 = (tile % tiles_v) * TP;
   const int g = h / (p.H / p.G);
+  float4 bv[CP / 16], xv[CP / 16];
+  {
+    const float* r = p.xbc + (int64_t)t0 * ch;
+#pragma unroll
+    for (int k = 0; k < CP / 16; ++k) {
+      const int s = ls + 16 * k;
+      bv[k] = load4<VEC>(r + (int64_t)s * ch + inner + g * p.N + e0 + le, s < n ? p.N - e0 - le : 0);
+      xv[k] = load4<VEC>(r + (int64_t)s * ch + h * p.Pd + c0 + le, s < n ? p.Pd - c0 - le : 0);
+    }
+  }
   if (tid < 32) chunk_log_decay(p.la + (int64_t)t0 * p.H + h, p.H, n, cum);
   __syncthreads();
   if (tid < CP) wgt[tid] = tid < n ? (float)exp(cum[n - 1] - cum[tid]) * p.dt[(int64_t)(t0 + tid) * p.H + h] : 0.f;
   if (tile == 0 && tid == 0) p.decay[slot * p.H + h] = (float)exp(cum[n - 1]);
   __syncthreads();
-  for (int i = tid; i < CP * TP; i += THREADS) {
-    const int s = i / TP, x = i % TP;
-    const float* r = p.xbc + (int64_t)(t0 + s) * ch;
-    a_s[s][x] = (s < n && e0 + x < p.N) ? r[inner + g * p.N + e0 + x] : 0.f;
-    b_s[s][x] = (s < n && c0 + x < p.Pd) ? r[h * p.Pd + c0 + x] * wgt[s] : 0.f;
+#pragma unroll
+  for (int k = 0; k < CP / 16; ++k) {
+    const float w = wgt[ls + 16 * k];
+    put4(&a_s[ls + 16 * k][le], bv[k]);
+    put4(&b_s[ls + 16 * k][le], make_float4(xv[k].x * w, xv[k].y * w, xv[k].z * w, xv[k].w * w));
   }
   __syncthreads();
-#pragma unroll 4
+#pragma unroll 8
   for (int s = 0; s < n; ++s) {
-    const float4 a = *reinterpret_cast<const float4*>(&a_s[s][ty * 4]);
-    const float4 w = *reinterpret_cast<const float4*>(&b_s[s][tx * 4]);
+    const float4 a = get4(&a_s[s][ty * 4]), w = get4(&b_s[s][tx * 4]);
     const float av[4] = {a.x, a.y, a.z, a.w}, wv[4] = {w.x, w.y, w.z, w.w};
 #pragma unroll
     for (int i = 0; i < 4; ++i)
@@ -343,12 +386,10 @@ __global__ void __launch_bounds__(THREADS) ssm_sums_kernel(const Params p) {
   }
   float* U = p.U + (slot * p.H + h) * (int64_t)p.N * p.Pd;
 #pragma unroll
-  for (int i = 0; i < 4; ++i)
-#pragma unroll
-    for (int j = 0; j < 4; ++j) {
-      const int e = e0 + ty * 4 + i, x = c0 + tx * 4 + j;
-      if (e < p.N && x < p.Pd) U[(int64_t)e * p.Pd + x] = acc[i][j];
-    }
+  for (int i = 0; i < 4; ++i) {
+    const int e = e0 + ty * 4 + i, x = c0 + tx * 4;
+    if (e < p.N) store4<VEC>(U + (int64_t)e * p.Pd + x, p.Pd - x, acc[i]);
+  }
 }
 
 // per V neighbouring elements of S: walk the request's chunks and leave in U's place the S that the chunk starts from;
@@ -395,13 +436,16 @@ __global__ void __launch_bounds__(THREADS) ssm_scan_kernel(const Params p) {
   stv<V>(S_g, S);
 }
 
-// y for one (chunk, head, 64 value columns); grid (chunks, H * column tiles, B)
-__global__ void __launch_bounds__(THREADS) ssm_outputs_kernel(const Params p) {
+// y for one (chunk, head, 64 value columns); grid (chunks, H * column tiles, B).  The passes over the state's channels load
+// the next pass's tiles into registers while they compute.
+template <bool VEC>
+__global__ void __launch_bounds__(THREADS, 3) ssm_outputs_kernel(const Params p) {
+  constexpr int LDC = KT + 4;
   __shared__ __align__(16) float tiles[CP * LDT];
-  static_assert(KT * LDT + KT * TP <= CP * LDT, "a pass's tiles fit where A lies afterwards");
-  float (*CT)[LDT] = reinterpret_cast<float (*)[LDT]>(tiles);                    // [state channel][token]
-  float (*S_s)[TP] = reinterpret_cast<float (*)[TP]>(tiles + KT * LDT);          // [state channel][value column]
-  float (*AT)[LDT] = reinterpret_cast<float (*)[LDT]>(tiles);                    // [token s][token t], after the passes
+  static_assert(CP * LDC + KT * TP <= CP * LDT, "a pass's tiles fit where A lies afterwards");
+  float (*C_s)[LDC] = reinterpret_cast<float (*)[LDC]>(tiles);                   // [token][state channel]
+  float (*S_s)[TP] = reinterpret_cast<float (*)[TP]>(tiles + CP * LDC);          // [state channel][value column]
+  float (*A_s)[LDT] = reinterpret_cast<float (*)[LDT]>(tiles);                   // [token t][token s], after the passes
   __shared__ __align__(16) float x_s[CP][TP];      // [token s][value column]
   __shared__ double cum[CP];
   __shared__ float dts[CP];
@@ -414,73 +458,99 @@ __global__ void __launch_bounds__(THREADS) ssm_outputs_kernel(const Params p) {
   const int n = min(CP, t_end - t0), tid = threadIdx.x, ch = p.channels(), inner = p.inner();
   const int ty = tid >> 4, tx = tid & 15, g = h / (p.H / p.G);
   const int64_t slot = chunk_slot(t_begin, b, c);
+  const float* S_prev = p.U + (slot * p.H + h) * (int64_t)p.N * p.Pd + c0;
+  const float* Cp = p.xbc + (int64_t)t0 * ch + inner + (p.G + g) * p.N;
+  // what this thread loads of a pass: C rows ct + 32 k at channels ce .., S rows (channels) sr + 16 k at columns sx ..
+  const int ct = tid >> 3, ce = (tid & 7) * 4, sr = tid >> 4, sx = (tid & 15) * 4;
+  float4 cv[CP / 32], sv[KT / 16];
+  auto fetch = [&](int e0) {
+#pragma unroll
+    for (int k = 0; k < CP / 32; ++k)
+      cv[k] = load4<VEC>(Cp + (int64_t)(ct + 32 * k) * ch + e0 + ce, ct + 32 * k < n ? p.N - e0 - ce : 0);
+#pragma unroll
+    for (int k = 0; k < KT / 16; ++k)
+      sv[k] = load4<VEC>(S_prev + (int64_t)(e0 + sr + 16 * k) * p.Pd + sx, e0 + sr + 16 * k < p.N ? p.Pd - c0 - sx : 0);
+  };
+  fetch(0);
+#pragma unroll
+  for (int k = 0; k < CP / 16; ++k) {
+    const int s = sr + 16 * k;
+    put4(&x_s[s][sx], load4<VEC>(p.xbc + (int64_t)(t0 + s) * ch + h * p.Pd + c0 + sx, s < n ? p.Pd - c0 - sx : 0));
+  }
   if (tid < 32) chunk_log_decay(p.la + (int64_t)t0 * p.H + h, p.H, n, cum);
   if (tid < CP) dts[tid] = tid < n ? p.dt[(int64_t)(t0 + tid) * p.H + h] : 0.f;
-  for (int i = tid; i < CP * TP; i += THREADS) {
-    const int s = i / TP, x = i % TP;
-    x_s[s][x] = (s < n && c0 + x < p.Pd) ? p.xbc[(int64_t)(t0 + s) * ch + h * p.Pd + c0 + x] : 0.f;
-  }
-  const float* S_prev = p.U + (slot * p.H + h) * (int64_t)p.N * p.Pd;
-  const float* Cp = p.xbc + (int64_t)t0 * ch + inner + (p.G + g) * p.N;
   float r[4][4] = {};
   for (int e0 = 0; e0 < p.N; e0 += KT) {
-    __syncthreads();
-    for (int i = tid; i < CP * KT; i += THREADS) {
-      const int t = i / KT, e = i % KT;
-      CT[e][t] = (t < n && e0 + e < p.N) ? Cp[(int64_t)t * ch + e0 + e] : 0.f;
-    }
-    for (int i = tid; i < KT * TP; i += THREADS) {
-      const int e = i / TP, x = i % TP;
-      S_s[e][x] = (e0 + e < p.N && c0 + x < p.Pd) ? S_prev[(int64_t)(e0 + e) * p.Pd + c0 + x] : 0.f;
-    }
-    __syncthreads();
-#pragma unroll 8
-    for (int e = 0; e < KT; ++e) {
-      const float4 q4 = *reinterpret_cast<const float4*>(&CT[e][ty * 4]);
-      const float4 s4 = *reinterpret_cast<const float4*>(&S_s[e][tx * 4]);
-      const float qv[4] = {q4.x, q4.y, q4.z, q4.w}, sv[4] = {s4.x, s4.y, s4.z, s4.w};
+    __syncthreads();                               // the last pass is done with the tiles
 #pragma unroll
-      for (int i = 0; i < 4; ++i)
+    for (int k = 0; k < CP / 32; ++k) put4(&C_s[ct + 32 * k][ce], cv[k]);
 #pragma unroll
-        for (int j = 0; j < 4; ++j) r[i][j] = fmaf(qv[i], sv[j], r[i][j]);
+    for (int k = 0; k < KT / 16; ++k) put4(&S_s[sr + 16 * k][sx], sv[k]);
+    __syncthreads();
+    if (e0 + KT < p.N) fetch(e0 + KT);
+#pragma unroll 2
+    for (int e = 0; e < KT; e += 4) {
+      float4 q[4];
+#pragma unroll
+      for (int i = 0; i < 4; ++i) q[i] = get4(&C_s[ty * 4 + i][e]);
+#pragma unroll
+      for (int u = 0; u < 4; ++u) {
+        const float4 s4 = get4(&S_s[e + u][tx * 4]);
+        const float sw[4] = {s4.x, s4.y, s4.z, s4.w};
+#pragma unroll
+        for (int i = 0; i < 4; ++i) {
+          const float qv = u == 0 ? q[i].x : u == 1 ? q[i].y : u == 2 ? q[i].z : q[i].w;
+#pragma unroll
+          for (int j = 0; j < 4; ++j) r[i][j] = fmaf(qv, sw[j], r[i][j]);
+        }
+      }
     }
   }
   __syncthreads();
-  // A[s][t] = (C_t . B_s) exp(c_t - c_s) dt_s for s <= t
+  // A[t][s] = (C_t . B_s) exp(c_t - c_s) dt_s for s <= t; r <- exp(c_t) r, which the sums over s then join
   const float* cb = p.cb + (slot * p.G + g) * (int64_t)CP * CP;
 #pragma unroll
   for (int i = 0; i < 4; ++i) {
     const int t = ty * 4 + i;
-    const float4 v = *reinterpret_cast<const float4*>(cb + t * CP + tx * 4);
+    const float4 v = get4(cb + t * CP + tx * 4);
     const float vv[4] = {v.x, v.y, v.z, v.w};
+    float a[4];
 #pragma unroll
     for (int j = 0; j < 4; ++j) {
       const int s = tx * 4 + j;
-      AT[s][t] = (s <= t && t < n) ? vv[j] * expf((float)(cum[t] - cum[s])) * dts[s] : 0.f;
+      a[j] = (s <= t && t < n) ? vv[j] * expf((float)(cum[t] - cum[s])) * dts[s] : 0.f;
     }
+    put4(&A_s[t][tx * 4], make_float4(a[0], a[1], a[2], a[3]));
+    const float d = expf((float)cum[t]);
+#pragma unroll
+    for (int j = 0; j < 4; ++j) r[i][j] *= d;
   }
   __syncthreads();
-  float o[4][4] = {};
-  const int last = min(ty * 4 + 3, n - 1);
-  for (int s = 0; s <= last; ++s) {
-    const float4 a4 = *reinterpret_cast<const float4*>(&AT[s][ty * 4]);
-    const float4 v4 = *reinterpret_cast<const float4*>(&x_s[s][tx * 4]);
-    const float av[4] = {a4.x, a4.y, a4.z, a4.w}, vv[4] = {v4.x, v4.y, v4.z, v4.w};
+  const int last = min(ty * 4 + 3, n - 1);         // (A is zero beyond t, x_s beyond the chunk's tokens)
+  for (int s = 0; s <= last; s += 4) {
+    float4 q[4];
 #pragma unroll
-    for (int i = 0; i < 4; ++i)
+    for (int i = 0; i < 4; ++i) q[i] = get4(&A_s[ty * 4 + i][s]);
 #pragma unroll
-      for (int j = 0; j < 4; ++j) o[i][j] = fmaf(av[i], vv[j], o[i][j]);
+    for (int u = 0; u < 4; ++u) {
+      const float4 x4 = get4(&x_s[s + u][tx * 4]);
+      const float xw[4] = {x4.x, x4.y, x4.z, x4.w};
+#pragma unroll
+      for (int i = 0; i < 4; ++i) {
+        const float qv = u == 0 ? q[i].x : u == 1 ? q[i].y : u == 2 ? q[i].z : q[i].w;
+#pragma unroll
+        for (int j = 0; j < 4; ++j) r[i][j] = fmaf(qv, xw[j], r[i][j]);
+      }
+    }
   }
   const float D = p.D[h];
 #pragma unroll
   for (int i = 0; i < 4; ++i) {
     const int t = ty * 4 + i;
     if (t >= n) continue;
-    const float d = expf((float)cum[t]);
-    float* dst = p.y + (int64_t)(t0 + t) * inner + (int64_t)h * p.Pd + c0 + tx * 4;
-#pragma unroll
-    for (int j = 0; j < 4; ++j)
-      if (c0 + tx * 4 + j < p.Pd) dst[j] = fmaf(D, x_s[t][tx * 4 + j], fmaf(d, r[i][j], o[i][j]));
+    const float4 x4 = get4(&x_s[t][tx * 4]);
+    const float o[4] = {fmaf(D, x4.x, r[i][0]), fmaf(D, x4.y, r[i][1]), fmaf(D, x4.z, r[i][2]), fmaf(D, x4.w, r[i][3])};
+    store4<VEC>(p.y + (int64_t)(t0 + t) * inner + (int64_t)h * p.Pd + c0 + tx * 4, p.Pd - c0 - tx * 4, o);
   }
 }
 
@@ -665,10 +735,12 @@ DINFER_API int dinfer_state_space(const float* proj, int64_t ldp, const float* c
     p.decay = p.la + r4((int64_t)T * H);
     if (ch % 4 == 0 && ldp % 4 == 0 && inner % 4 == 0 && al16(proj)) launch_prep<4>(p, stream);
     else launch_prep<1>(p, stream);
-    launch_pdl(ssm_sums_kernel, dim3(chunks, H * tiles_n * tiles_v + G, B), dim3(THREADS), 0, stream, p);
+    // 16-byte loads of the convolved rows, of the states and of y: every width and base allows them
+    const bool vec = P % 4 == 0 && N % 4 == 0 && al16(y);
+    launch_pdl(vec ? ssm_sums_kernel<true> : ssm_sums_kernel<false>, dim3(chunks, H * tiles_n * tiles_v + G, B), dim3(THREADS), 0, stream, p);
     if (state_vec) launch_pdl(ssm_scan_kernel<4>, dim3((unsigned)((size / 4 + THREADS - 1) / THREADS), B), dim3(THREADS), 0, stream, p);
     else launch_pdl(ssm_scan_kernel<1>, dim3((unsigned)((size + THREADS - 1) / THREADS), B), dim3(THREADS), 0, stream, p);
-    launch_pdl(ssm_outputs_kernel, dim3(chunks, H * tiles_v, B), dim3(THREADS), 0, stream, p);
+    launch_pdl(vec ? ssm_outputs_kernel<true> : ssm_outputs_kernel<false>, dim3(chunks, H * tiles_v, B), dim3(THREADS), 0, stream, p);
   }
   return cuda_status("state_space");
 }
