@@ -9,8 +9,8 @@
 //
 //   ssm_step      requests that bring one token: convolution, step size, state and read-out in one launch, a CTA per
 //                 (request, head, run of columns).  S goes through registers: its loads are asked for before the kernels
-//                 in front have finished (no kernel of a step but this one touches S), each element is read and written
-//                 once.  The decay is applied as S + S * expm1(..), which keeps the digits of a decay just below one.
+//                 in front have finished (no kernel of a step but this one touches a single token's S, and none in
+//                 front of it its convolution's inputs), each element is read and written once.  The decay is applied as S + S * expm1(..), which keeps the digits of a decay just below one.
 //   ssm_prep      requests that bring more: convolution and silu of x, B, C; dt and the decay's logarithm
 //   ssm_sums, ssm_scan, ssm_outputs
 //                 their chunks of 64 tokens side by side.  With c_t the running sum of the decays' logarithms inside a
@@ -90,22 +90,28 @@ __global__ void __launch_bounds__(THREADS, RPT == 16 ? 2 : (RPT == 8 ? 3 : 4)) s
   }
   const float* hist = row_state + p.hist;
   const int inner = p.inner(), ch = p.channels(), g = h / (p.H / p.G);
+  auto channel = [&](int i) {                                       // of x | B | C; -1: none
+    if (i < p.N) return inner + g * p.N + i;
+    if (i < 2 * p.N) return inner + (p.G + g) * p.N + i - p.N;
+    return c0 + i - 2 * p.N < p.Pd ? h * p.Pd + c0 + i - 2 * p.N : -1;
+  };
+  // the convolution's part of earlier inputs, which no kernel in front of this one writes either; each thread ends what it began
+  for (int i = tid; i < 2 * p.N + PT; i += THREADS) {
+    const int c = channel(i);
+    float a = 0.f;
+    if (c >= 0) {
+      const float* w = p.conv_w + (int64_t)c * p.taps;
+      a = p.conv_b[c];
+      if (!is_fresh)
+        for (int d = 0; d < p.taps - 1; ++d) a = fmaf(w[d], hist[(int64_t)d * ch + c], a);
+    }
+    sm[i] = a;
+  }
   pdl_wait();
   const float* row = p.P + (int64_t)t * p.ldp + inner;             // the convolution's inputs
   for (int i = tid; i < 2 * p.N + PT; i += THREADS) {
-    int c;                                                          // channel of x | B | C
-    if (i < p.N) c = inner + g * p.N + i;
-    else if (i < 2 * p.N) c = inner + (p.G + g) * p.N + i - p.N;
-    else c = c0 + i - 2 * p.N < p.Pd ? h * p.Pd + c0 + i - 2 * p.N : -1;
-    float v = 0.f;
-    if (c >= 0) {
-      const float* w = p.conv_w + (int64_t)c * p.taps;
-      float a = p.conv_b[c];
-      if (!is_fresh)
-        for (int d = 0; d < p.taps - 1; ++d) a = fmaf(w[d], hist[(int64_t)d * ch + c], a);
-      v = silu_f(fmaf(w[p.taps - 1], row[c], a));
-    }
-    sm[i] = v;
+    const int c = channel(i);
+    if (c >= 0) sm[i] = silu_f(fmaf(p.conv_w[(int64_t)c * p.taps + p.taps - 1], row[c], sm[i]));
   }
   const float dt = softplus_f(row[ch + h] + p.dt_bias[h]);
   const float g1 = expm1f(-expf(p.A_log[h]) * dt);
