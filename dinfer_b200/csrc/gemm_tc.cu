@@ -167,8 +167,9 @@ __device__ __forceinline__ float silu_mul_fast(float g, float u) { return __fdiv
 __device__ __forceinline__ float gelu_tanh_mul(float g, float u) {
   return 0.5f * g * (1.f + tanhf(0.7978845608028654f * (g + 0.044715f * g * g * g))) * u;
 }
+template <bool CLAMPED>
 __device__ __forceinline__ float gate_mul(float g, float u, const GemmParams& p) {
-  if (p.act == 3) return clamped_swish(g, u, p.a_pos, p.a_neg);
+  if (CLAMPED && p.act == 3) return clamped_swish(g, u, p.a_pos, p.a_neg);
   return p.act == 2 ? gelu_tanh_mul(g, u) : silu_mul(g, u);
 }
 __device__ __forceinline__ float grouped_act(float z, const GemmParams& p) {
@@ -194,7 +195,8 @@ template <int N_TILE, int STAGES> constexpr size_t gemm_smem_bytes(bool with_rec
 }
 
 // grid: (tiles of the 128-row operand, tiles of the N_TILE-row operand, K splits)
-// UNARY: the activation grp_act on the result (kernels of their own: its code slows the plain product down)
+// UNARY: the activation grp_act on the result, or the clamped gate (kernels of their own: their code slows the plain
+// product down)
 template <int N_TILE, int STAGES, typename OutT, bool UNARY>
 __global__ void __launch_bounds__(NTHREADS)
 gemm_tc_kernel(const __grid_constant__ CUtensorMap map_a, const __grid_constant__ CUtensorMap map_b, const GemmParams p) {
@@ -356,7 +358,7 @@ gemm_tc_kernel(const __grid_constant__ CUtensorMap map_a, const __grid_constant_
               const float g = __uint_as_float(v[j]);
               const float u = __shfl_down_sync(0xffffffffu, g, 1);
               if (!(lane & 1) && n + 1 < p.N && b0 + c0 + j < p.tokens)
-                out[(int64_t)(b0 + c0 + j) * p.ldc + (n >> 1)] = out_cast<OutT>(gate_mul(g, u, p));
+                out[(int64_t)(b0 + c0 + j) * p.ldc + (n >> 1)] = out_cast<OutT>(gate_mul<UNARY>(g, u, p));
             }
           } else if (!clustered) {
             if (n < p.N) {
@@ -446,7 +448,7 @@ gemm_tc_kernel(const __grid_constant__ CUtensorMap map_a, const __grid_constant_
           }
           if (p.ss_in) { g *= s_rstd[c]; u *= s_rstd[c]; }
           const int n = a0 + rank * rows_per + 2 * pr;
-          if (n + 1 < p.N) out[(int64_t)(b0 + c) * p.ldc + (n >> 1)] = out_cast<OutT>(gate_mul(g, u, p));
+          if (n + 1 < p.N) out[(int64_t)(b0 + c) * p.ldc + (n >> 1)] = out_cast<OutT>(gate_mul<UNARY>(g, u, p));
         }
       } else {
         for (int i = threadIdx.x; i < cols * rows_mine; i += NTHREADS) {
@@ -480,11 +482,12 @@ gemm_tc_kernel(const __grid_constant__ CUtensorMap map_a, const __grid_constant_
 // CTAs are persistent: a pair walks over tiles (token tile fastest, so that pairs running at the same time read the
 // same few weight tiles from L2), the shared-memory ring runs on across tiles, and the accumulator is double-buffered
 // in tensor memory (2 x 256 columns): the epilogue warps drain tile i while the MMAs of tile i + 1 run.  With
-// EPI_GATED the weight rows are (gate, up) pairs and the epilogue writes silu(gate) * up, half as wide; with EPI_ACT it
+// EPI_GATED the weight rows are (gate, up) pairs and the epilogue writes silu(gate) * up, half as wide, with EPI_CLAMPED
+// the clamped gate; with EPI_ACT it
 // applies the activation grp_act, with EPI_XIELU that one.
 // (Narrower tiles, chosen so that the last round of tiles leaves fewer SMs idle, were measured and are slower at
 // every shape.)
-constexpr int EPI_PLAIN = 0, EPI_GATED = 1, EPI_ACT = 2, EPI_XIELU = 3;
+constexpr int EPI_PLAIN = 0, EPI_GATED = 1, EPI_ACT = 2, EPI_XIELU = 3, EPI_CLAMPED = 4;
 constexpr int NT = 256;                                                       // columns of the pair's tile
 constexpr int C_STAGES = 6, C_ACC_BUFS = 2, C_TMEM_COLS = NT * C_ACC_BUFS;
 constexpr uint32_t C_A_BYTES = TILE_M * BLOCK_K * 2, C_B_BYTES = (NT / 2) * BLOCK_K * 2;   // this CTA's rows of both operands
@@ -612,7 +615,7 @@ gemm_tc_pair_kernel(const __grid_constant__ CUtensorMap map_a, const __grid_cons
     const int r = quarter * 32 + lane;
     OutT* out = reinterpret_cast<OutT*>(p.out);
     const bool vec = sizeof(OutT) == 2 && (p.ldc % 8 == 0) && ((reinterpret_cast<uintptr_t>(p.out) & 15) == 0);
-    const int n_out = EPI == EPI_GATED ? p.N / 2 : p.N;
+    const int n_out = EPI == EPI_GATED || EPI == EPI_CLAMPED ? p.N / 2 : p.N;
     uint32_t lt = 0;
     for (int tile = pair; tile < tiles; tile += pairs, ++lt) {
       if (p.tile_expert && p.tile_expert[m_of(tile)] < 0) { --lt; continue; }         // a tile without rows
@@ -664,13 +667,13 @@ gemm_tc_pair_kernel(const __grid_constant__ CUtensorMap map_a, const __grid_cons
         }
 #pragma unroll
         for (int h = 0; h < 2; ++h) {
-          if constexpr (EPI == EPI_GATED) {
+          if constexpr (EPI == EPI_GATED || EPI == EPI_CLAMPED) {
             const int o0 = (n0 + c0 + h * 16) >> 1;
             OutT* dst = out + (int64_t)t * p.ldc + o0;
             float y[8];
 #pragma unroll
             for (int j = 0; j < 8; ++j)
-              y[j] = p.act == 3 ? clamped_swish_fast(__uint_as_float(v[h][2 * j]), __uint_as_float(v[h][2 * j + 1]), p.a_pos, p.a_neg)
+              y[j] = EPI == EPI_CLAMPED ? clamped_swish_fast(__uint_as_float(v[h][2 * j]), __uint_as_float(v[h][2 * j + 1]), p.a_pos, p.a_neg)
                      : p.act == 2 ? gelu_tanh_mul(__uint_as_float(v[h][2 * j]), __uint_as_float(v[h][2 * j + 1]))
                                   : silu_mul_fast(__uint_as_float(v[h][2 * j]), __uint_as_float(v[h][2 * j + 1]));
             if (vec && o0 + 8 <= n_out) {
@@ -773,7 +776,7 @@ int launch_decode(const CUtensorMap& ma, const CUtensorMap& mb, const GemmParams
 }
 template <int N_TILE, int STAGES, typename OutT>
 int launch(const CUtensorMap& ma, const CUtensorMap& mb, const GemmParams& p, dim3 grid, cudaStream_t stream) {
-  return p.grp_act ? launch_decode<N_TILE, STAGES, OutT, true>(ma, mb, p, grid, stream)
+  return p.grp_act || p.act == 3 ? launch_decode<N_TILE, STAGES, OutT, true>(ma, mb, p, grid, stream)
                    : launch_decode<N_TILE, STAGES, OutT, false>(ma, mb, p, grid, stream);
 }
 
@@ -921,7 +924,7 @@ DINFER_API int dinfer_gemm_tc_all(const void* x, int64_t ldx, const void* w, int
   if ((rc = make_map(&ma, x, tokens, K, ldx, TILE_M))) return rc;
   if ((rc = make_map(&mb, w, N, K, ldw, NT / 2))) return rc;
 #define GO(EPI) (out_f32 ? launch_pair<float, EPI>(ma, mb, p, stream) : launch_pair<__nv_bfloat16, EPI>(ma, mb, p, stream))
-  if (act) return GO(EPI_GATED);
+  if (act) return act == 3 ? GO(EPI_CLAMPED) : GO(EPI_GATED);
   if (unary == 5) return GO(EPI_XIELU);
   return unary ? GO(EPI_ACT) : GO(EPI_PLAIN);
 #undef GO
@@ -961,7 +964,7 @@ DINFER_API int dinfer_gemm_tc_grouped(const void* x, int64_t ldx, const void* w,
   int rc;
   if ((rc = make_map(&ma, x, cap, K, ldx, TILE_M))) return rc;
   if ((rc = make_map(&mb, w, (int64_t)E * N, K, K, NT / 2))) return rc;
-  if (gate) return launch_pair<__nv_bfloat16, EPI_GATED>(ma, mb, p, stream);
+  if (gate) return gate == 3 ? launch_pair<__nv_bfloat16, EPI_CLAMPED>(ma, mb, p, stream) : launch_pair<__nv_bfloat16, EPI_GATED>(ma, mb, p, stream);
   return act ? launch_pair<__nv_bfloat16, EPI_ACT>(ma, mb, p, stream) : launch_pair<__nv_bfloat16, EPI_PLAIN>(ma, mb, p, stream);
 }
 
